@@ -9,7 +9,7 @@ from __future__ import annotations
 
 import dataclasses
 from dataclasses import dataclass
-from typing import Any, Mapping, Optional
+from typing import Any, Mapping, Optional, Union
 
 import torch
 
@@ -244,6 +244,176 @@ class LlamaConfig:
         if name not in presets:
             raise KeyError(f"unknown model {name!r}; have {sorted(presets)}")
         kw = dict(presets[name])
+        kw.update(over)
+        return cls(**kw)
+
+
+@dataclass(frozen=True)
+class RotaryConfig:
+    """Rotary positions on the first ``dims`` dimensions of a vector, pairs (2i, 2i + 1), frequencies
+    ``base ** (-2i / dims)``."""
+
+    base: float
+    dims: int
+
+    def inv_freq(self) -> list:
+        return [float(self.base) ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+
+
+@dataclass(frozen=True)
+class LatentAttentionConfig:
+    """Latent attention: per token a ``kv_rank`` latent and one rotated key part of ``rot_dim`` are cached; heads have
+    ``dim`` unrotated and ``rot_dim`` rotated query/key dimensions and ``vdim`` value dimensions."""
+
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot: RotaryConfig
+
+    def __post_init__(self):
+        if self.rot.dims % 2 or not 0 <= self.rot.dims <= self.rot_dim:
+            raise ValueError("rotary dims must be even and at most rot_dim")
+
+
+@dataclass(frozen=True)
+class GatedDeltaConfig:
+    """Gated delta rule with short convolutions over ``conv`` tokens: ``heads`` states of ``dim`` x ``vdim``, value head h
+    uses q/k head ``h // (heads // kv_heads)``."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+
+
+@dataclass(frozen=True)
+class DenseConfig:
+    """Two-matrix feed-forward ``down(relu(up x)^2)``."""
+
+    ff: int
+
+
+MixerConfig = Union[LatentAttentionConfig, GatedDeltaConfig]
+
+
+@dataclass(frozen=True)
+class LayerConfig:
+    """One decoder layer: a mixer, an optional feed-forward and, when the layer has no tensors of its own, the index of
+    the layer whose tensors it uses (its cache or state is its own all the same)."""
+
+    mixer: MixerConfig
+    mlp: Optional[DenseConfig] = None
+    weights_of: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class HybridConfig:
+    """Decoder whose layers are listed one by one, each with a mixer of its own kind. Mixer and feed-forward of a layer
+    read the same residual stream through norms of their own and are added to it together (the Dafelorn design)."""
+
+    vocab_size: int
+    d_model: int
+    layers: tuple
+    rms_eps: float
+    norm_gain_offset: float = 1.0     # gains of the layer and final norms are stored around zero
+
+    ARCHITECTURE = "Dafelorn"
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    def owner(self, i: int) -> int:
+        """The layer whose tensors layer ``i`` uses."""
+        seen = set()
+        while self.layers[i].weights_of is not None:
+            if i in seen:
+                raise ValueError("weights_of goes round in a circle")
+            seen.add(i)
+            i = self.layers[i].weights_of
+        return i
+
+    def n_params(self, include_embedding: bool = True) -> int:
+        d = self.d_model
+        n = self.vocab_size * d * (2 if include_embedding else 1)
+        for i, layer in enumerate(self.layers):
+            if self.owner(i) != i:
+                continue
+            m = layer.mixer
+            if isinstance(m, LatentAttentionConfig):
+                n += d * (m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim + m.heads + m.heads * m.vdim)
+                n += m.kv_rank * m.heads * (m.dim + m.vdim)
+            else:
+                n += d * (2 * m.kv_heads * m.dim + 3 * m.heads * m.vdim + 2 * m.heads)
+            if layer.mlp is not None:
+                n += 2 * d * layer.mlp.ff
+        return n
+
+    def cache_bytes_per_token(self, element_bytes: int = 2) -> int:
+        return sum((l.mixer.kv_rank + l.mixer.rot_dim) * element_bytes for l in self.layers
+                   if isinstance(l.mixer, LatentAttentionConfig))
+
+    @classmethod
+    def from_dict(cls, c: Mapping[str, Any]) -> "HybridConfig":
+        """Parse a ``config.json`` of this design."""
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            m = e["mixer"]
+            if e["type"] == "latent_attention":
+                mixer = LatentAttentionConfig(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"],
+                                              kv_rank=m["kv_rank"], scale=m["scale"],
+                                              rot=RotaryConfig(base=m["rot"]["base"], dims=m["rot"]["dims"]))
+            elif e["type"] == "delta":
+                mixer = GatedDeltaConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
+                                         conv=m["conv"])
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            mlp = e.get("mlp")
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            w = e.get("weights_of")
+            if w is not None and not 0 <= w < len(c["layers"]):
+                raise ValueError(f"layer {i}: weights_of {w} is not a layer")
+            layers.append(LayerConfig(mixer, None if mlp is None else DenseConfig(ff=mlp["ff"]), w))
+        out = cls(vocab_size=c["vocab"], d_model=c["width"], layers=tuple(layers), rms_eps=c["norm"]["eps"])
+        for i in range(out.n_layers):
+            j = out.owner(i)
+            if (out.layers[i].mixer, out.layers[i].mlp) != (out.layers[j].mixer, out.layers[j].mlp):
+                raise ValueError(f"layer {i} uses the tensors of layer {j} but has other sizes")
+        return out
+
+    @classmethod
+    def named(cls, name: str, **over) -> "HybridConfig":
+        """Presets of LLaMA-like sizes, three delta layers to one latent-attention layer."""
+        def stack(n, heads, dim, rot, rank, ff, dk):
+            lat = LatentAttentionConfig(heads=heads, dim=dim, rot_dim=rot, vdim=dim, kv_rank=rank,
+                                        scale=(dim + rot) ** -0.5, rot=RotaryConfig(10000.0, rot))
+            dl = GatedDeltaConfig(heads=heads, kv_heads=heads // 2, dim=dk, vdim=dk, conv=4)
+            return tuple(LayerConfig(lat if i % 4 == 3 else dl, DenseConfig(ff)) for i in range(n))
+
+        presets = {
+            "dafelorn-7b": dict(vocab_size=32000, d_model=4096, rms_eps=1e-6,
+                                stack=dict(n=32, heads=32, dim=128, rot=64, rank=512, ff=16512, dk=128)),
+            "dafelorn-1b": dict(vocab_size=32000, d_model=2048, rms_eps=1e-6,
+                                stack=dict(n=16, heads=16, dim=128, rot=64, rank=512, ff=8256, dk=128)),
+            "dafelorn-tiny": dict(vocab_size=1024, d_model=256, rms_eps=1e-6,
+                                  stack=dict(n=4, heads=2, dim=64, rot=32, rank=64, ff=768, dk=64)),
+        }
+        if name not in presets:
+            raise KeyError(f"unknown model {name!r}; have {sorted(presets)}")
+        kw = dict(presets[name])
+        st = dict(kw.pop("stack"))
+        if "n_layers" in over:
+            st["n"] = over.pop("n_layers")
+        kw["layers"] = stack(**st)
         kw.update(over)
         return cls(**kw)
 

@@ -1,0 +1,396 @@
+// Gated delta rule with short convolutions: the kernels around and of the recurrence
+//     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+// with one state S (dk x dv, fp32) per value head and per sequence.
+//   delta_prep_kernel : causal convolution over time + silu of the q, k and v channels, unit norms of q and k per head,
+//                       decay g and step size beta from their projections. One warp per (token, head).
+//   delta_scan_kernel : the recurrence over the tokens of a step. Columns of S (one per value channel) are independent:
+//                       eight lanes own one column, dk / 8 state elements each, in registers for the whole step; both
+//                       read-outs of a token (with k and with q) are taken from the decayed state before the write,
+//                       o = S'^T q + (q.k) u, so a token costs one reduction over eight lanes.
+//   delta_out_kernel  : per-head RMS norm of o, gain, silu gate.
+//   delta_step_kernel : all of it for one token per sequence (decode), one CTA per value head.
+// The convolution's history is a ring of `taps` rows per sequence, the row of position p at p % taps, kept in fp32: a
+// step reads the rows of the taps - 1 tokens before it and writes the rows of its own last tokens. The state is stored
+// transposed, (dv, dk), so that the eight lanes of a column read 128 contiguous bytes.
+// Everything here is fp32 except the projections that come in.
+#include "common/bounds.cuh"
+#include "common/host_util.h"
+#include "common/numeric.cuh"
+
+RA_BOUNDS_TRANSLATION_UNIT()
+
+namespace ra {
+namespace delta {
+
+struct Params {
+  int B, T, H, G, dk, dv, taps;  // T tokens per sequence in this step; row b * T + t
+  const void* proj;              // (rows, ldp): columns off_q / off_k / off_v / off_g
+  long long ldp;
+  int off_q, off_k, off_v, off_g;
+  const float* ba;               // (rows, ldba): beta's projection at 0, the decay's at off_a
+  long long ldba;
+  int off_a;
+  const void *conv_q, *conv_k, *conv_v;  // (channels, taps)
+  const void *a_log, *dt_bias, *norm_w;  // (H), (H), (dv)
+  float* ring;                   // (B, taps, C) with C = 2 G dk + H dv, channels in the order q, k, v
+  float* state;                  // (B, H, dv, dk)
+  float *q, *k, *v, *gb, *o;     // (rows, G, dk) x 2, (rows, H, dv), (rows, H, 2), (rows, H, dv)
+  void* out;                     // (rows, ldo)
+  long long ldo;
+  float eps, q_scale;
+  const long long* pos;          // position of the step's first token
+};
+
+__device__ __forceinline__ int ring_slot(long long p, int taps) { return static_cast<int>(p % taps); }
+
+// silu(convolution) of one channel at token t of the step. `c`: channel in the ring's order, `col`: its projection column.
+template <typename T>
+__device__ __forceinline__ float conv_silu(const Params& p, const T* proj_b, const float* ring_b, const T* w, int t,
+                                           long long pos0, int C, int c, int col) {
+  float s = 0.f;
+  for (int j = 0; j < p.taps; ++j) {
+    const int tt = t - (p.taps - 1 - j);
+    float x = 0.f;
+    if (tt >= 0)
+      x = to_f(proj_b[tt * p.ldp + col]);
+    else if (pos0 + tt >= 0)
+      x = ring_b[static_cast<long long>(ring_slot(pos0 + tt, p.taps)) * C + c];
+    s = fmaf(to_f(w[j]), x, s);
+  }
+  return silu_f(s);
+}
+
+__device__ __forceinline__ float decay_of(const Params& p, float a, float a_log, float dt) {
+  return expf(-expf(a_log) * softplus_f(a + dt));
+}
+
+// grid (rows, ceil((2 G + H) / 4)), four warps; unit u: q head u, k head u - G, v head u - 2 G
+template <typename T>
+__global__ void __launch_bounds__(128) delta_prep_kernel(const Params p) {
+  const int row = blockIdx.x, u = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (u >= 2 * p.G + p.H) return;
+  const int b = row / p.T, t = row - b * p.T;
+  const long long pos0 = *p.pos;
+  const int C = 2 * p.G * p.dk + p.H * p.dv;
+  const T* proj_b = static_cast<const T*>(p.proj) + static_cast<long long>(b) * p.T * p.ldp;
+  const float* ring_b = p.ring + static_cast<long long>(b) * p.taps * C;
+  if (u < 2 * p.G) {
+    const bool is_q = u < p.G;
+    const int hd = is_q ? u : u - p.G;
+    const T* w = static_cast<const T*>(is_q ? p.conv_q : p.conv_k) + static_cast<long long>(hd) * p.dk * p.taps;
+    const int col = (is_q ? p.off_q : p.off_k) + hd * p.dk, c0 = u * p.dk;
+    float* dst = (is_q ? p.q : p.k) + (static_cast<long long>(row) * p.G + hd) * p.dk;
+    float ss = 0.f;
+    for (int i = lane; i < p.dk; i += 32) {
+      const float x = conv_silu(p, proj_b, ring_b, w + i * p.taps, t, pos0, C, c0 + i, col + i);
+      dst[i] = x;
+      ss += x * x;
+    }
+    const float mul = (is_q ? p.q_scale : 1.f) / sqrtf(sum_warp(ss) + 1e-6f);
+    for (int i = lane; i < p.dk; i += 32) dst[i] *= mul;
+  } else {
+    const int hd = u - 2 * p.G;
+    const T* w = static_cast<const T*>(p.conv_v) + static_cast<long long>(hd) * p.dv * p.taps;
+    const int c0 = 2 * p.G * p.dk + hd * p.dv;
+    float* dst = p.v + (static_cast<long long>(row) * p.H + hd) * p.dv;
+    for (int i = lane; i < p.dv; i += 32)
+      dst[i] = conv_silu(p, proj_b, ring_b, w + i * p.taps, t, pos0, C, c0 + i, p.off_v + hd * p.dv + i);
+    if (lane == 0) {
+      const float* ba = p.ba + row * p.ldba;
+      float* gb = p.gb + (static_cast<long long>(row) * p.H + hd) * 2;
+      gb[0] = decay_of(p, ba[p.off_a + hd], to_f(static_cast<const T*>(p.a_log)[hd]),
+                       to_f(static_cast<const T*>(p.dt_bias)[hd]));
+      gb[1] = sigmoid_f(ba[hd]);
+    }
+  }
+}
+
+constexpr int SCAN_TB = 16;      // tokens staged in shared memory at a time
+constexpr int SCAN_COLS = 16;    // columns per CTA (four warps, eight lanes per column)
+
+// NJ: groups of four state elements per lane (dk <= 32 NJ). Lane l of a column owns elements 32 j + 4 l .. + 3.
+template <typename T, int NJ>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const Params p) {
+  constexpr int DKP = 32 * NJ;
+  __shared__ __align__(16) float sq[SCAN_TB][DKP], sk[SCAN_TB][DKP];
+  __shared__ float sv[SCAN_TB][SCAN_COLS], sgb[SCAN_TB][2];
+  const int h = blockIdx.y, b = blockIdx.z, kvh = h / (p.H / p.G);
+  const int tid = threadIdx.x, l = tid & 7, cl = tid >> 3;
+  const int col = blockIdx.x * SCAN_COLS + cl;
+  const bool in = col < p.dv;
+  const long long pos0 = *p.pos;
+
+  // ---- the rows of the step's last tokens go into the convolution ring (nobody reads the ring in this launch)
+  {
+    const int C = 2 * p.G * p.dk + p.H * p.dv;
+    const int blocks = gridDim.x * gridDim.y;
+    const int me = blockIdx.y * gridDim.x + blockIdx.x;
+    const int keep = min(p.T, p.taps);
+    const T* proj_b = static_cast<const T*>(p.proj) + static_cast<long long>(b) * p.T * p.ldp;
+    float* ring_b = p.ring + static_cast<long long>(b) * p.taps * C;
+    for (int i = me * 128 + tid; i < keep * C; i += blocks * 128) {
+      const int t = p.T - keep + i / C, c = i % C, nq = p.G * p.dk;
+      const int src = c < nq ? p.off_q + c : (c < 2 * nq ? p.off_k + c - nq : p.off_v + c - 2 * nq);
+      ring_b[static_cast<long long>(ring_slot(pos0 + t, p.taps)) * C + c] = to_f(proj_b[t * p.ldp + src]);
+    }
+  }
+
+  float S[NJ][4];
+  float* st = p.state + ((static_cast<long long>(b) * p.H + h) * p.dv + (in ? col : 0)) * p.dk;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = 32 * j + 4 * l + e;
+      S[j][e] = (in && i < p.dk) ? st[i] : 0.f;
+    }
+  for (int t0 = 0; t0 < p.T; t0 += SCAN_TB) {
+    const int nt = min(SCAN_TB, p.T - t0);
+    __syncthreads();
+    for (int i = tid; i < SCAN_TB * DKP; i += 128) {
+      const int t = i / DKP, e = i % DKP;
+      const bool ok = t < nt && e < p.dk;
+      const long long src = ((static_cast<long long>(b) * p.T + t0 + t) * p.G + kvh) * p.dk + e;
+      sq[t][e] = ok ? p.q[src] : 0.f;
+      sk[t][e] = ok ? p.k[src] : 0.f;
+    }
+    for (int i = tid; i < SCAN_TB * SCAN_COLS; i += 128) {
+      const int t = i / SCAN_COLS, c = blockIdx.x * SCAN_COLS + i % SCAN_COLS;
+      sv[t][i % SCAN_COLS] =
+          (t < nt && c < p.dv) ? p.v[((static_cast<long long>(b) * p.T + t0 + t) * p.H + h) * p.dv + c] : 0.f;
+    }
+    if (tid < SCAN_TB * 2) {
+      const int t = tid >> 1;
+      sgb[t][tid & 1] = t < nt ? p.gb[((static_cast<long long>(b) * p.T + t0 + t) * p.H + h) * 2 + (tid & 1)] : 0.f;
+    }
+    __syncthreads();
+    for (int t = 0; t < nt; ++t) {
+      const float g = sgb[t][0], beta = sgb[t][1];
+      float4 kk[NJ];
+      float dk_[4] = {0.f, 0.f, 0.f, 0.f}, dq_[4] = {0.f, 0.f, 0.f, 0.f}, qk = 0.f;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        kk[j] = load4(&sk[t][32 * j + 4 * l]);
+        const float4 qq = load4(&sq[t][32 * j + 4 * l]);
+        dk_[0] = fmaf(S[j][0], kk[j].x, dk_[0]);
+        dk_[1] = fmaf(S[j][1], kk[j].y, dk_[1]);
+        dk_[2] = fmaf(S[j][2], kk[j].z, dk_[2]);
+        dk_[3] = fmaf(S[j][3], kk[j].w, dk_[3]);
+        dq_[0] = fmaf(S[j][0], qq.x, dq_[0]);
+        dq_[1] = fmaf(S[j][1], qq.y, dq_[1]);
+        dq_[2] = fmaf(S[j][2], qq.z, dq_[2]);
+        dq_[3] = fmaf(S[j][3], qq.w, dq_[3]);
+        qk = fmaf(kk[j].x, qq.x, fmaf(kk[j].y, qq.y, fmaf(kk[j].z, qq.z, fmaf(kk[j].w, qq.w, qk))));
+      }
+      float a = (dk_[0] + dk_[1]) + (dk_[2] + dk_[3]), c = (dq_[0] + dq_[1]) + (dq_[2] + dq_[3]);
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) {
+        a += __shfl_xor_sync(0xffffffffu, a, o);
+        c += __shfl_xor_sync(0xffffffffu, c, o);
+        qk += __shfl_xor_sync(0xffffffffu, qk, o);
+      }
+      const float u = beta * (sv[t][cl] - g * a);
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        S[j][0] = fmaf(kk[j].x, u, g * S[j][0]);
+        S[j][1] = fmaf(kk[j].y, u, g * S[j][1]);
+        S[j][2] = fmaf(kk[j].z, u, g * S[j][2]);
+        S[j][3] = fmaf(kk[j].w, u, g * S[j][3]);
+      }
+      if (l == 0 && in) p.o[((static_cast<long long>(b) * p.T + t0 + t) * p.H + h) * p.dv + col] = fmaf(qk, u, g * c);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < NJ; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = 32 * j + 4 * l + e;
+      if (in && i < p.dk) st[i] = S[j][e];
+    }
+}
+
+// one warp per (row, head): out = o / rms(o) * norm_w * silu(gate)
+template <typename T>
+__global__ void __launch_bounds__(128) delta_out_kernel(const Params p) {
+  const long long unit = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (unit >= static_cast<long long>(p.B) * p.T * p.H) return;
+  const long long row = unit / p.H;
+  const int h = static_cast<int>(unit - row * p.H);
+  const float* o = p.o + unit * p.dv;
+  float ss = 0.f;
+  for (int i = lane; i < p.dv; i += 32) ss += o[i] * o[i];
+  const float rs = 1.f / sqrtf(sum_warp(ss) / p.dv + p.eps);
+  const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.off_g + h * p.dv;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dv;
+  for (int i = lane; i < p.dv; i += 32)
+    from_f(out[i], o[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
+}
+
+// One token per sequence: grid (H, B). The convolution ring is only read at the rows of earlier tokens and only written
+// at the row of this one (taps rows apart), so the CTAs that share a q/k head need no order among themselves.
+constexpr int STEP_THREADS = 512;
+template <typename T, int NJ>
+__global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p) {
+  constexpr int DKP = 32 * NJ;
+  extern __shared__ float step_smem[];  // q[DKP], k[DKP], v[dv], o[dv]
+  __shared__ float red[32];
+  __shared__ float scal[4];             // 1 / |q| * scale, 1 / |k|
+  float *sq = step_smem, *sk = sq + DKP, *sv = sk + DKP, *so = sv + p.dv;
+  const int h = blockIdx.x, b = blockIdx.y, kvh = h / (p.H / p.G);
+  const int tid = threadIdx.x, l = tid & 7, lane = tid & 31, warp = tid >> 5;
+  const long long pos = *p.pos;
+  const int C = 2 * p.G * p.dk + p.H * p.dv;
+  const T* proj_b = static_cast<const T*>(p.proj) + static_cast<long long>(b) * p.ldp;
+  float* ring_b = p.ring + static_cast<long long>(b) * p.taps * C;
+  float* ring_now = ring_b + static_cast<long long>(ring_slot(pos, p.taps)) * C;
+  const bool first_of_group = h % (p.H / p.G) == 0;
+
+  float* st = p.state + (static_cast<long long>(b) * p.H + h) * p.dv * p.dk;
+  for (int i = tid; i < 2 * DKP + p.dv; i += STEP_THREADS) {
+    const int kind = i < DKP ? 0 : (i < 2 * DKP ? 1 : 2);
+    const int e = kind == 0 ? i : (kind == 1 ? i - DKP : i - 2 * DKP);
+    float x = 0.f;
+    if (kind == 2 || e < p.dk) {
+      const int nq = p.G * p.dk;
+      const int c = kind == 2 ? 2 * nq + h * p.dv + e : kind * nq + kvh * p.dk + e;
+      const int col = kind == 2 ? p.off_v + h * p.dv + e : (kind == 0 ? p.off_q : p.off_k) + kvh * p.dk + e;
+      const T* w = static_cast<const T*>(kind == 0 ? p.conv_q : (kind == 1 ? p.conv_k : p.conv_v)) +
+                   static_cast<long long>(kind == 2 ? h * p.dv + e : kvh * p.dk + e) * p.taps;
+      x = conv_silu(p, proj_b, ring_b, w, 0, pos, C, c, col);
+      if (kind == 2 || first_of_group) ring_now[c] = to_f(proj_b[col]);
+    }
+    step_smem[i] = x;
+  }
+  __syncthreads();
+  if (warp < 2) {
+    const float* s = warp == 0 ? sq : sk;
+    float ss = 0.f;
+    for (int i = lane; i < DKP; i += 32) ss += s[i] * s[i];
+    ss = sum_warp(ss);
+    if (lane == 0) scal[warp] = (warp == 0 ? p.q_scale : 1.f) / sqrtf(ss + 1e-6f);
+  } else if (tid == 64) {
+    const float* ba = p.ba + b * p.ldba;
+    scal[2] = decay_of(p, ba[p.off_a + h], to_f(static_cast<const T*>(p.a_log)[h]), to_f(static_cast<const T*>(p.dt_bias)[h]));
+    scal[3] = sigmoid_f(ba[h]);
+  }
+  __syncthreads();
+  const float qm = scal[0], km = scal[1], g = scal[2], beta = scal[3];
+  float4 kk[NJ], qq[NJ];
+  float qk = 0.f;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+    kk[j] = load4(sk + 32 * j + 4 * l);
+    qq[j] = load4(sq + 32 * j + 4 * l);
+    kk[j] = make_float4(kk[j].x * km, kk[j].y * km, kk[j].z * km, kk[j].w * km);
+    qq[j] = make_float4(qq[j].x * qm, qq[j].y * qm, qq[j].z * qm, qq[j].w * qm);
+    qk += kk[j].x * qq[j].x + kk[j].y * qq[j].y + kk[j].z * qq[j].z + kk[j].w * qq[j].w;
+  }
+#pragma unroll
+  for (int o = 4; o > 0; o >>= 1) qk += __shfl_xor_sync(0xffffffffu, qk, o);
+  const bool vec = (p.dk & 3) == 0;
+  float ss = 0.f;
+  // the trip count is the same for every thread: the shuffles below see whole warps
+  for (int c0 = 0; c0 < p.dv; c0 += STEP_THREADS / 8) {
+    const int col = c0 + (tid >> 3);
+    const bool in = col < p.dv;
+    float* sc = st + static_cast<long long>(in ? col : 0) * p.dk;
+    float4 S[NJ];
+    float a = 0.f, c = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int i = 32 * j + 4 * l;
+      if (vec) {
+        S[j] = (in && i < p.dk) ? load4(sc + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      } else {
+        S[j].x = (in && i < p.dk) ? sc[i] : 0.f;
+        S[j].y = (in && i + 1 < p.dk) ? sc[i + 1] : 0.f;
+        S[j].z = (in && i + 2 < p.dk) ? sc[i + 2] : 0.f;
+        S[j].w = (in && i + 3 < p.dk) ? sc[i + 3] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      a += S[j].x * kk[j].x + S[j].y * kk[j].y + S[j].z * kk[j].z + S[j].w * kk[j].w;
+      c += S[j].x * qq[j].x + S[j].y * qq[j].y + S[j].z * qq[j].z + S[j].w * qq[j].w;
+    }
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) {
+      a += __shfl_xor_sync(0xffffffffu, a, o);
+      c += __shfl_xor_sync(0xffffffffu, c, o);
+    }
+    const float u = beta * ((in ? sv[col] : 0.f) - g * a);
+    const float ov = fmaf(qk, u, g * c);
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int i = 32 * j + 4 * l;
+      const float4 n = make_float4(fmaf(kk[j].x, u, g * S[j].x), fmaf(kk[j].y, u, g * S[j].y),
+                                   fmaf(kk[j].z, u, g * S[j].z), fmaf(kk[j].w, u, g * S[j].w));
+      if (!in) continue;
+      if (vec) {
+        if (i < p.dk) store4(sc + i, n);
+      } else {
+        if (i < p.dk) sc[i] = n.x;
+        if (i + 1 < p.dk) sc[i + 1] = n.y;
+        if (i + 2 < p.dk) sc[i + 2] = n.z;
+        if (i + 3 < p.dk) sc[i + 3] = n.w;
+      }
+    }
+    if (in && l == 0) {
+      so[col] = ov;
+      ss += ov * ov;
+    }
+  }
+  const float rs = 1.f / sqrtf(sum_block(ss, red) / p.dv + p.eps);
+  const T* gate = proj_b + p.off_g + h * p.dv;
+  T* out = static_cast<T*>(p.out) + b * p.ldo + h * p.dv;
+  for (int i = tid; i < p.dv; i += STEP_THREADS)
+    from_f(out[i], so[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
+}
+
+template <typename T>
+int launch_prefill(const Params& p, cudaStream_t s) {
+  const int rows = p.B * p.T;
+  delta_prep_kernel<T><<<dim3(rows, (2 * p.G + p.H + 3) / 4), 128, 0, s>>>(p);
+  int rc = check_launch("delta_prep_kernel");
+  if (rc) return rc;
+  const dim3 grid((p.dv + SCAN_COLS - 1) / SCAN_COLS, p.H, p.B);
+  if (p.dk <= 32) delta_scan_kernel<T, 1><<<grid, 128, 0, s>>>(p);
+  else if (p.dk <= 64) delta_scan_kernel<T, 2><<<grid, 128, 0, s>>>(p);
+  else if (p.dk <= 96) delta_scan_kernel<T, 3><<<grid, 128, 0, s>>>(p);
+  else if (p.dk <= 128) delta_scan_kernel<T, 4><<<grid, 128, 0, s>>>(p);
+  else delta_scan_kernel<T, 8><<<grid, 128, 0, s>>>(p);
+  if ((rc = check_launch("delta_scan_kernel"))) return rc;
+  delta_out_kernel<T><<<(rows * p.H + 3) / 4, 128, 0, s>>>(p);
+  return check_launch("delta_out_kernel");
+}
+
+template <typename T>
+int launch_step(const Params& p, cudaStream_t s) {
+  const dim3 grid(p.H, p.B);
+#define RA_STEP(NJ) delta_step_kernel<T, NJ><<<grid, STEP_THREADS, (64 * NJ + 2 * p.dv) * sizeof(float), s>>>(p)
+  if (p.dk <= 32) RA_STEP(1);
+  else if (p.dk <= 64) RA_STEP(2);
+  else if (p.dk <= 96) RA_STEP(3);
+  else if (p.dk <= 128) RA_STEP(4);
+  else RA_STEP(8);
+#undef RA_STEP
+  return check_launch("delta_step_kernel");
+}
+
+}  // namespace delta
+}  // namespace ra
+
+// `step` 1: one token per sequence through the fused kernel (q, k, v, gb, o unused). `f32`: proj, out and the mixer's
+// vectors are fp32, else bf16.
+extern "C" int ra_delta_mixer(const ra::delta::Params* p, int step, int f32, void* stream) {
+  using namespace ra;
+  if (p->B < 1 || p->T < 1 || p->H < 1 || p->G < 1 || p->H % p->G || p->dk < 1 || p->dk > 256 || p->dv < 1 ||
+      p->dv > 4096 || p->taps < 1 || p->B > 65535 || p->H > 65535 || (step && p->T != 1)) {
+    set_error("ra_delta_mixer: bad shape (key dim at most 256, value dim at most 4096)");
+    return kHostBadArg;
+  }
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (step) return f32 ? delta::launch_step<float>(*p, s) : delta::launch_step<__nv_bfloat16>(*p, s);
+  return f32 ? delta::launch_prefill<float>(*p, s) : delta::launch_prefill<__nv_bfloat16>(*p, s);
+}

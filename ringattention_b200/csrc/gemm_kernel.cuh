@@ -34,6 +34,12 @@ struct Params {
   // TMA loads, tensor map 1), and the epilogue writes silu(gate) * up, F columns of bf16, instead of the
   // 2F pre-activations. gate and up are rounded to bf16 first, so the result equals the two-pass path.
   int swiglu_F;  // 0 = off
+  // Plain K-major products only: squared-relu activation, and a tail of columns [n_split, N) (n_split a multiple of
+  // 32) that leaves in fp32 to a second output whatever C's type is (small projections that feed 32-bit arithmetic).
+  int relu2;
+  float* C2;  // null = no tail
+  long long ldc2;
+  int n_split;
 };
 
 constexpr int MAX_SHARDS = 8;
@@ -354,7 +360,22 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
         tmem_ld_wait();
         const int col0 = n0 + c * 32;
         if (row < p.M && col0 < p.N) {
-          if (p.c_fp32) {
+          if (p.relu2) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) {
+              const float v = fmaxf(__uint_as_float(r[e]), 0.f);
+              r[e] = __float_as_uint(v * v);
+            }
+          }
+          if (p.C2 && col0 >= p.n_split) {
+            float* dst = p.C2 + static_cast<long long>(row) * p.ldc2 + (col0 - p.n_split);
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              if (col0 + j * 4 < p.N && RA_IN_BOUNDS(col0 - p.n_split + 4 * j, 4, p.ldc2, kTagGemmStore))
+                *reinterpret_cast<float4*>(dst + 4 * j) =
+                    make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]), __uint_as_float(r[4 * j + 2]),
+                                __uint_as_float(r[4 * j + 3]));
+          } else if (p.c_fp32) {
             float* dst = reinterpret_cast<float*>(p.C) + static_cast<long long>(row) * p.ldc + col0;
 #pragma unroll
             for (int j = 0; j < 8; ++j) {

@@ -1,0 +1,263 @@
+// Latent attention: per token one latent vector c (rank r) and one rotated key part shared by all heads are cached;
+// keys and values of the heads are linear images of c. Kernels that work on the cached rows directly, with the key
+// projection moved to the query and the value projection to the output ("absorbed" form), at any sizes:
+//   latent_prep_kernel   : RMS norm of c, rotary positions (interleaved pairs) on the shared key part and on the rotated part
+//                          of every query head, append of [c | rotated key] to the cache
+//   latent_absorb_kernel : q_lat[h] = [W_uk[h]^T q_unrotated | q_rotated], fp32
+//   latent_attend_kernel : split-KV attention of the q_lat rows over the cached rows, fp32 online softmax
+//   latent_merge_kernel  : merge of the splits, attention sink, value projection, per-head output gate
+// A cached row is [c, padded to a multiple of 8 | rotated key, padded to a multiple of 8] in the engine's storage type.
+// Everything between the stored operands and the stored output is fp32.
+#include "common/bounds.cuh"
+#include "common/host_util.h"
+#include "common/numeric.cuh"
+
+RA_BOUNDS_TRANSLATION_UNIT()
+
+namespace ra {
+namespace latent {
+
+struct Params {
+  int B, T, H, dn, dr, dv, r;  // T tokens per sequence in this step; row b * T + t
+  int r_pad, row_w;            // columns before the rotated key in a cached row, columns of a cached row
+  int rot_dims;                // leading dimensions of the rotated part that turn
+  void* proj;                  // (rows, ldp): q heads at off_q (dn + dr each), [c | k_rot] at off_c, gates at off_g
+  long long ldp;
+  int off_q, off_c, off_g;
+  const void* c_norm;          // (r)
+  const float* inv_freq;       // (rot_dims / 2)
+  void* cache;                 // (B, S_max, row_w)
+  long long S_max;
+  const void *w_uk, *w_uv;     // (H * dn, ldw), (H * dv, ldw)
+  long long ldw;
+  const float* sink;           // (H), or null
+  float* q_lat;                // (rows, H, row_w)
+  float *o_part, *lse_part;    // (rows, H, splits, r), (rows, H, splits)
+  int splits;
+  void* out;                   // (rows, ldo)
+  long long ldo;
+  float eps, scale;
+  const long long* pos;        // position of the step's first token
+};
+
+// grid (rows): the row's latent and keys go to the cache, its queries are rotated in place
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prep_kernel(const Params p) {
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  const int b = blockIdx.x / p.T, t = blockIdx.x - b * p.T;
+  const long long pos = *p.pos + t;
+  T* proj = static_cast<T*>(p.proj) + row * p.ldp;
+  const T* c = proj + p.off_c;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < p.r; i += 128) {
+    const float x = to_f(c[i]);
+    ss += x * x;
+  }
+  const float rs = 1.f / sqrtf(sum_block(ss, red) / p.r + p.eps);
+  const bool store = pos < p.S_max && RA_IN_BOUNDS(pos, 1, p.S_max, kTagDecodeCacheRow);
+  T* dst = static_cast<T*>(p.cache) + (b * p.S_max + (store ? pos : 0)) * p.row_w;
+  if (store) {
+    for (int i = threadIdx.x; i < p.r_pad; i += 128)
+      from_f(dst[i], i < p.r ? to_f(c[i]) * rs * to_f(static_cast<const T*>(p.c_norm)[i]) : 0.f);
+    for (int i = p.r_pad + p.dr + threadIdx.x; i < p.row_w; i += 128) from_f(dst[i], 0.f);
+  }
+  // unit 0: the shared key part (from the projection to the cache); unit 1 + h: query head h, in place
+  const int pairs = (p.dr + 1) / 2;
+  for (int i = threadIdx.x; i < (p.H + 1) * pairs; i += 128) {
+    const int unit = i / pairs, j = i - unit * pairs;
+    T* src = unit == 0 ? proj + p.off_c + p.r : proj + p.off_q + (unit - 1) * (p.dn + p.dr) + p.dn;
+    float u = to_f(src[2 * j]), v = 2 * j + 1 < p.dr ? to_f(src[2 * j + 1]) : 0.f;
+    if (2 * j + 1 < p.rot_dims) {
+      float sn, cs;
+      sincosf(static_cast<float>(pos) * p.inv_freq[j], &sn, &cs);
+      const float u2 = u * cs - v * sn;
+      v = v * cs + u * sn;
+      u = u2;
+    }
+    T* to = unit == 0 ? dst + p.r_pad : src;
+    if (unit == 0 && !store) continue;
+    from_f(to[2 * j], u);
+    if (2 * j + 1 < p.dr) from_f(to[2 * j + 1], v);
+  }
+}
+
+// grid (rows, H, ceil(row_w / 128)): one thread per latent column
+template <typename T>
+__global__ void __launch_bounds__(128) latent_absorb_kernel(const Params p) {
+  extern __shared__ float sq[];  // (dn)
+  const long long row = blockIdx.x;
+  const int h = blockIdx.y;
+  const T* q = static_cast<const T*>(p.proj) + row * p.ldp + p.off_q + h * (p.dn + p.dr);
+  for (int i = threadIdx.x; i < p.dn; i += 128) sq[i] = to_f(q[i]);
+  __syncthreads();
+  const int c = blockIdx.z * 128 + threadIdx.x;
+  if (c >= p.row_w) return;
+  float a = 0.f;
+  if (c < p.r) {
+    const T* w = static_cast<const T*>(p.w_uk) + static_cast<long long>(h) * p.dn * p.ldw + c;
+    for (int i = 0; i < p.dn; ++i) a = fmaf(sq[i], to_f(w[i * p.ldw]), a);
+  } else if (c >= p.r_pad && c < p.r_pad + p.dr) {
+    a = to_f(q[p.dn + c - p.r_pad]);
+  }
+  p.q_lat[(row * p.H + h) * p.row_w + c] = a;
+}
+
+constexpr int ATT_WARPS = 8;
+
+// grid (splits, H, rows): a warp per cached row at a time, lanes over its columns. NV: columns per lane (row_w <= 32 NV).
+template <typename T, int NV>
+__global__ void __launch_bounds__(ATT_WARPS * 32) latent_attend_kernel(const Params p) {
+  __shared__ float sm_m[ATT_WARPS], sm_l[ATT_WARPS];
+  extern __shared__ float sm_o[];  // [ATT_WARPS][r]
+  const int split = blockIdx.x, h = blockIdx.y;
+  const long long row = blockIdx.z;
+  const int b = blockIdx.z / p.T, t = blockIdx.z - b * p.T;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  long long n = *p.pos + t + 1;  // visible rows
+  if (n > p.S_max) n = p.S_max;
+  const long long per = (n + p.splits - 1) / p.splits;
+  const long long r0 = split * per, r1 = min(n, r0 + per);
+  const float* ql = p.q_lat + (row * p.H + h) * p.row_w;
+  float q[NV], acc[NV];
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int c = lane + 32 * j;
+    q[j] = c < p.row_w ? ql[c] * p.scale : 0.f;
+    acc[j] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  const T* base = static_cast<const T*>(p.cache) + b * p.S_max * p.row_w;
+  for (long long i = r0 + warp; i < r1; i += ATT_WARPS) {  // uniform over the warp
+    const T* kr = base + i * p.row_w;
+    float x[NV], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int c = lane + 32 * j;
+      x[j] = c < p.row_w ? to_f(kr[c]) : 0.f;
+      s = fmaf(q[j], x[j], s);
+    }
+    s = sum_warp(s);
+    const float mn = fmaxf(m, s), alpha = expf(m - mn), w = expf(s - mn);
+    l = l * alpha + w;
+    m = mn;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) acc[j] = fmaf(w, x[j], acc[j] * alpha);
+  }
+  if (lane == 0) {
+    sm_m[warp] = m;
+    sm_l[warp] = l;
+  }
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int c = lane + 32 * j;
+    if (c < p.r) sm_o[warp * p.r + c] = acc[j];
+  }
+  __syncthreads();
+  float mx = -INFINITY, lt = 0.f, f[ATT_WARPS];
+#pragma unroll
+  for (int w = 0; w < ATT_WARPS; ++w) mx = fmaxf(mx, sm_m[w]);
+#pragma unroll
+  for (int w = 0; w < ATT_WARPS; ++w) {
+    f[w] = sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - mx);
+    lt += sm_l[w] * f[w];
+  }
+  const long long pi = (row * p.H + h) * p.splits + split;
+  for (int c = threadIdx.x; c < p.r; c += ATT_WARPS * 32) {
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < ATT_WARPS; ++w) o += sm_o[w * p.r + c] * f[w];
+    p.o_part[pi * p.r + c] = lt > 0.f ? o / lt : 0.f;
+  }
+  if (threadIdx.x == 0) p.lse_part[pi] = lt > 0.f ? mx + logf(lt) : -INFINITY;
+}
+
+// grid (H, rows): latent output of the head from its splits, then the head's value projection
+template <typename T>
+__global__ void __launch_bounds__(256) latent_merge_kernel(const Params p) {
+  extern __shared__ float so[];  // (r)
+  const int h = blockIdx.x;
+  const long long row = blockIdx.y;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const float* lp = p.lse_part + (row * p.H + h) * p.splits;
+  const float* op = p.o_part + (row * p.H + h) * p.splits * p.r;
+  float mx = p.sink ? p.sink[h] : -INFINITY;
+  for (int s = 0; s < p.splits; ++s) mx = fmaxf(mx, lp[s]);
+  float den = p.sink ? expf(p.sink[h] - mx) : 0.f;
+  for (int s = 0; s < p.splits; ++s) den += expf(lp[s] - mx);
+  const T* proj = static_cast<const T*>(p.proj) + row * p.ldp;
+  const float mul = sigmoid_f(to_f(proj[p.off_g + h])) / den;
+  for (int c = threadIdx.x; c < p.r; c += 256) {
+    float o = 0.f;
+    for (int s = 0; s < p.splits; ++s) o = fmaf(expf(lp[s] - mx), op[s * p.r + c], o);
+    so[c] = o * mul;
+  }
+  __syncthreads();
+  T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dv;
+  for (int v = warp; v < p.dv; v += 8) {
+    const T* w = static_cast<const T*>(p.w_uv) + (static_cast<long long>(h) * p.dv + v) * p.ldw;
+    float a = 0.f;
+    for (int c = lane; c < p.r; c += 32) a = fmaf(so[c], to_f(w[c]), a);
+    a = sum_warp(a);
+    if (lane == 0) from_f(out[v], a);
+  }
+}
+
+template <typename T, int NV>
+int launch_attend(const Params& p, cudaStream_t s) {
+  const int smem = ATT_WARPS * p.r * static_cast<int>(sizeof(float));
+  if (smem > 48 * 1024 &&
+      cudaFuncSetAttribute(latent_attend_kernel<T, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+    set_error("ra_latent_attend: shared memory");
+    return kHostLaunchFail;
+  }
+  latent_attend_kernel<T, NV><<<dim3(p.splits, p.H, p.B * p.T), ATT_WARPS * 32, smem, s>>>(p);
+  return check_launch("latent_attend_kernel");
+}
+
+template <typename T>
+int run_absorbed(const Params& p, cudaStream_t s) {
+  const int rows = p.B * p.T;
+  latent_absorb_kernel<T><<<dim3(rows, p.H, (p.row_w + 127) / 128), 128, p.dn * sizeof(float), s>>>(p);
+  int rc = check_launch("latent_absorb_kernel");
+  if (rc) return rc;
+  if (p.row_w <= 128) rc = launch_attend<T, 4>(p, s);
+  else if (p.row_w <= 256) rc = launch_attend<T, 8>(p, s);
+  else if (p.row_w <= 640) rc = launch_attend<T, 20>(p, s);
+  else rc = launch_attend<T, 40>(p, s);
+  if (rc) return rc;
+  latent_merge_kernel<T><<<dim3(p.H, rows), 256, p.r * sizeof(float), s>>>(p);
+  return check_launch("latent_merge_kernel");
+}
+
+int check(const Params* p) {
+  if (p->B < 1 || p->T < 1 || p->H < 1 || p->H > 65535 || p->dn < 0 || p->dr < 0 || p->dv < 1 || p->r < 1 || p->row_w > 1280 ||
+      p->r_pad < p->r || p->row_w < p->r_pad + p->dr || p->rot_dims > p->dr || p->rot_dims % 2 || p->splits < 1 ||
+      static_cast<long long>(p->B) * p->T > 65535) {
+    set_error("ra_latent: bad shape (a cached row has at most 1280 columns, a call at most 65535 rows)");
+    return kHostBadArg;
+  }
+  return kHostOk;
+}
+
+}  // namespace latent
+}  // namespace ra
+
+extern "C" int ra_latent_prep(const ra::latent::Params* p, int f32, void* stream) {
+  using namespace ra;
+  int rc = latent::check(p);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (f32) latent::latent_prep_kernel<float><<<p->B * p->T, 128, 0, s>>>(*p);
+  else latent::latent_prep_kernel<__nv_bfloat16><<<p->B * p->T, 128, 0, s>>>(*p);
+  return check_launch("latent_prep_kernel");
+}
+
+// after ra_latent_prep: attention of the step's rows over the cache in the absorbed form
+extern "C" int ra_latent_absorbed(const ra::latent::Params* p, int f32, void* stream) {
+  using namespace ra;
+  int rc = latent::check(p);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return f32 ? latent::run_absorbed<float>(*p, s) : latent::run_absorbed<__nv_bfloat16>(*p, s);
+}

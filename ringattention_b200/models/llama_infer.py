@@ -21,8 +21,7 @@ of the chunk being prefilled are masked causally at their true positions.
 from __future__ import annotations
 
 import ctypes
-import time
-from typing import List, Optional
+from typing import Optional
 
 import torch
 import torch.distributed as dist
@@ -35,11 +34,13 @@ from ..ops import flash
 from ..ops import kernels as K
 from ..ops.flash import MaskSpec, Positions
 from ..parallel.mesh import AxisContext, resolve_axis
+from .cache import KVCache
+from .engine import InferenceEngine
 from .llama import _LayerFFNLinears
 from .params import FlatParams
 
 
-class LlamaInference:
+class LlamaInference(InferenceEngine):
     def __init__(self, cfg: LlamaConfig, max_context: int, batch: int = 1, device="cuda", seed: int = 0,
                  axis: "AxisContext | str | None" = None, params: Optional[FlatParams] = None,
                  symm_ring=None, streams: int = 0, max_new_tokens: int = 512):
@@ -48,11 +49,11 @@ class LlamaInference:
         K/V of its own decoded tokens in a small private tail (``max_new_tokens`` long, striped over the ranks).
         This is how a batch of long-context requests fits when distinct contexts do not: four 1M-token contexts
         of the 7B model would need 2 TiB of KV."""
+        super().__init__(batch, device, max(batch, int(streams)))
         self.cfg = cfg
         if streams and (batch != 1 or not 1 <= streams <= 8):
             raise ValueError("shared-prefix decoding takes batch = 1 and 1..8 streams")
         self.streams = int(streams)
-        self.device = torch.device(device)
         self.axis = resolve_axis(axis)
         self.rank, self.world = self.axis.rank, self.axis.size
         self.group = self.axis.group
@@ -62,7 +63,6 @@ class LlamaInference:
 
             self.symm_ring = SymmRing(self.group, self.device)
         self.params = params if params is not None else FlatParams(cfg, self.device, seed, with_optimizer=False)
-        self.B = batch
         self.H, self.D, self.d = cfg.n_heads, cfg.head_dim, cfg.d_model
         if max_context % (self.world * 128):
             raise ValueError("max_context must be a multiple of 128 * sp")
@@ -73,27 +73,15 @@ class LlamaInference:
         # only rows of the chunk being prefilled need their true positions (causal rule inside the chunk).
         self.n_rows = 0                             # local rows written by prefill
         self.prefill_len = 0                        # positions covered by prefill
-        # Heads-major storage (B, 2, H, S_max, D): the rows of one (k|v, head) are contiguous, so every CTA of the
-        # split-KV decode kernel streams one long run instead of 256-byte pieces 16 KB apart. The kernels see
-        # (B, S_max, H, D) views with strides; the flash kernel's tensor maps and the decode kernel take any strides.
-        self._cache = [torch.zeros(batch, 2, self.H, self.S_max, self.D, device=self.device, dtype=torch.bfloat16)
-                       for _ in range(cfg.n_layers)]
-        self.k_cache = [c[:, 0].permute(0, 2, 1, 3) for c in self._cache]   # (B, S_max, H, D) views
-        self.v_cache = [c[:, 1].permute(0, 2, 1, 3) for c in self._cache]
-        self.length = 0                             # tokens in the cache (global)
-        # [position, step] on the device: lets one recorded CUDA graph serve every decode step
-        self.state = torch.zeros(2, dtype=torch.int64, device=self.device)
-        self._graph = None
+        # (B, S_max, H, D) views of every layer's cache
+        self._kv = [KVCache(batch, self.H, self.S_max, self.D, self.device) for _ in range(cfg.n_layers)]
+        self.k_cache, self.v_cache = [c.k for c in self._kv], [c.v for c in self._kv]
         self._xchg = 0                              # prefill exchanges so far (parity picks the peer-memory buffer)
-        self._tok_buf = torch.zeros(max(batch, self.streams), dtype=torch.int32, device=self.device)
         if self.streams:
             t_tail = (max_new_tokens + self.world - 1) // self.world + 1
-            self._tail = [torch.zeros(self.streams, 2, self.H, t_tail, self.D, device=self.device, dtype=torch.bfloat16)
-                          for _ in range(cfg.n_layers)]
-            self.k_tail = [c[:, 0].permute(0, 2, 1, 3) for c in self._tail]  # (streams, T, H, D) views
-            self.v_tail = [c[:, 1].permute(0, 2, 1, 3) for c in self._tail]
+            self._tail = [KVCache(self.streams, self.H, t_tail, self.D, self.device) for _ in range(cfg.n_layers)]
+            self.k_tail, self.v_tail = [c.k for c in self._tail], [c.v for c in self._tail]  # (streams, T, H, D) views
             self._sp_work = [dict() for _ in range(cfg.n_layers)]
-        self._logits_buf = None
 
     # ------------------------------------------------------------------ helpers
     def _rows_to(self, src: torch.Tensor, dst_ptr: int, rows: int, row_bytes: int, src_ld: int, dst_ld: int) -> None:
@@ -230,69 +218,10 @@ class LlamaInference:
         K.decode_advance(self.state)
         return logits
 
-    @torch.no_grad()
-    def decode_step(self, tokens: torch.Tensor) -> torch.Tensor:
-        """One token per sequence: ``tokens (B,)`` -> logits ``(B, vocab)`` fp32 (same on all ranks)."""
-        self.state[0] = self.length
-        logits = self._decode_body(tokens.to(self.device, torch.int32).reshape(-1).contiguous())
-        self.length += 1
-        return logits
+    def _clear_cache(self) -> None:
+        self.n_rows = self.prefill_len = 0
 
-    @torch.no_grad()
-    def decode_step_graph(self) -> torch.Tensor:
-        """Greedy step on the token in ``self._tok_buf`` through a CUDA graph recorded on first use:
-        one replay per token instead of 7 launches per layer. Writes the next token back into
-        ``self._tok_buf`` and returns it. Call :meth:`decode_step` at least once before (buffers and
-        kernels must exist before capture)."""
-        if self._graph is None:
-            self.state[0] = self.length
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                logits = self._decode_body(self._tok_buf)
-                self._tok_buf.copy_(logits.argmax(dim=-1).to(torch.int32))
-            self._graph = g
-        self._graph.replay()
-        self.length += 1
-        return self._tok_buf
-
-    def reset(self) -> None:
-        """Forget the cached context (the cache memory is kept). The recorded decode graph is dropped
-        too: it holds the row count and length of the prefilled context as launch constants."""
-        self.length = self.n_rows = self.prefill_len = 0
-        self.state.zero_()
-        self._graph = None
-
-    @torch.no_grad()
-    def generate(self, prompt: torch.Tensor, new_tokens: int, chunk: int = 32768, use_graph: bool = True):
-        """Chunked prefill of ``prompt (B, T)`` followed by greedy decoding. Returns the generated
-        tokens ``(B, new_tokens)`` and timing: prefill seconds, per-token decode latencies."""
-        B, T = prompt.shape
-        if self.length:
-            self.reset()
-        torch.cuda.synchronize()
-        t0 = time.perf_counter()
-        logits = None
-        for c0 in range(0, T, chunk):
-            logits = self.prefill_chunk(prompt[:, c0:c0 + chunk])
-        torch.cuda.synchronize()
-        t_prefill = time.perf_counter() - t0
-        out: List[torch.Tensor] = []
-        lat: List[float] = []
-        nxt = logits.argmax(dim=-1)
+    def first_tokens(self, logits: torch.Tensor) -> torch.Tensor:
         if self.streams:  # the streams start from the `streams` most likely continuations of the shared prefix
-            nxt = logits[0].topk(self.streams).indices
-        for i in range(new_tokens):
-            out.append(nxt.clone())
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            if use_graph and i >= 2:
-                if i == 2:
-                    self._tok_buf.copy_(nxt.to(torch.int32))
-                nxt = self.decode_step_graph()
-            else:
-                nxt = self.decode_step(nxt).argmax(dim=-1)
-            e1.record()
-            torch.cuda.synchronize()
-            lat.append(e0.elapsed_time(e1))
-        return torch.stack([t.to(torch.int64) for t in out], dim=1), {"prefill_s": t_prefill, "decode_ms": lat}
+            return logits[0].topk(self.streams).indices
+        return self.sample(logits)

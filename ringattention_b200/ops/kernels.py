@@ -88,6 +88,33 @@ def linear_wgrad(dy, x, dw_acc):
     return gemm(dy, x, a_mn=True, b_mn=True, out=dw_acc, residual=dw_acc)
 
 
+def linear_ex(x, w, out, *, residual=None, tail=None, n_split: Optional[int] = None, relu2: bool = False):
+    """``out = act(x W^T (+ residual))`` with an inference layer's epilogues, in bf16 or true fp32 by the type of ``x``.
+
+    ``x (M, K)`` and ``w (N, K)`` share a type; ``out`` (a row-strided view) is of that type or fp32. ``residual`` has
+    ``out``'s type and may be ``out``. ``tail``: an fp32 view that takes the columns from ``n_split`` on."""
+    M, Kd = x.shape
+    N = w.shape[0]
+    assert w.shape[1] == Kd and x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1 and x.dtype == w.dtype
+    n_split = N if tail is None else int(n_split)
+    assert out.shape[0] == M and out.shape[1] >= n_split
+    if residual is not None:
+        assert residual.dtype == out.dtype and residual.stride(1) == 1 and not relu2
+    if tail is not None:
+        assert tail.dtype == torch.float32 and tail.stride(1) == 1 and tail.shape[1] >= N - n_split
+    ldr = residual.stride(0) if residual is not None else 0
+    ld2 = tail.stride(0) if tail is not None else 0
+    if x.dtype == torch.float32:
+        assert out.dtype == torch.float32
+        _lib.call("ra_linear_f32", ptr(x), ptr(w), ptr(out), ptr(residual), ptr(tail), M, N, Kd, c_ll(x.stride(0)),
+                  c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2), stream_ptr())
+        return out
+    _lib.call("ra_gemm_bf16_ex", ptr(x), ptr(w), ptr(out), ptr(residual), ptr(tail), M, N, Kd, c_ll(x.stride(0)),
+              c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2),
+              int(out.dtype == torch.float32), 8, _status(), stream_ptr())
+    return out
+
+
 # ---------------------------------------------------------------------------------------------
 # normalisation / rope / activation
 # ---------------------------------------------------------------------------------------------
@@ -141,6 +168,31 @@ def swiglu_bwd_(gu, dh):
     assert gu.is_contiguous() and dh.is_contiguous()
     _lib.call("ra_swiglu_bwd", ptr(gu), ptr(dh), ptr(gu), c_ll(rows), f2 // 2, stream_ptr())
     return gu
+
+
+# ---------------------------------------------------------------------------------------------
+# 32-bit residual stream
+# ---------------------------------------------------------------------------------------------
+def embed_f32(tokens, table, d: int, out):
+    """``out (rows, ld)`` fp32 <- the tokens' rows of ``table`` (bf16 or fp32); columns past ``d`` are zeroed."""
+    assert tokens.dtype == torch.int32 and tokens.is_contiguous() and out.dtype == torch.float32 and out.is_contiguous()
+    _lib.call("ra_embed_f32", ptr(tokens), ptr(table), c_ll(table.stride(0)), ptr(out), c_ll(out.stride(0)),
+              tokens.numel(), d, table.shape[0], int(table.dtype == torch.float32), stream_ptr())
+    return out
+
+
+def norm_f32(x, d: int, eps: float, gain_offset: float, w1, w2=None, rows_idx=None):
+    """RMS norm of the fp32 rows of ``x (rows, ld)`` over the first ``d`` columns with gains ``gain_offset + w``; a second
+    gain gives a second output of the same rows. Outputs have the gains' type; ``rows_idx`` picks rows."""
+    rows = x.shape[0] if rows_idx is None else rows_idx.numel()
+    ld = x.stride(0)
+    y1 = torch.empty(rows, ld, device=x.device, dtype=w1.dtype)
+    y2 = torch.empty_like(y1) if w2 is not None else None
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and w1.numel() == ld and (w2 is None or w2.numel() == ld)
+    assert rows_idx is None or rows_idx.dtype == torch.int32
+    _lib.call("ra_norm_f32", ptr(x), ptr(rows_idx), ptr(w1), ptr(w2), ptr(y1), ptr(y2), rows, d, ld, c_ll(ld), c_ll(ld),
+              c_f(eps), c_f(gain_offset), int(w1.dtype == torch.float32), stream_ptr())
+    return y1, y2
 
 
 # ---------------------------------------------------------------------------------------------
