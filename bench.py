@@ -58,6 +58,12 @@ def parse_args():
                     help="also report device milliseconds per phase of a step (measured in the end-to-end steps)")
     ap.add_argument("--time-budget", type=float, default=600.0,
                     help="wall-clock seconds for the whole run, counted from process start (0 = no limit)")
+    ap.add_argument("--serve", action="store_true",
+                    help="instead of the headline workload: prefill and decode throughput of the inference engines, hybrid "
+                         "decoders beside LLaMA at equal size (1 GPU)")
+    from ringattention_b200.utils import servebench
+
+    servebench.add_arguments(ap)
     return ap.parse_args()
 
 
@@ -164,6 +170,10 @@ def main() -> int:
     args = parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.serve:
+        from ringattention_b200.utils import servebench
+
+        return servebench.main(args)
 
     import torch
     import torch.distributed as dist

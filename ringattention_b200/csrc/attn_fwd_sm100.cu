@@ -45,29 +45,43 @@ struct FwdParams {
   long long copy_n16;
   int copy_ctas;
   int* status;
+  // Two-part keys (NR > 0): width of the values that is stored (the tile's columns past it are zero), per-head attention
+  // sink (one more entry exp(sink) in the denominator, without a value), per-head output gate sigmoid(gate[row, h])
+  int dv;
+  const float* sink;            // (H), or null
+  const __nv_bfloat16* gate;    // (B * Sq, gate_ld), or null
+  long long gate_ld;
 };
 
-template <int D>
+// NS: 64-wide slabs of the query/key width, DV: value width of the tile. The second K stage is given up where it does not
+// fit beside two tiles of wide queries; V keeps two.
+template <int NS, int DV>
 struct FwdSmem {
-  static constexpr int Q_TILE_BYTES = 128 * D * 2;
-  static constexpr int KV_TILE_BYTES = 128 * D * 2;
   static constexpr int SLAB_BYTES = 128 * 64 * 2;  // one 64-wide d slab of a 128-row tile
+  static constexpr int Q_TILE_BYTES = NS * SLAB_BYTES;
+  static constexpr int K_TILE_BYTES = NS * SLAB_BYTES;
+  static constexpr int V_TILE_BYTES = 128 * DV * 2;
+  static constexpr int K_STAGES = (2 + KV_STAGES) * Q_TILE_BYTES + KV_STAGES * V_TILE_BYTES <= 200 * 1024 ? KV_STAGES : 1;
   static constexpr int Q_OFF = 0;
   static constexpr int K_OFF = Q_OFF + 2 * Q_TILE_BYTES;
-  static constexpr int V_OFF = K_OFF + KV_STAGES * KV_TILE_BYTES;
-  static constexpr int AUX_OFF = V_OFF + KV_STAGES * KV_TILE_BYTES;  // seg/bias staging
+  static constexpr int V_OFF = K_OFF + K_STAGES * K_TILE_BYTES;
+  static constexpr int AUX_OFF = V_OFF + KV_STAGES * V_TILE_BYTES;  // seg/bias staging
   static constexpr int AUX_BYTES = 2 /*wg*/ * 2 /*buf*/ * 128 * 4 * 2 /*seg+bias*/;
   static constexpr int BAR_OFF = AUX_OFF + AUX_BYTES;
   static constexpr int VIS_OFF = BAR_OFF + 256;  // [2 q tiles][VIS_WORDS] visibility of the kv tiles
   static constexpr int TOTAL = VIS_OFF + 2 * VIS_WORDS * 4 + 1024;
 };
 
-template <int D>
+// NQ: slabs of the query/key part that every head has of its own; NR: slabs of a second part (maps tma_q2, tma_k2) whose
+// keys all heads share; DV: value width. NR = 0 is plain attention with head dim 64 NQ = DV.
+template <int NQ, int NR, int DV>
 __global__ void __launch_bounds__(FWD_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
-                const __grid_constant__ CUtensorMap tma_v, const FwdParams p) {
-  using SM = FwdSmem<D>;
-  constexpr int NSLAB = D / 64;
+                const __grid_constant__ CUtensorMap tma_v, const __grid_constant__ CUtensorMap tma_q2,
+                const __grid_constant__ CUtensorMap tma_k2, const FwdParams p) {
+  constexpr int NSLAB = NQ + NR, VSLAB = DV / 64;
+  using SM = FwdSmem<NSLAB, DV>;
+  constexpr int K_STAGES = SM::K_STAGES;
 
   // A failure recorded earlier on this stream (for example a ring barrier that timed out) turns
   // every later attention kernel into a no-op, so nothing touches the memory of a lost peer.
@@ -144,6 +158,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
     tma_prefetch_desc(&tma_q);
     tma_prefetch_desc(&tma_k);
     tma_prefetch_desc(&tma_v);
+    if (NR) {
+      tma_prefetch_desc(&tma_q2);
+      tma_prefetch_desc(&tma_k2);
+    }
   }
   if (warp == 1) {
     tmem_alloc(tmem_slot, 512);
@@ -181,25 +199,27 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
       for (int w = 0; w < 2; ++w)
 #pragma unroll
         for (int s = 0; s < NSLAB; ++s)
-          tma_load_4d(sQ + w * SM::Q_TILE_BYTES + s * SM::SLAB_BYTES, &tma_q, q_full, s * 64, h,
-                      q0 + w * 128, b);
+          tma_load_4d(sQ + w * SM::Q_TILE_BYTES + s * SM::SLAB_BYTES, s < NQ ? &tma_q : &tma_q2, q_full,
+                      (s < NQ ? s : s - NQ) * 64, h, q0 + w * 128, b);
       int it = 0;
       for (int j = min(next_vis(0, 0), next_vis(1, 0)); j < nk;
            j = min(next_vis(0, j + 1), next_vis(1, j + 1))) {
         const int k0 = j * 128;
         const int st = it & 1;
         const uint32_t ph = (it >> 1) & 1;
-        if (!mbar_wait_relaxed(&k_empty[st], ph ^ 1u, wc, kTimeoutSmemEmpty)) break;
-        mbar_arrive_expect_tx(&k_full[st], SM::KV_TILE_BYTES);
+        const int kst = it % K_STAGES;
+        const uint32_t kph = (it / K_STAGES) & 1;
+        if (!mbar_wait_relaxed(&k_empty[kst], kph ^ 1u, wc, kTimeoutSmemEmpty)) break;
+        mbar_arrive_expect_tx(&k_full[kst], SM::K_TILE_BYTES);
 #pragma unroll
         for (int s = 0; s < NSLAB; ++s)
-          tma_load_4d(sK + st * SM::KV_TILE_BYTES + s * SM::SLAB_BYTES, &tma_k, &k_full[st], s * 64,
-                      h, k0, b);
+          tma_load_4d(sK + kst * SM::K_TILE_BYTES + s * SM::SLAB_BYTES, s < NQ ? &tma_k : &tma_k2, &k_full[kst],
+                      (s < NQ ? s : s - NQ) * 64, s < NQ ? h : 0, k0, b);
         if (!mbar_wait_relaxed(&v_empty[st], ph ^ 1u, wc, kTimeoutSmemEmpty)) break;
-        mbar_arrive_expect_tx(&v_full[st], SM::KV_TILE_BYTES);
+        mbar_arrive_expect_tx(&v_full[st], SM::V_TILE_BYTES);
 #pragma unroll
-        for (int s = 0; s < NSLAB; ++s)
-          tma_load_4d(sV + st * SM::KV_TILE_BYTES + s * SM::SLAB_BYTES, &tma_v, &v_full[st], s * 64,
+        for (int s = 0; s < VSLAB; ++s)
+          tma_load_4d(sV + st * SM::V_TILE_BYTES + s * SM::SLAB_BYTES, &tma_v, &v_full[st], s * 64,
                       h, k0, b);
         ++it;
       }
@@ -210,16 +230,16 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
     {
       const bool leader = elect_one();
       constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, 0, 0);
-      constexpr uint32_t idesc_o = make_idesc_bf16(128, D, 0, 1);
+      constexpr uint32_t idesc_o = make_idesc_bf16(128, DV, 0, 1);
       const uint64_t q_desc[2] = {make_smem_desc(smem_u32(sQ), 16, 1024),
                                   make_smem_desc(smem_u32(sQ + SM::Q_TILE_BYTES), 16, 1024)};
       const uint64_t k_desc[2] = {make_smem_desc(smem_u32(sK), 16, 1024),
-                                  make_smem_desc(smem_u32(sK + SM::KV_TILE_BYTES), 16, 1024)};
+                                  make_smem_desc(smem_u32(sK + (K_STAGES - 1) * SM::K_TILE_BYTES), 16, 1024)};
       const uint64_t v_desc[2] = {make_smem_desc(smem_u32(sV), SM::SLAB_BYTES, 1024),
-                                  make_smem_desc(smem_u32(sV + SM::KV_TILE_BYTES), SM::SLAB_BYTES, 1024)};
+                                  make_smem_desc(smem_u32(sV + SM::V_TILE_BYTES), SM::SLAB_BYTES, 1024)};
       auto issue_s = [&](int w, int st) {
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < NSLAB * 4; ++kk) {
           const uint32_t off = (kk >> 2) * SM::SLAB_BYTES + (kk & 3) * 32;
           if (leader)
             umma_ss(tS[w], desc_advance(q_desc[w], off), desc_advance(k_desc[st], off), idesc_s,
@@ -263,8 +283,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
         const int jn = next_visible(j + 1, n0, n1);
         const int st = it & 1;
         const uint32_t ph = (it >> 1) & 1;
-        const int stn = (it + 1) & 1;
-        const uint32_t phn = ((it + 1) >> 1) & 1;
+        const int stn = (it + 1) % K_STAGES;  // K stage of the next tile
+        const uint32_t phn = ((it + 1) / K_STAGES) & 1;
         if (!mbar_wait(&v_full[st], ph, wc, kTimeoutSmemFull)) break;
         bool k_ready = false;
         if (v0) {
@@ -438,7 +458,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
           tc_fence_after();
           const float alpha = (m_new == -INFINITY) ? 1.0f : exp2_approx(m_ref - m_new);
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t o[32];
             tmem_ld_x32(tO[w] + lane_base + c * 32, o);
             tmem_ld_wait();
@@ -501,14 +521,20 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
         lse = mxl + __logf(tot);
       }
     }
-    if (row_valid && RA_IN_BOUNDS(lse_idx, 1, static_cast<long long>(p.B) * p.H * mk.Sq, kTagAttnFwdLse))
+    if ((!NR || p.lse_out) && row_valid &&
+        RA_IN_BOUNDS(lse_idx, 1, static_cast<long long>(p.B) * p.H * mk.Sq, kTagAttnFwdLse))
       p.lse_out[lse_idx] = lse;
-    const float mul = inv_l * w_this;
+    float mul = inv_l * w_this;
+    if (NR && row_valid) {
+      if (p.sink) mul /= 1.f + expf(p.sink[h] - lse);
+      if (p.gate)
+        mul /= 1.f + expf(-__bfloat162float(p.gate[(static_cast<long long>(b) * mk.Sq + qi) * p.gate_ld + h]));
+    }
     const float* oprev_row =
-        p.o_prev ? p.o_prev + ((static_cast<long long>(b) * mk.Sq + qi) * p.H + h) * D : nullptr;
+        p.o_prev ? p.o_prev + ((static_cast<long long>(b) * mk.Sq + qi) * p.H + h) * DV : nullptr;
     const long long o_off = b * p.o_stride_b + static_cast<long long>(qi) * p.o_stride_s + h * p.o_stride_h;
 #pragma unroll 1
-    for (int c = 0; c < D / 32; ++c) {
+    for (int c = 0; c < DV / 32; ++c) {
       uint32_t o[32];
       if (cnt > 0) {
         tmem_ld_x32(tO[w] + lane_base + c * 32, o);
@@ -517,7 +543,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
 #pragma unroll
         for (int i = 0; i < 32; ++i) o[i] = 0u;
       }
-      if (row_valid && RA_IN_BOUNDS(qi, 1, mk.Sq, kTagAttnFwdOut) && RA_IN_BOUNDS(c * 32, 32, D, kTagAttnFwdOut)) {
+      if (row_valid && RA_IN_BOUNDS(qi, 1, mk.Sq, kTagAttnFwdOut) && RA_IN_BOUNDS(c * 32, 32, DV, kTagAttnFwdOut)) {
         float f[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(o[i]) * mul;
@@ -541,6 +567,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + o_off + c * 32;
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
+            if (NR && c * 32 + i * 8 >= p.dv) continue;
             uint4 v;
             v.x = pack_bf16x2(f[8 * i], f[8 * i + 1]);
             v.y = pack_bf16x2(f[8 * i + 2], f[8 * i + 3]);
@@ -576,6 +603,21 @@ int make_bshd_map(CUtensorMap* m, const void* base, int B, int S, int H, int D, 
                      static_cast<uint64_t>(sb) * 2};
   uint32_t box[4] = {64, 1, 128, 1};
   return ra::make_tmap_bf16_sw128(m, base, 4, dims, str, box);
+}
+
+template <int NQ, int NR, int DV>
+int launch_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq2,
+               const CUtensorMap& tk2, const ra::attn::FwdParams& p, long long grid, cudaStream_t s) {
+  using namespace ra::attn;
+  auto kern = attn_fwd_kernel<NQ, NR, DV>;
+  constexpr int smem = FwdSmem<NQ + NR, DV>::TOTAL;
+  static_assert(smem <= 227 * 1024, "tile buffers do not fit in shared memory");
+  if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+    ra::set_error("attn_fwd: smem attribute");
+    return ra::kHostLaunchFail;
+  }
+  kern<<<static_cast<unsigned>(grid), FWD_THREADS, smem, s>>>(tq, tk, tv, tq2, tk2, p);
+  return ra::check_launch("attn_fwd_kernel");
 }
 }  // namespace
 
@@ -658,20 +700,78 @@ extern "C" int ra_attn_fwd(const RaAttnFwdArgs* a) {
   p.copy_n16 = a->copy_bytes / 16;
   p.copy_ctas = (a->copy_src && a->copy_bytes > 0) ? a->copy_ctas : 0;
   p.status = a->status;
-  const int n_qpairs = (a->Sq + 255) / 256;
-  const long long grid = static_cast<long long>(n_qpairs) * a->H * a->B + p.copy_ctas;
+  p.dv = a->D;
+  p.sink = nullptr;
+  p.gate = nullptr;
+  p.gate_ld = 0;
+  const long long grid = static_cast<long long>((a->Sq + 255) / 256) * a->H * a->B + p.copy_ctas;
   cudaStream_t s = static_cast<cudaStream_t>(a->stream);
-  cudaError_t e;
-  if (a->D == 128) {
-    auto kern = attn_fwd_kernel<128>;
-    e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, FwdSmem<128>::TOTAL);
-    if (e != cudaSuccess) { set_error("attn_fwd: smem attribute"); return kHostLaunchFail; }
-    kern<<<static_cast<unsigned>(grid), FWD_THREADS, FwdSmem<128>::TOTAL, s>>>(tq, tk, tv, p);
-  } else {
-    auto kern = attn_fwd_kernel<64>;
-    e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, FwdSmem<64>::TOTAL);
-    if (e != cudaSuccess) { set_error("attn_fwd: smem attribute"); return kHostLaunchFail; }
-    kern<<<static_cast<unsigned>(grid), FWD_THREADS, FwdSmem<64>::TOTAL, s>>>(tq, tk, tv, p);
+  return a->D == 128 ? launch_fwd<2, 0, 128>(tq, tk, tv, tq, tk, p, grid, s)
+                     : launch_fwd<1, 0, 64>(tq, tk, tv, tq, tk, p, grid, s);
+}
+
+// Causal attention with two-part queries and keys: score = (q1 . k1 + q2 . k2) * scale, where k2 is shared by all heads.
+// q (B, Sq, H, d1 + d2) with q1 first, k1 (B, Sk, H, d1), k2 (B, Sk, d2), v (B, Sk, H, dv), out (B, Sq, H, dv); bf16, element
+// strides, innermost contiguous; query i sits at position q_pos0 + i, key j at j. d1 <= 128, d2 <= 64, dv <= 128, all
+// multiples of 8. `sink` (H) fp32 and `gate` (B * Sq, gate_ld) bf16 are optional (see FwdParams).
+struct RaAttnTwoPartArgs {
+  const void* q; long long q_sb, q_ss, q_sh;
+  const void* k1; long long k1_sb, k1_ss, k1_sh;
+  const void* k2; long long k2_sb, k2_ss;
+  const void* v; long long v_sb, v_ss, v_sh;
+  void* out; long long o_sb, o_ss, o_sh;
+  const float* sink;
+  const void* gate; long long gate_ld;
+  int B, H, Sq, Sk, d1, d2, dv;
+  float scale;
+  int q_pos0;
+  int* status;
+  void* stream;
+};
+
+extern "C" int ra_attn_two_part(const RaAttnTwoPartArgs* a) {
+  using namespace ra;
+  using namespace ra::attn;
+  const long long odd = (a->q_sb | a->q_ss | a->q_sh | a->k1_sb | a->k1_ss | a->k1_sh | a->k2_sb | a->k2_ss | a->v_sb |
+                         a->v_ss | a->v_sh | a->o_sb | a->o_ss | a->o_sh) & 7;
+  if (a->B < 1 || a->H < 1 || a->Sq < 1 || a->Sk < 1 || a->q_pos0 < 0 || a->d1 < 8 || a->d1 > 128 || a->d1 % 8 ||
+      a->d2 < 8 || a->d2 > 64 || a->d2 % 8 || a->dv < 8 || a->dv > 128 || a->dv % 8 || odd ||
+      ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k1) | reinterpret_cast<uintptr_t>(a->k2) |
+        reinterpret_cast<uintptr_t>(a->v) | reinterpret_cast<uintptr_t>(a->out)) & 15)) {
+    set_error("ra_attn_two_part: bad shape or alignment");
+    return kHostBadArg;
   }
-  return check_launch("attn_fwd_kernel");
+  CUtensorMap tq, tk, tv, tq2, tk2;
+  int rc;
+  const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a->q);
+  if ((rc = make_bshd_map(&tq, q, a->B, a->Sq, a->H, a->d1, a->q_sb, a->q_ss, a->q_sh))) return rc;
+  if ((rc = make_bshd_map(&tq2, q + a->d1, a->B, a->Sq, a->H, a->d2, a->q_sb, a->q_ss, a->q_sh))) return rc;
+  if ((rc = make_bshd_map(&tk, a->k1, a->B, a->Sk, a->H, a->d1, a->k1_sb, a->k1_ss, a->k1_sh))) return rc;
+  if ((rc = make_bshd_map(&tk2, a->k2, a->B, a->Sk, 1, a->d2, a->k2_sb, a->k2_ss, a->k2_ss))) return rc;
+  if ((rc = make_bshd_map(&tv, a->v, a->B, a->Sk, a->H, a->dv, a->v_sb, a->v_ss, a->v_sh))) return rc;
+  FwdParams p = {};
+  p.B = a->B;
+  p.H = a->H;
+  p.mask.Sq = a->Sq;
+  p.mask.Sk = a->Sk;
+  p.mask.cbs = 1;
+  p.mask.qmap = PosMap{a->q_pos0, 0, 1 << 30};
+  p.mask.kmap = PosMap{0, 0, 1 << 30};
+  p.scale_log2 = a->scale * kLog2e;
+  p.out = a->out;
+  p.o_stride_b = a->o_sb;
+  p.o_stride_s = a->o_ss;
+  p.o_stride_h = a->o_sh;
+  p.status = a->status;
+  p.dv = a->dv;
+  p.sink = a->sink;
+  p.gate = static_cast<const __nv_bfloat16*>(a->gate);
+  p.gate_ld = a->gate_ld;
+  const long long grid = static_cast<long long>((a->Sq + 255) / 256) * a->H * a->B;
+  cudaStream_t s = static_cast<cudaStream_t>(a->stream);
+  if (a->d1 > 64)
+    return a->dv > 64 ? launch_fwd<2, 1, 128>(tq, tk, tv, tq2, tk2, p, grid, s)
+                      : launch_fwd<2, 1, 64>(tq, tk, tv, tq2, tk2, p, grid, s);
+  return a->dv > 64 ? launch_fwd<1, 1, 128>(tq, tk, tv, tq2, tk2, p, grid, s)
+                    : launch_fwd<1, 1, 64>(tq, tk, tv, tq2, tk2, p, grid, s);
 }

@@ -932,17 +932,35 @@ constexpr int LM_WTILE = LM_COLS * LM_KC * 2;     // bytes of a weight chunk
 constexpr int LM_XTILE = 8 * LM_KC * 2;           // bytes of an x chunk (eight rows)
 constexpr int LM_STAGE = LM_WTILE + LM_XTILE;
 
-__global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const __nv_bfloat16* __restrict__ x,
-                                                                        const __nv_bfloat16* __restrict__ w,
-                                                                        __nv_bfloat16* __restrict__ y,
-                                                                        const __nv_bfloat16* __restrict__ res, int M,
-                                                                        int N, int K) {
+// Columns of the product fall into up to three segments with outputs of their own (an inference layer's projections in
+// one launch): [0, n32_from) bf16 to y, [n32_from, act_from) fp32 to y32 (added to what is there when `add32`: the 32-bit
+// residual stream), [act_from, N) squared relu in bf16 to ya; the last segment multiplies x2 instead of x (the same rows
+// through another norm). Segment borders are multiples of LM_COLS.
+struct LmParams {
+  const __nv_bfloat16 *x, *x2;
+  long long ldx;
+  const __nv_bfloat16* w;      // (N, K)
+  __nv_bfloat16* y;
+  long long ldy;
+  const __nv_bfloat16* res;    // addend of the first segment (leading dimension ldy), or null
+  float* y32;
+  long long ldy32;
+  __nv_bfloat16* ya;
+  long long ldya;
+  int n32_from, act_from, add32;
+  int M, N, K;
+};
+
+__global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const LmParams p) {
   extern __shared__ uint4 lm_ring[];  // [LM_WARPS][LM_ST][weights | x]
   __shared__ float red[LM_WARPS][8][LM_COLS];
+  const int M = p.M, N = p.N, K = p.K;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   uint8_t* ring = reinterpret_cast<uint8_t*>(lm_ring) + warp * (LM_ST * LM_STAGE);
   const int col0 = blockIdx.x * LM_COLS;
+  const __nv_bfloat16* w = p.w;
+  const __nv_bfloat16* x = col0 >= p.act_from ? p.x2 : p.x;
   const int n_kc = (K + LM_KC - 1) / LM_KC;  // chunks of K; warp w takes chunks w, w + 4, ... (the CTA reads 1 KB of a row at a time)
   const int my_kc = warp < n_kc ? (n_kc - warp + LM_WARPS - 1) / LM_WARPS : 0;
 
@@ -963,7 +981,7 @@ __global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const __
       const int piece = lane + 32 * j;
       const int row = piece >> 4, ch = piece & 15;
       const bool in = row < M && k0 + ch * 8 < K;
-      const __nv_bfloat16* src = x + static_cast<long long>(in ? row : 0) * K + (in ? k0 + ch * 8 : 0);
+      const __nv_bfloat16* src = x + (in ? row : 0) * p.ldx + (in ? k0 + ch * 8 : 0);
       cp_async16(wt + LM_WTILE + row * (LM_KC * 2) + ((ch ^ (row & 7)) << 4), src, in ? 16 : 0);
     }
   };
@@ -1022,9 +1040,19 @@ __global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const __
     float v = 0.f;
 #pragma unroll
     for (int k = 0; k < LM_WARPS; ++k) v += red[k][m][c];
-    const long long o = static_cast<long long>(m) * N + col0 + c;
-    if (res) v += __bfloat162float(res[o]);
-    if (RA_IN_BOUNDS(col0 + c, 1, N, kTagSmallMLinear)) y[o] = __float2bfloat16(v);
+    const int col = col0 + c;
+    if (!RA_IN_BOUNDS(col, 1, N, kTagSmallMLinear)) continue;
+    if (col0 >= p.act_from) {
+      v = fmaxf(v, 0.f);
+      p.ya[m * p.ldya + col - p.act_from] = __float2bfloat16(v * v);
+    } else if (col0 >= p.n32_from) {
+      float* dst = p.y32 + m * p.ldy32 + col - p.n32_from;
+      *dst = p.add32 ? *dst + v : v;
+    } else {
+      const long long o = m * p.ldy + col;
+      if (p.res) v += __bfloat162float(p.res[o]);
+      p.y[o] = __float2bfloat16(v);
+    }
   }
 }
 
@@ -1341,14 +1369,9 @@ extern "C" int ra_small_m_linear_fused(const void* x, const void* w, void* y, co
   return check_launch("small_m_linear_pro_kernel");
 }
 
-// y = x W^T (+ res) for 1 <= M <= 8 rows on the tensor cores (x as it is: no prologue on this path).
-extern "C" int ra_small_m_linear_mma(const void* x, const void* w, void* y, const void* res, int M, int N, int K,
-                                     void* stream) {
+namespace {
+int launch_small_m_mma(const ra::decode::LmParams& p, cudaStream_t s) {
   using namespace ra::decode;
-  if (M < 1 || M > 8 || K % 8 || N < 1) {
-    set_error("ra_small_m_linear_mma: need 1 <= M <= 8 and K % 8 == 0");
-    return kHostBadArg;
-  }
   constexpr int smem = LM_WARPS * LM_ST * LM_STAGE;  // 72 KB
   static bool attr_done[64] = {};
   int dev = 0;
@@ -1357,16 +1380,61 @@ extern "C" int ra_small_m_linear_mma(const void* x, const void* w, void* y, cons
     if (cudaFuncSetAttribute(small_m_linear_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
         cudaSuccess) {
       cudaGetLastError();
-      set_error("ra_small_m_linear_mma: cannot raise the shared-memory limit");
+      set_error("small_m_linear_mma: cannot raise the shared-memory limit");
       return kHostLaunchFail;
     }
     attr_done[dev] = true;
   }
-  const int blocks = (N + LM_COLS - 1) / LM_COLS;
-  small_m_linear_mma_kernel<<<blocks, LM_THREADS, smem, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const __nv_bfloat16*>(x), static_cast<const __nv_bfloat16*>(w), static_cast<__nv_bfloat16*>(y),
-      static_cast<const __nv_bfloat16*>(res), M, N, K);
+  small_m_linear_mma_kernel<<<(p.N + LM_COLS - 1) / LM_COLS, LM_THREADS, smem, s>>>(p);
   return check_launch("small_m_linear_mma_kernel");
+}
+}  // namespace
+
+// y = x W^T (+ res) for 1 <= M <= 8 rows on the tensor cores (x as it is: no prologue on this path).
+extern "C" int ra_small_m_linear_mma(const void* x, const void* w, void* y, const void* res, int M, int N, int K,
+                                     void* stream) {
+  using namespace ra::decode;
+  if (M < 1 || M > 8 || K % 8 || N < 1) {
+    set_error("ra_small_m_linear_mma: need 1 <= M <= 8 and K % 8 == 0");
+    return kHostBadArg;
+  }
+  LmParams p = {};
+  p.x = p.x2 = static_cast<const __nv_bfloat16*>(x);
+  p.ldx = K;
+  p.w = static_cast<const __nv_bfloat16*>(w);
+  p.y = static_cast<__nv_bfloat16*>(y);
+  p.ldy = N;
+  p.res = static_cast<const __nv_bfloat16*>(res);
+  p.n32_from = p.act_from = (N + LM_COLS - 1) / LM_COLS * LM_COLS;  // one segment
+  p.M = M; p.N = N; p.K = K;
+  return launch_small_m_mma(p, static_cast<cudaStream_t>(stream));
+}
+
+// The same product with the three output segments of LmParams; w is (N, K) dense. n32_from and act_from are multiples
+// of 16 (at least N when a segment is absent); ldx is a multiple of 8.
+extern "C" int ra_small_m_linear_segments(const void* x, const void* x2, long long ldx, const void* w, void* y,
+                                          long long ldy, float* y32, long long ldy32, int add32, void* ya,
+                                          long long ldya, int n32_from, int act_from, int M, int N, int K, void* stream) {
+  using namespace ra::decode;
+  if (M < 1 || M > 8 || K % 8 || N < 1 || ldx % 8 || n32_from % LM_COLS || act_from % LM_COLS || n32_from > act_from ||
+      (n32_from > 0 && !y) || (n32_from < act_from && n32_from < N && !y32) || (act_from < N && (!ya || !x2)) ||
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(x2) | reinterpret_cast<uintptr_t>(w)) & 15)) {
+    set_error("ra_small_m_linear_segments: bad shape");
+    return kHostBadArg;
+  }
+  LmParams p = {};
+  p.x = static_cast<const __nv_bfloat16*>(x);
+  p.x2 = static_cast<const __nv_bfloat16*>(x2);
+  p.ldx = ldx;
+  p.w = static_cast<const __nv_bfloat16*>(w);
+  p.y = static_cast<__nv_bfloat16*>(y);
+  p.ldy = ldy;
+  p.y32 = y32; p.ldy32 = ldy32; p.add32 = add32;
+  p.ya = static_cast<__nv_bfloat16*>(ya);
+  p.ldya = ldya;
+  p.n32_from = n32_from; p.act_from = act_from;
+  p.M = M; p.N = N; p.K = K;
+  return launch_small_m_mma(p, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int ra_rope_append(void* qkv, void* k_cache, void* v_cache, long long sb, long long ss, long long sh,

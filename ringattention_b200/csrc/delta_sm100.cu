@@ -349,19 +349,25 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p
 }
 
 template <typename T>
-int launch_prefill(const Params& p, cudaStream_t s) {
-  const int rows = p.B * p.T;
-  delta_prep_kernel<T><<<dim3(rows, (2 * p.G + p.H + 3) / 4), 128, 0, s>>>(p);
-  int rc = check_launch("delta_prep_kernel");
-  if (rc) return rc;
+int launch_prep(const Params& p, cudaStream_t s) {
+  delta_prep_kernel<T><<<dim3(p.B * p.T, (2 * p.G + p.H + 3) / 4), 128, 0, s>>>(p);
+  return check_launch("delta_prep_kernel");
+}
+
+template <typename T>
+int launch_scan(const Params& p, cudaStream_t s) {
   const dim3 grid((p.dv + SCAN_COLS - 1) / SCAN_COLS, p.H, p.B);
   if (p.dk <= 32) delta_scan_kernel<T, 1><<<grid, 128, 0, s>>>(p);
   else if (p.dk <= 64) delta_scan_kernel<T, 2><<<grid, 128, 0, s>>>(p);
   else if (p.dk <= 96) delta_scan_kernel<T, 3><<<grid, 128, 0, s>>>(p);
   else if (p.dk <= 128) delta_scan_kernel<T, 4><<<grid, 128, 0, s>>>(p);
   else delta_scan_kernel<T, 8><<<grid, 128, 0, s>>>(p);
-  if ((rc = check_launch("delta_scan_kernel"))) return rc;
-  delta_out_kernel<T><<<(rows * p.H + 3) / 4, 128, 0, s>>>(p);
+  return check_launch("delta_scan_kernel");
+}
+
+template <typename T>
+int launch_out(const Params& p, cudaStream_t s) {
+  delta_out_kernel<T><<<(p.B * p.T * p.H + 3) / 4, 128, 0, s>>>(p);
   return check_launch("delta_out_kernel");
 }
 
@@ -378,19 +384,30 @@ int launch_step(const Params& p, cudaStream_t s) {
   return check_launch("delta_step_kernel");
 }
 
+int check(const Params* p) {
+  if (p->B < 1 || p->T < 1 || p->H < 1 || p->G < 1 || p->H % p->G || p->dk < 1 || p->dk > 256 || p->dv < 1 ||
+      p->dv > 4096 || p->taps < 1 || p->B > 65535 || p->H > 65535 ||
+      static_cast<long long>(p->B) * p->T * p->H > (1ll << 31) - 4) {
+    set_error("ra_delta: bad shape (key dim at most 256, value dim at most 4096)");
+    return kHostBadArg;
+  }
+  return kHostOk;
+}
+
 }  // namespace delta
 }  // namespace ra
 
-// `step` 1: one token per sequence through the fused kernel (q, k, v, gb, o unused). `f32`: proj, out and the mixer's
-// vectors are fp32, else bf16.
-extern "C" int ra_delta_mixer(const ra::delta::Params* p, int step, int f32, void* stream) {
-  using namespace ra;
-  if (p->B < 1 || p->T < 1 || p->H < 1 || p->G < 1 || p->H % p->G || p->dk < 1 || p->dk > 256 || p->dv < 1 ||
-      p->dv > 4096 || p->taps < 1 || p->B > 65535 || p->H > 65535 || (step && p->T != 1)) {
-    set_error("ra_delta_mixer: bad shape (key dim at most 256, value dim at most 4096)");
-    return kHostBadArg;
+// One launcher per kernel. `f32`: proj, out and the mixer's vectors are fp32, else bf16. ra_delta_step takes T = 1 and
+// leaves q, k, v, gb and o unused; the other three together are a step of any length.
+#define RA_DELTA_ENTRY(NAME, LAUNCH)                                                                       \
+  extern "C" int NAME(const ra::delta::Params* p, int f32, void* stream) {                                 \
+    const int rc = ra::delta::check(p);                                                                    \
+    if (rc) return rc;                                                                                     \
+    cudaStream_t s = static_cast<cudaStream_t>(stream);                                                    \
+    return f32 ? ra::delta::LAUNCH<float>(*p, s) : ra::delta::LAUNCH<__nv_bfloat16>(*p, s);                \
   }
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (step) return f32 ? delta::launch_step<float>(*p, s) : delta::launch_step<__nv_bfloat16>(*p, s);
-  return f32 ? delta::launch_prefill<float>(*p, s) : delta::launch_prefill<__nv_bfloat16>(*p, s);
-}
+RA_DELTA_ENTRY(ra_delta_prep, launch_prep)
+RA_DELTA_ENTRY(ra_delta_scan, launch_scan)
+RA_DELTA_ENTRY(ra_delta_out, launch_out)
+RA_DELTA_ENTRY(ra_delta_step, launch_step)
+#undef RA_DELTA_ENTRY

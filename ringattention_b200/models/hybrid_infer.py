@@ -69,14 +69,20 @@ class HybridInference(InferenceEngine):
         main = n if L.n_split is None else L.n_split
         proj = torch.empty(rows, main, device=dev, dtype=self.dtype)
         tail = None if main == n else torch.empty(rows, n - main, device=dev, dtype=torch.float32)
-        K.linear_ex(h1, L.in_w, proj, tail=tail, n_split=L.n_split)
         both = torch.empty(rows, L.out_w.shape[1], device=dev, dtype=self.dtype)  # [heads | activations]
+        acts = both[:, L.o_cols:] if L.up_w is not None else None
+        few = rows <= 8 and self.dtype == torch.bfloat16
+        if few:  # every projection of the layer's input in one launch
+            K.linear_segments(h1, L.step_w, x2=h2, y=proj, y32=tail, ya=acts, n32_from=L.n_split,
+                              act_from=None if acts is None else L.step_w.shape[0] - L.up_w.shape[0])
+        else:
+            K.linear_ex(h1, L.in_w, proj, tail=tail, n_split=L.n_split)
         o_real = layer.mixer.heads * layer.mixer.vdim
         if o_real != L.o_cols:
             both[:, o_real:L.o_cols].zero_()
         self._mixer(i, L, proj, tail, both[:, :o_real], T, n_rows)
-        if L.up_w is not None:
-            K.linear_ex(h2, L.up_w, both[:, L.o_cols:], relu2=True)
+        if acts is not None and not few:
+            K.linear_ex(h2, L.up_w, acts, relu2=True)
         K.linear_ex(both, L.out_w, x, residual=x)
 
     def _forward(self, tokens: torch.Tensor, T: int, n_rows: int, rows_idx: Optional[torch.Tensor],

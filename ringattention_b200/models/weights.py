@@ -127,11 +127,12 @@ def random_source(cfg: HybridConfig, device, seed: int = 0) -> Callable[[str], t
 class LayerWeights:
     """Packed tensors of one layer (see the module docstring)."""
 
-    in_w: torch.Tensor                  # mixer input projections
+    step_w: torch.Tensor                # [mixer input projections | up projection], one launch of a decode step
+    in_w: torch.Tensor                  # the first part of it, zero rows up to a multiple of 16 included
     offs: Tuple[int, ...]               # first column of each projection in the product
     n_split: Optional[int]              # columns from here on leave in fp32 (decay and step-size projections)
     off_a: int
-    up_w: Optional[torch.Tensor]
+    up_w: Optional[torch.Tensor]        # the second part
     out_w: torch.Tensor                 # [mixer output projection | feed-forward down projection]
     o_cols: int                         # columns of the mixer part (padded)
     mix: Dict[str, torch.Tensor]
@@ -204,16 +205,17 @@ class HybridWeights:
         ff = 0 if layer.mlp is None else layer.mlp.ff
         L.out_w = torch.zeros(self.dp, L.o_cols + round8(ff), device=self.device, dtype=self.dtype)
         L.out_w[:self.d, :o.shape[1]] = o
-        L.up_w = L.norm2 = None
+        L.step_w, L.up_w, L.norm2 = L.in_w, None, None
         if layer.mlp is not None:
             L.norm2 = self._vec(p + "norm2")
-            L.up_w = self._rows([self._tensor(p + "mlp.up")])[0]
+            L.step_w, (_, up) = self._rows([L.in_w[:, :self.d], self._tensor(p + "mlp.up")], align=[8, 16])
+            L.in_w, L.up_w = L.step_w[:up], L.step_w[up:]
             L.out_w[:self.d, L.o_cols:L.o_cols + ff] = self._tensor(p + "mlp.down")
         return L
 
     def bytes(self) -> int:
         n = self.embed.numel() + self.head.numel()
         for L in self.layers.values():
-            n += L.in_w.numel() + L.out_w.numel() + (0 if L.up_w is None else L.up_w.numel())
+            n += L.step_w.numel() + L.out_w.numel()
             n += L.mix["ukv"].numel() if "ukv" in L.mix else 0
         return n * self.embed.element_size()

@@ -109,10 +109,38 @@ def linear_ex(x, w, out, *, residual=None, tail=None, n_split: Optional[int] = N
         _lib.call("ra_linear_f32", ptr(x), ptr(w), ptr(out), ptr(residual), ptr(tail), M, N, Kd, c_ll(x.stride(0)),
                   c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2), stream_ptr())
         return out
+    if M <= 8 and w.is_contiguous() and (residual is None or (residual.data_ptr() == out.data_ptr() and
+                                                              out.dtype == torch.float32)):
+        if out.dtype == torch.float32:
+            return linear_segments(x, w, y32=out, add32=residual is not None)
+        if relu2:
+            return linear_segments(x, w, x2=x, ya=out, act_from=0)
+        return linear_segments(x, w, y=out, y32=tail, n32_from=None if tail is None else n_split)
     _lib.call("ra_gemm_bf16_ex", ptr(x), ptr(w), ptr(out), ptr(residual), ptr(tail), M, N, Kd, c_ll(x.stride(0)),
               c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2),
               int(out.dtype == torch.float32), 8, _status(), stream_ptr())
     return out
+
+
+def linear_segments(x, w, *, x2=None, y=None, y32=None, ya=None, n32_from: Optional[int] = None,
+                    act_from: Optional[int] = None, add32: bool = False):
+    """At most 8 rows: ``x W^T`` in one launch with the columns in up to three segments, each with an output of its own:
+    bf16 to ``y``, from ``n32_from`` on fp32 to ``y32`` (added to it with ``add32``), from ``act_from`` on the squared relu
+    of ``x2 W^T`` in bf16 to ``ya``. Borders are multiples of 16; outputs are row-strided views. Without ``y`` the fp32
+    segment starts at 0. Returns ``y``, ``y32`` or ``ya``, the first that is there."""
+    M, Kd = x.shape
+    N = w.shape[0]
+    end = (N + 15) // 16 * 16
+    act_from = end if act_from is None else act_from
+    n32_from = (act_from if y is not None or act_from == 0 else 0) if n32_from is None else n32_from
+    assert M <= 8 and w.is_contiguous() and w.shape[1] == Kd and x.stride(1) == 1 and x.dtype == w.dtype == torch.bfloat16
+    assert x2 is None or (x2.shape == x.shape and x2.stride() == x.stride())
+    for t, n in ((y, min(n32_from, N)), (y32, min(act_from, N) - n32_from), (ya, N - act_from)):
+        assert t is None or (t.shape[0] == M and t.stride(1) == 1 and t.shape[1] >= n)
+    ld = lambda t: c_ll(0 if t is None else t.stride(0))
+    _lib.call("ra_small_m_linear_segments", ptr(x), ptr(x2), c_ll(x.stride(0)), ptr(w), ptr(y), ld(y), ptr(y32), ld(y32),
+              int(add32), ptr(ya), ld(ya), n32_from, act_from, M, N, Kd, stream_ptr())
+    return y if y is not None else (y32 if y32 is not None else ya)
 
 
 # ---------------------------------------------------------------------------------------------

@@ -4,10 +4,12 @@ and softmax are fp32 in both."""
 from __future__ import annotations
 
 import ctypes
+import os
 
 import torch
 
 from . import _lib
+from . import kernels as K
 
 c_ll = ctypes.c_longlong
 c_vp = ctypes.c_void_p
@@ -61,8 +63,8 @@ def delta_mixer(proj, ba, out, *, B: int, T: int, m, offs, off_a: int, w, ring, 
         gb = torch.empty(rows, H, 2, **f32)
         a.q, a.k, a.v, a.gb, a.o = _p(q), _p(k), _p(v), _p(gb), _p(o)
     a.out, a.ldo, a.eps, a.q_scale, a.pos = _p(out), out.stride(0), eps, dk ** -0.5, _p(pos)
-    _lib.call("ra_delta_mixer", ctypes.byref(a), int(step), int(proj.dtype == torch.float32), _lib.stream_ptr(),
-              n_kernels=1 if step else 3)
+    for entry in ("ra_delta_step",) if step else ("ra_delta_prep", "ra_delta_scan", "ra_delta_out"):
+        _lib.call(entry, ctypes.byref(a), int(proj.dtype == torch.float32), _lib.stream_ptr())
 
 
 class _LatentParams(ctypes.Structure):
@@ -84,10 +86,9 @@ def latent_mixer(proj, out, *, B: int, T: int, m, offs, w, cache, n_rows: int, e
     """Latent attention of ``T`` new tokens of each of ``B`` sequences over the cached rows, which the new tokens join.
 
     ``proj (B*T, ld)``: query heads, [latent | shared key] and output gates at columns ``offs`` (the rotated query parts are
-    turned in place). ``cache (B, S_max, row)``; ``n_rows``: an upper bound of the rows that will be visible (sizes the
-    grid only). ``w``: ``c_norm``, ``inv_freq``, ``uk``, ``uv``, ``sink``. ``m``: a
-    :class:`~ringattention_b200.config.LatentAttentionConfig`."""
-    dev = proj.device
+    turned in place). ``cache (B, S_max, row)``; ``n_rows``: the rows that will be visible, or for a single token an upper
+    bound of them (it sizes grids; the kernels take the count from ``pos``). ``w``: ``c_norm``, ``inv_freq``, ``ukv`` with
+    its parts ``uk`` and ``uv``, ``sink``. ``m``: a :class:`~ringattention_b200.config.LatentAttentionConfig`."""
     rows, H = B * T, m.heads
     assert proj.shape[0] == rows and proj.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype
     assert cache.is_contiguous() and cache.dtype == proj.dtype and cache.shape[0] == B
@@ -99,13 +100,74 @@ def latent_mixer(proj, out, *, B: int, T: int, m, offs, w, cache, n_rows: int, e
     a.off_q, a.off_c, a.off_g = offs
     a.c_norm, a.inv_freq, a.cache, a.S_max = _p(w["c_norm"]), _p(w["inv_freq"]), _p(cache), cache.shape[1]
     a.w_uk, a.w_uv, a.ldw, a.sink = _p(w["uk"]), _p(w["uv"]), w["uk"].stride(0), _p(w["sink"])
+    a.out, a.ldo, a.eps, a.scale, a.pos = _p(out), out.stride(0), eps, m.scale, _p(pos)
+    a.splits, is32 = 1, int(proj.dtype == torch.float32)
+    _lib.call("ra_latent_prep", ctypes.byref(a), is32, _lib.stream_ptr())
+    if T >= EXPAND_MIN_TOKENS and two_part_fits(m, proj, out, offs):
+        return _latent_expanded(proj, out, B, T, m, offs, w, cache, n_rows)
+    f32 = dict(device=proj.device, dtype=torch.float32)
     a.splits = latent_splits(rows, H, n_rows)
-    f32 = dict(device=dev, dtype=torch.float32)
     q_lat = torch.empty(rows, H, a.row_w, **f32)
     o_part = torch.empty(rows, H, a.splits, m.kv_rank, **f32)
     lse = torch.empty(rows, H, a.splits, **f32)
     a.q_lat, a.o_part, a.lse_part = _p(q_lat), _p(o_part), _p(lse)
-    a.out, a.ldo, a.eps, a.scale, a.pos = _p(out), out.stride(0), eps, m.scale, _p(pos)
-    is32 = int(proj.dtype == torch.float32)
-    _lib.call("ra_latent_prep", ctypes.byref(a), is32, _lib.stream_ptr())
     _lib.call("ra_latent_absorbed", ctypes.byref(a), is32, _lib.stream_ptr(), n_kernels=3)
+
+
+# From this many tokens of a sequence per step on, keys and values are made from the cached latents (one product over all
+# of them, H (dim + vdim) columns) and the tensor-core attention runs per head; below, the queries go to the latents.
+EXPAND_MIN_TOKENS = int(os.environ.get("RINGATTN_B200_LATENT_EXPAND_MIN_TOKENS", "96"))
+
+
+class _TwoPartArgs(ctypes.Structure):
+    _fields_ = [("q", c_vp), ("q_sb", c_ll), ("q_ss", c_ll), ("q_sh", c_ll),
+                ("k1", c_vp), ("k1_sb", c_ll), ("k1_ss", c_ll), ("k1_sh", c_ll),
+                ("k2", c_vp), ("k2_sb", c_ll), ("k2_ss", c_ll),
+                ("v", c_vp), ("v_sb", c_ll), ("v_ss", c_ll), ("v_sh", c_ll),
+                ("out", c_vp), ("o_sb", c_ll), ("o_ss", c_ll), ("o_sh", c_ll),
+                ("sink", c_vp), ("gate", c_vp), ("gate_ld", c_ll),
+                ("B", c_i), ("H", c_i), ("Sq", c_i), ("Sk", c_i), ("d1", c_i), ("d2", c_i), ("dv", c_i),
+                ("scale", c_f), ("q_pos0", c_i), ("status", c_vp), ("stream", c_vp)]
+
+
+def two_part_attention(q, k1, k2, v, out, *, scale: float, q_pos0: int, sink=None, gate=None) -> None:
+    """Causal attention on the tensor cores with two-part keys: ``score = (q1 . k1 + q2 . k2) * scale``.
+
+    ``q (B, Sq, H, d1 + d2)``, ``k1 (B, Sk, H, d1)``, ``k2 (B, Sk, d2)`` shared by the heads, ``v (B, Sk, H, dv)``, ``out (B, Sq,
+    H, dv)``: bf16 views, innermost contiguous. Query i sits at position ``q_pos0 + i``. ``sink (H,)`` fp32: one more entry
+    ``exp(sink)`` in each denominator; ``gate (B*Sq, H)``: bf16 view, the head's output is multiplied by its sigmoid."""
+    B, Sq, H, _ = q.shape
+    a = _TwoPartArgs()
+    a.q, (a.q_sb, a.q_ss, a.q_sh) = _p(q), q.stride()[:3]
+    a.k1, (a.k1_sb, a.k1_ss, a.k1_sh) = _p(k1), k1.stride()[:3]
+    a.k2, (a.k2_sb, a.k2_ss) = _p(k2), k2.stride()[:2]
+    a.v, (a.v_sb, a.v_ss, a.v_sh) = _p(v), v.stride()[:3]
+    a.out, (a.o_sb, a.o_ss, a.o_sh) = _p(out), out.stride()[:3]
+    a.sink, a.gate, a.gate_ld = _p(sink), _p(gate), 0 if gate is None else gate.stride(0)
+    a.B, a.H, a.Sq, a.Sk = B, H, Sq, k1.shape[1]
+    a.d1, a.d2, a.dv = k1.shape[3], k2.shape[2], v.shape[3]
+    a.scale, a.q_pos0 = scale, q_pos0
+    a.status, a.stream = _lib.status_tensor(q.device).data_ptr(), torch.cuda.current_stream().cuda_stream
+    _lib.call("ra_attn_two_part", ctypes.byref(a))
+
+
+def two_part_fits(m, proj, out, offs) -> bool:
+    """Sizes the tensor-core kernel takes (every part starts at a multiple of 16 bytes)."""
+    return (proj.dtype == torch.bfloat16 and 8 <= m.dim <= 128 and 8 <= m.rot_dim <= 64 and 8 <= m.vdim <= 128
+            and not (m.dim % 8 or m.rot_dim % 8 or m.vdim % 8 or offs[0] % 8 or proj.stride(0) % 8 or out.stride(0) % 8
+                     or out.data_ptr() % 16))
+
+
+def _latent_expanded(proj, out, B: int, T: int, m, offs, w, cache, n: int) -> None:
+    H, dn, dr, dv = m.heads, m.dim, m.rot_dim, m.vdim
+    S_max, width = cache.shape[1:]
+    r_pad = (m.kv_rank + 7) // 8 * 8
+    kv = torch.empty(B, n, w["ukv"].shape[0], device=proj.device, dtype=proj.dtype)
+    for b in range(B):
+        K.linear_ex(cache[b, :n, :r_pad], w["ukv"], kv[b])
+    ld = proj.stride(0)
+    q = proj.as_strided((B, T, H, dn + dr), (T * ld, ld, dn + dr, 1), proj.storage_offset() + offs[0])
+    o = out.as_strided((B, T, H, dv), (T * out.stride(0), out.stride(0), dv, 1), out.storage_offset())
+    two_part_attention(q, kv[:, :, :H * dn].view(B, n, H, dn), cache[:, :n, r_pad:r_pad + dr],
+                       kv[:, :, w["uv_off"]:w["uv_off"] + H * dv].view(B, n, H, dv), o, scale=m.scale, q_pos0=n - T,
+                       sink=w["sink"], gate=proj[:, offs[2]:offs[2] + H])
