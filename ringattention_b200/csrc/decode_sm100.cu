@@ -23,6 +23,7 @@
 
 #include "common/bounds.cuh"
 #include "common/host_util.h"
+#include "common/mma_sync.cuh"
 #include "common/sm100.cuh"
 
 RA_BOUNDS_TRANSLATION_UNIT()
@@ -78,17 +79,6 @@ __device__ __forceinline__ uint4 pack8(const float* f) {
 #pragma unroll
   for (int i = 0; i < 4; ++i) b[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
   return u;
-}
-
-// 16-byte asynchronous copy global -> shared; `bytes` = 0 writes zeros without reading the source.
-__device__ __forceinline__ void cp_async16(void* smem_dst, const void* gsrc, int bytes) {
-  const uint32_t d = static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst));
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(gsrc), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
 constexpr int DEC_UNROLL = 4;  // cache rows per thread and loop trip
@@ -307,26 +297,6 @@ __global__ void __launch_bounds__(THREADS) decode_splitkv_kernel(const SplitPara
 // XOR-swizzled by the row so that ldmatrix is conflict-free); only __syncwarp() is needed around a stage. The legacy
 // mma.sync path is the right size here: the kernel is bound by HBM, a 128-row tcgen05 tile would bring nothing but a
 // longer hand-off chain per tile.
-__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem_row) {
-  const uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(smem_row));
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(a));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* smem_row) {
-  const uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(smem_row));
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(a));
-}
-// d += a * b for m16n8k16, bf16 inputs, fp32 accumulation; rows 8..15 of a are zero (a1 = a3 = 0)
-__device__ __forceinline__ void mma_16816_top(float (&d)[4], uint32_t a0, uint32_t a2, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a0), "r"(0u), "r"(a2), "r"(0u), "r"(b0), "r"(b1));
-}
-
 constexpr int MMA_ST = 3;       // stages of a warp's ring
 constexpr int MMA_ROWS = 16;    // cache rows per chunk
 

@@ -13,56 +13,12 @@
 // step reads the rows of the taps - 1 tokens before it and writes the rows of its own last tokens. The state is stored
 // transposed, (dv, dk), so that the eight lanes of a column read 128 contiguous bytes.
 // Everything here is fp32 except the projections that come in.
-#include "common/bounds.cuh"
-#include "common/host_util.h"
-#include "common/numeric.cuh"
+#include "delta_common.cuh"
 
 RA_BOUNDS_TRANSLATION_UNIT()
 
 namespace ra {
 namespace delta {
-
-struct Params {
-  int B, T, H, G, dk, dv, taps;  // T tokens per sequence in this step; row b * T + t
-  const void* proj;              // (rows, ldp): columns off_q / off_k / off_v / off_g
-  long long ldp;
-  int off_q, off_k, off_v, off_g;
-  const float* ba;               // (rows, ldba): beta's projection at 0, the decay's at off_a
-  long long ldba;
-  int off_a;
-  const void *conv_q, *conv_k, *conv_v;  // (channels, taps)
-  const void *a_log, *dt_bias, *norm_w;  // (H), (H), (dv)
-  float* ring;                   // (B, taps, C) with C = 2 G dk + H dv, channels in the order q, k, v
-  float* state;                  // (B, H, dv, dk)
-  float *q, *k, *v, *gb, *o;     // (rows, G, dk) x 2, (rows, H, dv), (rows, H, 2), (rows, H, dv)
-  void* out;                     // (rows, ldo)
-  long long ldo;
-  float eps, q_scale;
-  const long long* pos;          // position of the step's first token
-};
-
-__device__ __forceinline__ int ring_slot(long long p, int taps) { return static_cast<int>(p % taps); }
-
-// silu(convolution) of one channel at token t of the step. `c`: channel in the ring's order, `col`: its projection column.
-template <typename T>
-__device__ __forceinline__ float conv_silu(const Params& p, const T* proj_b, const float* ring_b, const T* w, int t,
-                                           long long pos0, int C, int c, int col) {
-  float s = 0.f;
-  for (int j = 0; j < p.taps; ++j) {
-    const int tt = t - (p.taps - 1 - j);
-    float x = 0.f;
-    if (tt >= 0)
-      x = to_f(proj_b[tt * p.ldp + col]);
-    else if (pos0 + tt >= 0)
-      x = ring_b[static_cast<long long>(ring_slot(pos0 + tt, p.taps)) * C + c];
-    s = fmaf(to_f(w[j]), x, s);
-  }
-  return silu_f(s);
-}
-
-__device__ __forceinline__ float decay_of(const Params& p, float a, float a_log, float dt) {
-  return expf(-expf(a_log) * softplus_f(a + dt));
-}
 
 // grid (rows, ceil((2 G + H) / 4)), four warps; unit u: q head u, k head u - G, v head u - 2 G
 template <typename T>
@@ -98,8 +54,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const Params p) {
     if (lane == 0) {
       const float* ba = p.ba + row * p.ldba;
       float* gb = p.gb + (static_cast<long long>(row) * p.H + hd) * 2;
-      gb[0] = decay_of(p, ba[p.off_a + hd], to_f(static_cast<const T*>(p.a_log)[hd]),
-                       to_f(static_cast<const T*>(p.dt_bias)[hd]));
+      gb[0] = expf(log_decay(ba[p.off_a + hd], to_f(static_cast<const T*>(p.a_log)[hd]), to_f(static_cast<const T*>(p.dt_bias)[hd])));
       gb[1] = sigmoid_f(ba[hd]);
     }
   }
@@ -120,20 +75,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const Params p) {
   const bool in = col < p.dv;
   const long long pos0 = *p.pos;
 
-  // ---- the rows of the step's last tokens go into the convolution ring (nobody reads the ring in this launch)
-  {
-    const int C = 2 * p.G * p.dk + p.H * p.dv;
-    const int blocks = gridDim.x * gridDim.y;
-    const int me = blockIdx.y * gridDim.x + blockIdx.x;
-    const int keep = min(p.T, p.taps);
-    const T* proj_b = static_cast<const T*>(p.proj) + static_cast<long long>(b) * p.T * p.ldp;
-    float* ring_b = p.ring + static_cast<long long>(b) * p.taps * C;
-    for (int i = me * 128 + tid; i < keep * C; i += blocks * 128) {
-      const int t = p.T - keep + i / C, c = i % C, nq = p.G * p.dk;
-      const int src = c < nq ? p.off_q + c : (c < 2 * nq ? p.off_k + c - nq : p.off_v + c - 2 * nq);
-      ring_b[static_cast<long long>(ring_slot(pos0 + t, p.taps)) * C + c] = to_f(proj_b[t * p.ldp + src]);
-    }
-  }
+  // nobody reads the ring in this launch
+  save_ring<T>(p, b, pos0, (blockIdx.y * gridDim.x + blockIdx.x) * 128 + tid, gridDim.x * gridDim.y * 128);
 
   float S[NJ][4];
   float* st = p.state + ((static_cast<long long>(b) * p.H + h) * p.dv + (in ? col : 0)) * p.dk;
@@ -271,7 +214,7 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p
     if (lane == 0) scal[warp] = (warp == 0 ? p.q_scale : 1.f) / sqrtf(ss + 1e-6f);
   } else if (tid == 64) {
     const float* ba = p.ba + b * p.ldba;
-    scal[2] = decay_of(p, ba[p.off_a + h], to_f(static_cast<const T*>(p.a_log)[h]), to_f(static_cast<const T*>(p.dt_bias)[h]));
+    scal[2] = expf(log_decay(ba[p.off_a + h], to_f(static_cast<const T*>(p.a_log)[h]), to_f(static_cast<const T*>(p.dt_bias)[h])));
     scal[3] = sigmoid_f(ba[h]);
   }
   __syncthreads();

@@ -30,7 +30,21 @@ class _DeltaParams(ctypes.Structure):
                 ("a_log", c_vp), ("dt_bias", c_vp), ("norm_w", c_vp),
                 ("ring", c_vp), ("state", c_vp),
                 ("q", c_vp), ("k", c_vp), ("v", c_vp), ("gb", c_vp), ("o", c_vp),
-                ("out", c_vp), ("ldo", c_ll), ("eps", c_f), ("q_scale", c_f), ("pos", c_vp)]
+                ("out", c_vp), ("ldo", c_ll), ("eps", c_f), ("q_scale", c_f), ("pos", c_vp),
+                ("n_chunks", c_i), ("ws_qk", c_vp), ("ws_w", c_vp), ("ws_u", c_vp), ("ws_m", c_vp), ("ws_d", c_vp),
+                ("status", c_vp)]
+
+
+# From this many tokens per step on the recurrence runs in chunks on the tensor cores (bf16 engines; 32-bit operands as
+# sums of two bf16 numbers); below, and in fp32 engines, token by token on the CUDA cores.
+CHUNK_MIN_TOKENS = int(os.environ.get("RINGATTN_B200_DELTA_CHUNK_MIN_TOKENS", "48"))
+CHUNK = 64
+
+
+def delta_chunk_fits(m, proj, offs) -> bool:
+    """Sizes the chunked kernels take."""
+    return (proj.dtype == torch.bfloat16 and m.dim in (64, 128) and m.vdim in (64, 128) and m.conv <= 4
+            and not any(o % 4 for o in offs) and proj.stride(0) % 4 == 0 and proj.data_ptr() % 16 == 0)
 
 
 def delta_mixer(proj, ba, out, *, B: int, T: int, m, offs, off_a: int, w, ring, state, eps: float, pos) -> None:
@@ -56,14 +70,27 @@ def delta_mixer(proj, ba, out, *, B: int, T: int, m, offs, off_a: int, w, ring, 
     a.conv_q, a.conv_k, a.conv_v = _p(w["conv_q"]), _p(w["conv_k"]), _p(w["conv_v"])
     a.a_log, a.dt_bias, a.norm_w = _p(w["a_log"]), _p(w["dt_bias"]), _p(w["norm"])
     a.ring, a.state = _p(ring), _p(state)
+    a.out, a.ldo, a.eps, a.q_scale, a.pos = _p(out), out.stride(0), eps, dk ** -0.5, _p(pos)
+    entries = ("ra_delta_step",)
     if not step:
         f32 = dict(device=dev, dtype=torch.float32)
-        q, k = torch.empty(rows, G, dk, **f32), torch.empty(rows, G, dk, **f32)
-        v, o = torch.empty(rows, H, dv, **f32), torch.empty(rows, H, dv, **f32)
-        gb = torch.empty(rows, H, 2, **f32)
-        a.q, a.k, a.v, a.gb, a.o = _p(q), _p(k), _p(v), _p(gb), _p(o)
-    a.out, a.ldo, a.eps, a.q_scale, a.pos = _p(out), out.stride(0), eps, dk ** -0.5, _p(pos)
-    for entry in ("ra_delta_step",) if step else ("ra_delta_prep", "ra_delta_scan", "ra_delta_out"):
+        o = torch.empty(rows, H, dv, **f32)
+        a.o = _p(o)
+        if T >= CHUNK_MIN_TOKENS and delta_chunk_fits(m, proj, offs):
+            n = a.n_chunks = (T + CHUNK - 1) // CHUNK
+            u8 = dict(device=dev, dtype=torch.uint8)
+            ws = (torch.empty(B, G, n, 8 * CHUNK * dk, **u8), torch.empty(B, H, n, 4 * CHUNK * dk, **u8),
+                  torch.empty(B, H, n, dv * CHUNK, **f32), torch.empty(B, H, n, 4 * CHUNK * CHUNK + 4 * CHUNK, **u8),
+                  torch.empty(B, H, n, CHUNK + 4, **f32))
+            a.ws_qk, a.ws_w, a.ws_u, a.ws_m, a.ws_d = (_p(t) for t in ws)
+            a.status = _lib.status_tensor(dev).data_ptr()
+            entries = ("ra_delta_chunk_prep", "ra_delta_chunk_scan", "ra_delta_out")
+        else:
+            q, k = torch.empty(rows, G, dk, **f32), torch.empty(rows, G, dk, **f32)
+            v, gb = torch.empty(rows, H, dv, **f32), torch.empty(rows, H, 2, **f32)
+            a.q, a.k, a.v, a.gb = _p(q), _p(k), _p(v), _p(gb)
+            entries = ("ra_delta_prep", "ra_delta_scan", "ra_delta_out")
+    for entry in entries:
         _lib.call(entry, ctypes.byref(a), int(proj.dtype == torch.float32), _lib.stream_ptr())
 
 

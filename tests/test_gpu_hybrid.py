@@ -146,7 +146,8 @@ def run_delta(m, proj, ba, w, state, ring, pos, sizes, dtype, eps):
 
 
 @pytest.mark.parametrize("dtype", BOTH)
-@pytest.mark.parametrize("shape", [(6, 2, 24, 40, 4), (4, 4, 128, 128, 3), (2, 1, 200, 24, 2), (3, 3, 64, 96, 1), (4, 2, 128, 64, 4)])
+@pytest.mark.parametrize("shape", [(6, 2, 24, 40, 4), (4, 4, 128, 128, 3), (2, 1, 200, 24, 2), (3, 3, 64, 96, 1), (4, 2, 128, 64, 4), (5, 1, 64, 128, 2),
+                                   (2, 2, 64, 64, 1), (40, 20, 128, 128, 4)])
 def test_delta_mixer_alone(dtype, shape):
     """Decays from almost 0 to almost 1, large and small step sizes, repeated keys (where the delta rule differs most from
     a plain sum), whole and in pieces, with the state carried on."""
@@ -186,7 +187,7 @@ def test_delta_mixer_alone(dtype, shape):
         got, _ = run_delta(m, proj.cuda(), ba.cuda(), wc, state, ring, 0, sizes, dtype, 1e-5)
         tol = 2e-4 if dtype == torch.float32 else 0.02
         assert (got.double().cpu() - want).abs().max() <= tol * want.abs().max(), sizes
-        # the state is fp32 in both types: only the order of its sums differs from the reference
+        # the state is fp32 in both types: the order of its sums, and in the chunked form the two-term operands, differ
         assert (state[0].double().cpu() - S.transpose(1, 2)).abs().max() <= 2e-4 * S.abs().max(), sizes
 
 
