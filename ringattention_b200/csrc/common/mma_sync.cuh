@@ -43,7 +43,7 @@ __device__ __forceinline__ void mma_16816_top(float (&d)[4], uint32_t a0, uint32
 }
 
 __device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -69,11 +69,17 @@ __device__ __forceinline__ void split_a_frag(const float (&c)[4], const float (&
   split_pack(d[0], d[1], hi[2], lo[2]);
   split_pack(d[2], d[3], hi[3], lo[3]);
 }
-__device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0,
-                                          uint32_t bh1, uint32_t bl0, uint32_t bl1) {
-  mma_16816(d, ah, bh0, bh1);
-  mma_16816(d, ah, bl0, bl1);
-  mma_16816(d, al, bh0, bh1);
+// Two column tiles (b[0..1] and b[2..3], as ldmatrix.x4 delivers them) of each of N products that share the A fragment:
+// d[2 i], d[2 i + 1] += A B_i. The three terms run over all tiles in turn, so that no MMA waits for the one before it.
+template <int N>
+__device__ __forceinline__ void mma_split(float (*const (&d)[2 * N])[4], const uint32_t (&ah)[4], const uint32_t (&al)[4],
+                                          const uint32_t (&bh)[N][4], const uint32_t (&bl)[N][4]) {
+#pragma unroll
+  for (int i = 0; i < 2 * N; ++i) mma_16816(*d[i], ah, bh[i >> 1][2 * (i & 1)], bh[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+  for (int i = 0; i < 2 * N; ++i) mma_16816(*d[i], ah, bl[i >> 1][2 * (i & 1)], bl[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+  for (int i = 0; i < 2 * N; ++i) mma_16816(*d[i], al, bh[i >> 1][2 * (i & 1)], bh[i >> 1][2 * (i & 1) + 1]);
 }
 
 }  // namespace ra

@@ -47,6 +47,9 @@ __device__ __forceinline__ float sum_block(float v, float* red) {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// with the hardware's exponential and division (a few units in the last place of fp32): for activations that are rounded
+// to bf16 or might as well be
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 }  // namespace ra

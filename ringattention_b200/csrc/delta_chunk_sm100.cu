@@ -47,14 +47,34 @@ struct PrepSmem {
   static constexpr int Q_HI = 0, Q_LO = QK, K_HI = 2 * QK, K_LO = 3 * QK;
   static constexpr int V = 4 * QK;                      // fp32 (CH, DV)
   static constexpr int A = V + CH * DV * 4;             // fp32 (CH, CH)
-  static constexpr int S = A + CH * CH * 4;             // beta, log-decay sums
-  static constexpr int TOTAL = S + 2 * CH * 4;
+  static constexpr int S = A + CH * CH * 4;             // beta, log-decay sums, -beta c
+  static constexpr int TOTAL = S + 3 * CH * 4;
 };
 
-// silu(convolution) of N neighbouring channels at eight consecutive tokens t0 .. t0 + 7 of the step; fn(row, values)
+// The rows t0 - 3 .. t0 + 7 of N neighbouring channels, as they lie in the projections (rows outside the step: zero).
+constexpr int CONV_ROWS = 8 + CONV_MAX - 1;
+template <int N>
+__device__ __forceinline__ void conv_load(const Params& p, const bf16* src, int t0, uint32_t (&raw)[CONV_ROWS][N / 2]) {
+#pragma unroll
+  for (int i = 0; i < CONV_ROWS; ++i) {
+    const int t = t0 - (CONV_MAX - 1) + i;
+    const bool in = t >= 0 && t < p.T;
+    const bf16* s = src + (in ? t : 0) * p.ldp;
+    if (N == 4) {
+      const uint2 v = __ldg(reinterpret_cast<const uint2*>(s));
+      raw[i][0] = in ? v.x : 0u;
+      raw[i][N / 2 - 1] = in ? v.y : 0u;
+    } else {
+      const uint32_t v = __ldg(reinterpret_cast<const uint32_t*>(s));
+      raw[i][0] = in ? v : 0u;
+    }
+  }
+}
+
+// silu(convolution) of those channels at the eight tokens t0 .. t0 + 7; fn(row, values). `c`: first channel in the ring's order.
 template <int N, typename F>
-__device__ __forceinline__ void conv_rows(const Params& p, const bf16* proj_b, const float* ring_b, int C, const bf16* w, int c,
-                                          int col, int t0, long long pos0, F fn) {
+__device__ __forceinline__ void conv_rows(const Params& p, const uint32_t (&raw)[CONV_ROWS][N / 2], const float* ring_b, int C,
+                                          const bf16* w, int c, int t0, long long pos0, F fn) {
   float wt[CONV_MAX][N], win[CONV_MAX][N];
 #pragma unroll
   for (int j = 0; j < CONV_MAX; ++j)
@@ -63,39 +83,36 @@ __device__ __forceinline__ void conv_rows(const Params& p, const bf16* proj_b, c
       const int jj = j - (CONV_MAX - p.taps);
       wt[j][e] = jj >= 0 ? to_f(w[e * p.taps + jj]) : 0.f;
     }
-  auto load = [&](int t, float (&x)[N]) {
-    if (t >= 0 && t < p.T) {
-      const bf16* src = proj_b + t * p.ldp + col;
-      if (N == 4) {
-        const float4 v = load4(src);
-        x[0] = v.x; x[1] = v.y; x[2 % N] = v.z; x[3 % N] = v.w;
-      } else {
-        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src));
-        x[0] = v.x; x[1] = v.y;
-      }
-    } else {
-      const bool past = t < 0 && pos0 + t >= 0 && -t < p.taps;
-      const float* src = ring_b + (past ? static_cast<long long>(ring_slot(pos0 + t, p.taps)) * C : 0) + c;
+  auto row = [&](int i, float (&x)[N]) {
 #pragma unroll
-      for (int e = 0; e < N; ++e) x[e] = past ? src[e] : 0.f;
+    for (int e = 0; e < N; e += 2) {
+      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[i][e / 2]));
+      x[e] = v.x;
+      x[e + 1] = v.y;
+    }
+    const int t = t0 - (CONV_MAX - 1) + i;
+    if (t < 0 && pos0 + t >= 0 && -t < p.taps) {  // the step's first tokens look at earlier steps
+      const float* src = ring_b + static_cast<long long>(ring_slot(pos0 + t, p.taps)) * C + c;
+#pragma unroll
+      for (int e = 0; e < N; ++e) x[e] = src[e];
     }
   };
 #pragma unroll
-  for (int j = 1; j < CONV_MAX; ++j) load(t0 - CONV_MAX + j, win[j]);
+  for (int j = 1; j < CONV_MAX; ++j) row(j - 1, win[j]);
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
 #pragma unroll
     for (int j = 0; j + 1 < CONV_MAX; ++j)
 #pragma unroll
       for (int e = 0; e < N; ++e) win[j][e] = win[j + 1][e];
-    load(t0 + i, win[CONV_MAX - 1]);
+    row(i + CONV_MAX - 1, win[CONV_MAX - 1]);
     float y[N];
 #pragma unroll
     for (int e = 0; e < N; ++e) {
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < CONV_MAX; ++j) s = fmaf(wt[j][e], win[j][e], s);
-      y[e] = t0 + i < p.T ? silu_f(s) : 0.f;
+      y[e] = t0 + i < p.T ? silu_fast(s) : 0.f;
     }
     fn(i, y);
   }
@@ -108,7 +125,7 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
   float* sV = reinterpret_cast<float*>(smem + SM::V);
   float* sA = reinterpret_cast<float*>(smem + SM::A);
   float* sBeta = reinterpret_cast<float*>(smem + SM::S);
-  float* sCs = sBeta + CH;
+  float *sCs = sBeta + CH, *sBc = sCs + CH;
   const int chunk = blockIdx.x, h = blockIdx.y, b = blockIdx.z, rep = p.H / p.G, kvh = h / rep;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int t0 = chunk * CH;
@@ -125,12 +142,13 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
 
   // ---- step sizes and running sums of the log decays (padding tokens: no decay, no step)
   if (warp == 0) {
-    float lg[2];
+    float lg[2], be[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int t = 2 * lane + i;
       lg[i] = 0.f;
-      float beta = 0.f;
+      float& beta = be[i];
+      beta = 0.f;
       if (t0 + t < p.T) {
         const float* ba = p.ba + (static_cast<long long>(b) * p.T + t0 + t) * p.ldba;
         lg[i] = log_decay(ba[p.off_a + h], to_f(static_cast<const bf16*>(p.a_log)[h]),
@@ -150,8 +168,11 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
     sCs[2 * lane] = c0;
     sCs[2 * lane + 1] = c1;
     float* g_c = reinterpret_cast<float*>(g_m + 2 * M_TILE);
-    g_c[2 * lane] = expf(c0);
-    g_c[2 * lane + 1] = expf(c1);
+    const float e0 = expf(c0), e1 = expf(c1);
+    g_c[2 * lane] = e0;
+    g_c[2 * lane + 1] = e1;
+    sBc[2 * lane] = -be[0] * e0;
+    sBc[2 * lane + 1] = -be[1] * e1;
     g_d[2 * lane] = expf(last - c0);
     g_d[2 * lane + 1] = expf(last - c1);
     if (lane == 0) g_d[CH] = expf(last);
@@ -159,36 +180,39 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
 
   // ---- convolutions, silu, unit norms: a warp takes eight tokens, a lane DK / 32 channels
   {
-    constexpr int N = DK / 32;
+    constexpr int N = DK / 32, NV = DV / 32;
     const bool write = h % rep == 0;
+    const int tw = t0 + warp * 8, cq = kvh * DK + lane * N, cv = h * DV + lane * NV;
+    uint32_t rq[CONV_ROWS][N / 2], rk[CONV_ROWS][N / 2], rv[CONV_ROWS][NV / 2];
+    conv_load<N>(p, proj_b + p.off_q + cq, tw, rq);
+    conv_load<N>(p, proj_b + p.off_k + cq, tw, rk);
+    conv_load<NV>(p, proj_b + p.off_v + cv, tw, rv);
+    auto unit_row = [&](int i, float (&y)[N], float mul, uint8_t* hi_tile, uint8_t* lo_tile) {
+      float ss = 0.f;
 #pragma unroll
-    for (int which = 0; which < 2; ++which) {
-      const int c = which * p.G * DK + kvh * DK + lane * N;
-      const bf16* w = static_cast<const bf16*>(which ? p.conv_k : p.conv_q) + (static_cast<long long>(kvh) * DK + lane * N) * p.taps;
-      const float mul = which ? 1.f : p.q_scale;
-      conv_rows<N>(p, proj_b, ring_b, C, w, c, (which ? p.off_k : p.off_q) + kvh * DK + lane * N, t0 + warp * 8, pos0,
-                   [&](int i, float (&y)[N]) {
-                     float ss = 0.f;
+      for (int e = 0; e < N; ++e) ss += y[e] * y[e];
+      const float f = mul / sqrtf(sum_warp(ss) + 1e-6f);
+      const uint32_t off = tile_off(warp * 8 + i, lane * N, DK);
+      uint32_t hi[N / 2], lo[N / 2];
 #pragma unroll
-                     for (int e = 0; e < N; ++e) ss += y[e] * y[e];
-                     const float f = mul / sqrtf(sum_warp(ss) + 1e-6f);
-                     const int row = warp * 8 + i;
-                     const uint32_t off = tile_off(row, lane * N, DK);
-#pragma unroll
-                     for (int e = 0; e < N; e += 2) {
-                       uint32_t hi, lo;
-                       split_pack(y[e] * f, y[e + 1] * f, hi, lo);
-                       *reinterpret_cast<uint32_t*>(smem + (which ? SM::K_HI : SM::Q_HI) + off + e * 2) = hi;
-                       *reinterpret_cast<uint32_t*>(smem + (which ? SM::K_LO : SM::Q_LO) + off + e * 2) = lo;
-                     }
-                   });
-    }
-    constexpr int NV = DV / 32;
-    const int c = 2 * p.G * DK + h * DV + lane * NV;
-    conv_rows<NV>(p, proj_b, ring_b, C, static_cast<const bf16*>(p.conv_v) + (static_cast<long long>(h) * DV + lane * NV) * p.taps,
-                  c, p.off_v + h * DV + lane * NV, t0 + warp * 8, pos0, [&](int i, float (&y)[NV]) {
-#pragma unroll
-                    for (int e = 0; e < NV; ++e) sV[(warp * 8 + i) * DV + lane * NV + e] = y[e];
+      for (int e = 0; e < N; e += 2) split_pack(y[e] * f, y[e + 1] * f, hi[e / 2], lo[e / 2]);
+      if (N == 4) {
+        *reinterpret_cast<uint2*>(hi_tile + off) = make_uint2(hi[0], hi[N / 2 - 1]);
+        *reinterpret_cast<uint2*>(lo_tile + off) = make_uint2(lo[0], lo[N / 2 - 1]);
+      } else {
+        *reinterpret_cast<uint32_t*>(hi_tile + off) = hi[0];
+        *reinterpret_cast<uint32_t*>(lo_tile + off) = lo[0];
+      }
+    };
+    conv_rows<N>(p, rq, ring_b, C, static_cast<const bf16*>(p.conv_q) + static_cast<long long>(cq) * p.taps, cq, tw, pos0,
+                 [&](int i, float (&y)[N]) { unit_row(i, y, p.q_scale, smem + SM::Q_HI, smem + SM::Q_LO); });
+    conv_rows<N>(p, rk, ring_b, C, static_cast<const bf16*>(p.conv_k) + static_cast<long long>(cq) * p.taps, p.G * DK + cq, tw,
+                 pos0, [&](int i, float (&y)[N]) { unit_row(i, y, 1.f, smem + SM::K_HI, smem + SM::K_LO); });
+    conv_rows<NV>(p, rv, ring_b, C, static_cast<const bf16*>(p.conv_v) + static_cast<long long>(cv) * p.taps,
+                  2 * p.G * DK + cv, tw, pos0, [&](int i, float (&y)[NV]) {
+                    float* dst = sV + (warp * 8 + i) * DV + lane * NV;
+                    if (NV == 4) store4(dst, make_float4(y[0], y[1], y[2 % NV], y[3 % NV]));
+                    else *reinterpret_cast<float2*>(dst) = make_float2(y[0], y[1]);
                   });
     __syncthreads();
     if (write) {  // the four tiles are contiguous and already have the image's layout
@@ -221,12 +245,12 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
 #pragma unroll
       for (int np = 0; np < 4; ++np) {
         if (np > mt) continue;
-        uint32_t bh[4], bl[4];
+        uint32_t bh[1][4], bl[1][4];
         const int br = np * 16 + (mat >> 1) * 8 + rr, bp = 2 * ks + (mat & 1);
-        ldmatrix_x4(bh, piece(b_hi, br, bp, DK));
-        ldmatrix_x4(bl, piece(b_lo, br, bp, DK));
-        mma_split(acc[np][0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-        mma_split(acc[np][1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        ldmatrix_x4(bh[0], piece(b_hi, br, bp, DK));
+        ldmatrix_x4(bl[0], piece(b_lo, br, bp, DK));
+        float(*const d[2])[4] = {&acc[np][0], &acc[np][1]};
+        mma_split<1>(d, ah, al, bh, bl);
       }
     }
 #pragma unroll
@@ -261,17 +285,16 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
     const bool is_w = tid < DK;
     const int col = is_w ? tid : tid - DK;
     float x[CH];
+    if (is_w) {
 #pragma unroll
-    for (int i = 0; i < CH; ++i) {
-      float r;
-      if (is_w) {
+      for (int i = 0; i < CH; ++i) {
         const uint32_t off = tile_off(i, col, DK);
-        r = -(to_f(*reinterpret_cast<const bf16*>(smem + SM::K_HI + off)) +
-              to_f(*reinterpret_cast<const bf16*>(smem + SM::K_LO + off))) * expf(sCs[i]);
-      } else {
-        r = sV[i * DV + col];
+        x[i] = sBc[i] * (to_f(*reinterpret_cast<const bf16*>(smem + SM::K_HI + off)) +
+                         to_f(*reinterpret_cast<const bf16*>(smem + SM::K_LO + off)));
       }
-      x[i] = r * sBeta[i];
+    } else {
+#pragma unroll
+      for (int i = 0; i < CH; ++i) x[i] = sBeta[i] * sV[i * DV + col];
     }
 #pragma unroll
     for (int i = 1; i < CH; ++i) {
@@ -393,15 +416,13 @@ __global__ void __launch_bounds__(NW * 32) delta_chunk_scan_kernel(const Params 
 #pragma unroll
       for (int np = 0; np < 4; ++np) {
         const int row = np * 16 + (mat >> 1) * 8 + rr, pc = 2 * ks + (mat & 1);
-        uint32_t bh_[4], bl_[4];
-        ldmatrix_x4(bh_, piece(smem + SM::W, row, pc, DK));
-        ldmatrix_x4(bl_, piece(smem + SM::W + SM::T, row, pc, DK));
-        mma_split(U[2 * np], ah, al, bh_[0], bh_[1], bl_[0], bl_[1]);
-        mma_split(U[2 * np + 1], ah, al, bh_[2], bh_[3], bl_[2], bl_[3]);
-        ldmatrix_x4(bh_, piece(smem + SM::Q, row, pc, DK));
-        ldmatrix_x4(bl_, piece(smem + SM::Q + SM::T, row, pc, DK));
-        mma_split(O[2 * np], ah, al, bh_[0], bh_[1], bl_[0], bl_[1]);
-        mma_split(O[2 * np + 1], ah, al, bh_[2], bh_[3], bl_[2], bl_[3]);
+        uint32_t bhi[2][4], blo[2][4];
+        ldmatrix_x4(bhi[0], piece(smem + SM::W, row, pc, DK));
+        ldmatrix_x4(blo[0], piece(smem + SM::W + SM::T, row, pc, DK));
+        ldmatrix_x4(bhi[1], piece(smem + SM::Q, row, pc, DK));
+        ldmatrix_x4(blo[1], piece(smem + SM::Q + SM::T, row, pc, DK));
+        float(*const d[4])[4] = {&U[2 * np], &U[2 * np + 1], &O[2 * np], &O[2 * np + 1]};
+        mma_split<2>(d, ah, al, bhi, blo);
       }
     }
     ok = __syncthreads_and(ok);
@@ -425,11 +446,11 @@ __global__ void __launch_bounds__(NW * 32) delta_chunk_scan_kernel(const Params 
 #pragma unroll
       for (int np = ks; np < 4; ++np) {  // tokens before this block of writes do not see it
         const int row = np * 16 + (mat >> 1) * 8 + rr, pc = 2 * ks + (mat & 1);
-        uint32_t bh_[4], bl_[4];
-        ldmatrix_x4(bh_, piece(smem + SM::M, row, pc, CH));
-        ldmatrix_x4(bl_, piece(smem + SM::M + M_TILE, row, pc, CH));
-        mma_split(O[2 * np], ah, al, bh_[0], bh_[1], bl_[0], bl_[1]);
-        mma_split(O[2 * np + 1], ah, al, bh_[2], bh_[3], bl_[2], bl_[3]);
+        uint32_t bhi[1][4], blo[1][4];
+        ldmatrix_x4(bhi[0], piece(smem + SM::M, row, pc, CH));
+        ldmatrix_x4(blo[0], piece(smem + SM::M + M_TILE, row, pc, CH));
+        float(*const d[2])[4] = {&O[2 * np], &O[2 * np + 1]};
+        mma_split<1>(d, ah, al, bhi, blo);
       }
     }
     ok = __syncthreads_and(ok);
@@ -467,13 +488,16 @@ __global__ void __launch_bounds__(NW * 32) delta_chunk_scan_kernel(const Params 
       uint32_t ah[4], al[4];
       split_a_frag(U[2 * ks], U[2 * ks + 1], ah, al);
 #pragma unroll
-      for (int np = 0; np < NS / 2; ++np) {
+      for (int np = 0; np < NS / 2; np += 2) {
         const int row = ks * 16 + (mat & 1) * 8 + rr, pc = 2 * np + (mat >> 1);
-        uint32_t bh_[4], bl_[4];
-        ldmatrix_x4_trans(bh_, piece(smem + SM::K, row, pc, DK));
-        ldmatrix_x4_trans(bl_, piece(smem + SM::K + SM::T, row, pc, DK));
-        mma_split(S[2 * np], ah, al, bh_[0], bh_[1], bl_[0], bl_[1]);
-        mma_split(S[2 * np + 1], ah, al, bh_[2], bh_[3], bl_[2], bl_[3]);
+        uint32_t bhi[2][4], blo[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          ldmatrix_x4_trans(bhi[i], piece(smem + SM::K, row, pc + 2 * i, DK));
+          ldmatrix_x4_trans(blo[i], piece(smem + SM::K + SM::T, row, pc + 2 * i, DK));
+        }
+        float(*const d[4])[4] = {&S[2 * np], &S[2 * np + 1], &S[2 * np + 2], &S[2 * np + 3]};
+        mma_split<2>(d, ah, al, bhi, blo);
       }
     }
     ok = __syncthreads_and(ok);

@@ -153,7 +153,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const Params p) {
 }
 
 // one warp per (row, head): out = o / rms(o) * norm_w * silu(gate)
-template <typename T>
+// VEC: four values per lane and access (everything starts at multiples of four elements)
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(128) delta_out_kernel(const Params p) {
   const long long unit = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -162,12 +163,27 @@ __global__ void __launch_bounds__(128) delta_out_kernel(const Params p) {
   const int h = static_cast<int>(unit - row * p.H);
   const float* o = p.o + unit * p.dv;
   float ss = 0.f;
-  for (int i = lane; i < p.dv; i += 32) ss += o[i] * o[i];
+  if (VEC)
+    for (int i = lane * 4; i < p.dv; i += 128) {
+      const float4 x = load4(o + i);
+      ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+  else
+    for (int i = lane; i < p.dv; i += 32) ss += o[i] * o[i];
   const float rs = 1.f / sqrtf(sum_warp(ss) / p.dv + p.eps);
   const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.off_g + h * p.dv;
   T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dv;
-  for (int i = lane; i < p.dv; i += 32)
-    from_f(out[i], o[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
+  const T* w = static_cast<const T*>(p.norm_w);
+  constexpr bool fast = sizeof(T) == 2;
+  auto f = [&](float x, float wt, float gt) { return x * rs * wt * (fast ? silu_fast(gt) : silu_f(gt)); };
+  if (VEC) {
+    for (int i = lane * 4; i < p.dv; i += 128) {
+      const float4 x = load4(o + i), wt = load4(w + i), gt = load4(gate + i);
+      store4(out + i, make_float4(f(x.x, wt.x, gt.x), f(x.y, wt.y, gt.y), f(x.z, wt.z, gt.z), f(x.w, wt.w, gt.w)));
+    }
+  } else {
+    for (int i = lane; i < p.dv; i += 32) from_f(out[i], f(o[i], to_f(w[i]), to_f(gate[i])));
+  }
 }
 
 // One token per sequence: grid (H, B). The convolution ring is only read at the rows of earlier tokens and only written
@@ -310,7 +326,12 @@ int launch_scan(const Params& p, cudaStream_t s) {
 
 template <typename T>
 int launch_out(const Params& p, cudaStream_t s) {
-  delta_out_kernel<T><<<(p.B * p.T * p.H + 3) / 4, 128, 0, s>>>(p);
+  const int blocks = (p.B * p.T * p.H + 3) / 4;
+  if (p.dv % 4 == 0 && p.ldo % 4 == 0 && p.ldp % 4 == 0 && p.off_g % 4 == 0 && !((reinterpret_cast<uintptr_t>(p.out) |
+      reinterpret_cast<uintptr_t>(p.proj) | reinterpret_cast<uintptr_t>(p.norm_w) | reinterpret_cast<uintptr_t>(p.o)) & 15))
+    delta_out_kernel<T, true><<<blocks, 128, 0, s>>>(p);
+  else
+    delta_out_kernel<T, false><<<blocks, 128, 0, s>>>(p);
   return check_launch("delta_out_kernel");
 }
 

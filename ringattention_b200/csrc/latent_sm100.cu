@@ -8,37 +8,12 @@
 //   latent_merge_kernel  : merge of the splits, attention sink, value projection, per-head output gate
 // A cached row is [c, padded to a multiple of 8 | rotated key, padded to a multiple of 8] in the engine's storage type.
 // Everything between the stored operands and the stored output is fp32.
-#include "common/bounds.cuh"
-#include "common/host_util.h"
-#include "common/numeric.cuh"
+#include "latent_common.cuh"
 
 RA_BOUNDS_TRANSLATION_UNIT()
 
 namespace ra {
 namespace latent {
-
-struct Params {
-  int B, T, H, dn, dr, dv, r;  // T tokens per sequence in this step; row b * T + t
-  int r_pad, row_w;            // columns before the rotated key in a cached row, columns of a cached row
-  int rot_dims;                // leading dimensions of the rotated part that turn
-  void* proj;                  // (rows, ldp): q heads at off_q (dn + dr each), [c | k_rot] at off_c, gates at off_g
-  long long ldp;
-  int off_q, off_c, off_g;
-  const void* c_norm;          // (r)
-  const float* inv_freq;       // (rot_dims / 2)
-  void* cache;                 // (B, S_max, row_w)
-  long long S_max;
-  const void *w_uk, *w_uv;     // (H * dn, ldw), (H * dv, ldw)
-  long long ldw;
-  const float* sink;           // (H), or null
-  float* q_lat;                // (rows, H, row_w)
-  float *o_part, *lse_part;    // (rows, H, splits, r), (rows, H, splits)
-  int splits;
-  void* out;                   // (rows, ldo)
-  long long ldo;
-  float eps, scale;
-  const long long* pos;        // position of the step's first token
-};
 
 // grid (rows): the row's latent and keys go to the cache, its queries are rotated in place
 template <typename T>
@@ -47,38 +22,12 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const Params p) {
   const long long row = blockIdx.x;
   const int b = blockIdx.x / p.T, t = blockIdx.x - b * p.T;
   const long long pos = *p.pos + t;
-  T* proj = static_cast<T*>(p.proj) + row * p.ldp;
-  const T* c = proj + p.off_c;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < p.r; i += 128) {
-    const float x = to_f(c[i]);
-    ss += x * x;
-  }
-  const float rs = 1.f / sqrtf(sum_block(ss, red) / p.r + p.eps);
-  const bool store = pos < p.S_max && RA_IN_BOUNDS(pos, 1, p.S_max, kTagDecodeCacheRow);
-  T* dst = static_cast<T*>(p.cache) + (b * p.S_max + (store ? pos : 0)) * p.row_w;
-  if (store) {
-    for (int i = threadIdx.x; i < p.r_pad; i += 128)
-      from_f(dst[i], i < p.r ? to_f(c[i]) * rs * to_f(static_cast<const T*>(p.c_norm)[i]) : 0.f);
-    for (int i = p.r_pad + p.dr + threadIdx.x; i < p.row_w; i += 128) from_f(dst[i], 0.f);
-  }
-  // unit 0: the shared key part (from the projection to the cache); unit 1 + h: query head h, in place
+  append_row<T>(p, row, b, pos, red);
   const int pairs = (p.dr + 1) / 2;
-  for (int i = threadIdx.x; i < (p.H + 1) * pairs; i += 128) {
-    const int unit = i / pairs, j = i - unit * pairs;
-    T* src = unit == 0 ? proj + p.off_c + p.r : proj + p.off_q + (unit - 1) * (p.dn + p.dr) + p.dn;
-    float u = to_f(src[2 * j]), v = 2 * j + 1 < p.dr ? to_f(src[2 * j + 1]) : 0.f;
-    if (2 * j + 1 < p.rot_dims) {
-      float sn, cs;
-      sincosf(static_cast<float>(pos) * p.inv_freq[j], &sn, &cs);
-      const float u2 = u * cs - v * sn;
-      v = v * cs + u * sn;
-      u = u2;
-    }
-    T* to = unit == 0 ? dst + p.r_pad : src;
-    if (unit == 0 && !store) continue;
-    from_f(to[2 * j], u);
-    if (2 * j + 1 < p.dr) from_f(to[2 * j + 1], v);
+  for (int i = threadIdx.x; i < p.H * pairs; i += 128) {
+    const int h = i / pairs, j = i - h * pairs;
+    T* q = static_cast<T*>(p.proj) + row * p.ldp + p.off_q + h * (p.dn + p.dr) + p.dn;
+    rotate_pair(p, q, q, j, pos);
   }
 }
 
@@ -100,7 +49,7 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const Params p) {
   } else if (c >= p.r_pad && c < p.r_pad + p.dr) {
     a = to_f(q[p.dn + c - p.r_pad]);
   }
-  p.q_lat[(row * p.H + h) * p.row_w + c] = a;
+  static_cast<float*>(p.q_lat)[(row * p.H + h) * p.row_w + c] = a;
 }
 
 constexpr int ATT_WARPS = 8;
@@ -118,7 +67,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) latent_attend_kernel(const Par
   if (n > p.S_max) n = p.S_max;
   const long long per = (n + p.splits - 1) / p.splits;
   const long long r0 = split * per, r1 = min(n, r0 + per);
-  const float* ql = p.q_lat + (row * p.H + h) * p.row_w;
+  const float* ql = static_cast<const float*>(p.q_lat) + (row * p.H + h) * p.row_w;
   float q[NV], acc[NV];
 #pragma unroll
   for (int j = 0; j < NV; ++j) {

@@ -101,7 +101,28 @@ class _LatentParams(ctypes.Structure):
                 ("c_norm", c_vp), ("inv_freq", c_vp), ("cache", c_vp), ("S_max", c_ll),
                 ("w_uk", c_vp), ("w_uv", c_vp), ("ldw", c_ll), ("sink", c_vp),
                 ("q_lat", c_vp), ("o_part", c_vp), ("lse_part", c_vp), ("splits", c_i),
-                ("out", c_vp), ("ldo", c_ll), ("eps", c_f), ("scale", c_f), ("pos", c_vp)]
+                ("out", c_vp), ("ldo", c_ll), ("eps", c_f), ("scale", c_f), ("pos", c_vp), ("status", c_vp)]
+
+
+def latent_few_fits(m, proj, cache, w) -> bool:
+    """Sizes the tensor-core kernels for few tokens take."""
+    return (proj.dtype == torch.bfloat16 and m.kv_rank % 16 == 0 and m.kv_rank <= 512 and cache.shape[2] % 16 == 0
+            and cache.shape[2] <= 576 and m.rot_dim % 2 == 0 and 1 <= m.dim <= 1024 and w["uk"].stride(0) % 8 == 0
+            and w["uk"].data_ptr() % 16 == 0 and w["uv"].data_ptr() % 16 == 0)
+
+
+def _latent_few(a, m, rows: int, B: int, T: int, n_rows: int, dev) -> None:
+    """A step of few tokens on the tensor cores: 16 or 32 (token, head) rows per CTA over a range of the cache."""
+    H = m.heads
+    blocks = (T * H + 15) // 16 if T * H <= 16 else (T * H + 31) // 32
+    tiles = (n_rows + 63) // 64
+    a.splits = max(1, min((tiles + 1) // 2, 148 // (blocks * B)))
+    q_lat = torch.empty(rows, H, a.row_w, device=dev, dtype=torch.bfloat16)
+    o_part = torch.empty(rows, H, a.splits, m.kv_rank, device=dev, dtype=torch.float32)
+    lse = torch.empty(rows, H, a.splits, device=dev, dtype=torch.float32)
+    a.q_lat, a.o_part, a.lse_part, a.status = _p(q_lat), _p(o_part), _p(lse), _lib.status_tensor(dev).data_ptr()
+    for entry in ("ra_latent_few_query", "ra_latent_few_attend", "ra_latent_few_output"):
+        _lib.call(entry, ctypes.byref(a), _lib.stream_ptr())
 
 
 def latent_splits(rows: int, heads: int, n_rows: int) -> int:
@@ -129,8 +150,11 @@ def latent_mixer(proj, out, *, B: int, T: int, m, offs, w, cache, n_rows: int, e
     a.w_uk, a.w_uv, a.ldw, a.sink = _p(w["uk"]), _p(w["uv"]), w["uk"].stride(0), _p(w["sink"])
     a.out, a.ldo, a.eps, a.scale, a.pos = _p(out), out.stride(0), eps, m.scale, _p(pos)
     a.splits, is32 = 1, int(proj.dtype == torch.float32)
+    expand = T >= EXPAND_MIN_TOKENS and two_part_fits(m, proj, out, offs)
+    if not expand and T < EXPAND_MIN_TOKENS and latent_few_fits(m, proj, cache, w):
+        return _latent_few(a, m, rows, B, T, n_rows, proj.device)
     _lib.call("ra_latent_prep", ctypes.byref(a), is32, _lib.stream_ptr())
-    if T >= EXPAND_MIN_TOKENS and two_part_fits(m, proj, out, offs):
+    if expand:
         return _latent_expanded(proj, out, B, T, m, offs, w, cache, n_rows)
     f32 = dict(device=proj.device, dtype=torch.float32)
     a.splits = latent_splits(rows, H, n_rows)

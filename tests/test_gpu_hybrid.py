@@ -252,7 +252,7 @@ def run_latent(m, offs, proj, w, sizes, dtype, eps, ctx):
 
 
 LATENT_SHAPES = [(3, 20, 6, 28, 52), (4, 128, 64, 128, 256), (16, 128, 64, 128, 512), (5, 64, 32, 64, 128), (1, 16, 2, 8, 24),
-                 (2, 48, 16, 96, 80)]
+                 (2, 48, 16, 96, 80), (20, 40, 24, 32, 208), (33, 24, 8, 16, 40), (16, 32, 16, 24, 16)]
 
 
 @pytest.mark.parametrize("dtype", BOTH)
