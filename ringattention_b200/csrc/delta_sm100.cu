@@ -152,9 +152,13 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const Params p) {
     }
 }
 
-// one warp per (row, head): out = o / rms(o) * norm_w * silu(gate)
-// VEC: four values per lane and access (everything starts at multiples of four elements)
-template <typename T, bool VEC>
+// out = o / rms(o) * norm_w * silu(gate) per (row, head)
+template <typename T>
+__device__ __forceinline__ float gate_f(float g) {
+  return sizeof(T) == 2 ? silu_fast(g) : silu_f(g);
+}
+// one warp per (row, head), any sizes
+template <typename T>
 __global__ void __launch_bounds__(128) delta_out_kernel(const Params p) {
   const long long unit = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -163,26 +167,40 @@ __global__ void __launch_bounds__(128) delta_out_kernel(const Params p) {
   const int h = static_cast<int>(unit - row * p.H);
   const float* o = p.o + unit * p.dv;
   float ss = 0.f;
-  if (VEC)
-    for (int i = lane * 4; i < p.dv; i += 128) {
-      const float4 x = load4(o + i);
-      ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
-    }
-  else
-    for (int i = lane; i < p.dv; i += 32) ss += o[i] * o[i];
+  for (int i = lane; i < p.dv; i += 32) ss += o[i] * o[i];
   const float rs = 1.f / sqrtf(sum_warp(ss) / p.dv + p.eps);
   const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.off_g + h * p.dv;
   T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dv;
-  const T* w = static_cast<const T*>(p.norm_w);
-  constexpr bool fast = sizeof(T) == 2;
-  auto f = [&](float x, float wt, float gt) { return x * rs * wt * (fast ? silu_fast(gt) : silu_f(gt)); };
-  if (VEC) {
-    for (int i = lane * 4; i < p.dv; i += 128) {
-      const float4 x = load4(o + i), wt = load4(w + i), gt = load4(gate + i);
-      store4(out + i, make_float4(f(x.x, wt.x, gt.x), f(x.y, wt.y, gt.y), f(x.z, wt.z, gt.z), f(x.w, wt.w, gt.w)));
-    }
-  } else {
-    for (int i = lane; i < p.dv; i += 32) from_f(out[i], f(o[i], to_f(w[i]), to_f(gate[i])));
+  for (int i = lane; i < p.dv; i += 32)
+    from_f(out[i], o[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * gate_f<T>(to_f(gate[i])));
+}
+// dv = 4 * LANES: LANES lanes per (row, head), four values each, and four rows' heads per lane with all loads in flight;
+// everything starts at multiples of four elements
+template <typename T, int LANES>
+__global__ void __launch_bounds__(256) delta_out_vec_kernel(const Params p) {
+  constexpr int UPB = 256 / LANES, UNITS = 4;  // units per CTA and round, rounds
+  const unsigned n = static_cast<unsigned>(p.B) * p.T * p.H, H = p.H;  // below 2^31 (checked by the launcher)
+  const unsigned u0 = blockIdx.x * (UPB * UNITS) + threadIdx.x / LANES;
+  const int i = (threadIdx.x % LANES) * 4;
+  const float4 w = load4(static_cast<const T*>(p.norm_w) + i);
+  float4 x[UNITS], g[UNITS];
+#pragma unroll
+  for (int k = 0; k < UNITS; ++k) {
+    const unsigned u = min(u0 + k * UPB, n - 1), row = u / H, h = u - row * H;
+    x[k] = load4(p.o + static_cast<long long>(u) * p.dv + i);
+    g[k] = load4(static_cast<const T*>(p.proj) + row * p.ldp + p.off_g + h * p.dv + i);
+  }
+#pragma unroll
+  for (int k = 0; k < UNITS; ++k) {
+    float ss = x[k].x * x[k].x + x[k].y * x[k].y + x[k].z * x[k].z + x[k].w * x[k].w;
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float rs = 1.f / sqrtf(ss / p.dv + p.eps);
+    const unsigned u = u0 + k * UPB, row = u / H, h = u - row * H;
+    if (u < n)
+      store4(static_cast<T*>(p.out) + row * p.ldo + h * p.dv + i,
+             make_float4(x[k].x * rs * w.x * gate_f<T>(g[k].x), x[k].y * rs * w.y * gate_f<T>(g[k].y),
+                         x[k].z * rs * w.z * gate_f<T>(g[k].z), x[k].w * rs * w.w * gate_f<T>(g[k].w)));
   }
 }
 
@@ -326,12 +344,16 @@ int launch_scan(const Params& p, cudaStream_t s) {
 
 template <typename T>
 int launch_out(const Params& p, cudaStream_t s) {
-  const int blocks = (p.B * p.T * p.H + 3) / 4;
-  if (p.dv % 4 == 0 && p.ldo % 4 == 0 && p.ldp % 4 == 0 && p.off_g % 4 == 0 && !((reinterpret_cast<uintptr_t>(p.out) |
-      reinterpret_cast<uintptr_t>(p.proj) | reinterpret_cast<uintptr_t>(p.norm_w) | reinterpret_cast<uintptr_t>(p.o)) & 15))
-    delta_out_kernel<T, true><<<blocks, 128, 0, s>>>(p);
+  const long long n = static_cast<long long>(p.B) * p.T * p.H;
+  const bool vec = (p.dv == 128 || p.dv == 64) && p.ldo % 4 == 0 && p.ldp % 4 == 0 && p.off_g % 4 == 0 &&
+                   !((reinterpret_cast<uintptr_t>(p.out) | reinterpret_cast<uintptr_t>(p.proj) |
+                      reinterpret_cast<uintptr_t>(p.norm_w) | reinterpret_cast<uintptr_t>(p.o)) & 15);
+  if (vec && p.dv == 128)
+    delta_out_vec_kernel<T, 32><<<static_cast<unsigned>((n + 31) / 32), 256, 0, s>>>(p);
+  else if (vec)
+    delta_out_vec_kernel<T, 16><<<static_cast<unsigned>((n + 63) / 64), 256, 0, s>>>(p);
   else
-    delta_out_kernel<T, false><<<blocks, 128, 0, s>>>(p);
+    delta_out_kernel<T><<<static_cast<unsigned>((n + 3) / 4), 128, 0, s>>>(p);
   return check_launch("delta_out_kernel");
 }
 

@@ -12,12 +12,20 @@ namespace resid {
 
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ tokens, const T* __restrict__ table, long long ld_table,
-                             float* __restrict__ x, long long ldx, int d, int vocab) {
+                             float* __restrict__ x, long long ldx, int d, int vocab, bool vec) {
   const long long r = blockIdx.x;
   int tok = tokens[r];
   if (!RA_IN_BOUNDS(tok, 1, vocab, kTagEmbeddingToken)) tok = 0;
   tok = min(max(tok, 0), vocab - 1);
-  for (int i = threadIdx.x; i < ldx; i += blockDim.x) x[r * ldx + i] = i < d ? to_f(table[tok * ld_table + i]) : 0.f;
+  const T* src = table + tok * ld_table;
+  float* dst = x + r * ldx;
+  if (vec) {  // ldx, ld_table multiples of four; the last group may hold padding
+#pragma unroll 4
+    for (int i = threadIdx.x * 4; i + 3 < d; i += blockDim.x * 4) store4(dst + i, load4(src + i));
+    for (int i = (d & ~3) + threadIdx.x; i < ldx; i += blockDim.x) dst[i] = i < d ? to_f(src[i]) : 0.f;
+  } else {
+    for (int i = threadIdx.x; i < ldx; i += blockDim.x) dst[i] = i < d ? to_f(src[i]) : 0.f;
+  }
 }
 
 struct NormParams {
@@ -90,11 +98,13 @@ extern "C" int ra_embed_f32(const int* tokens, const void* table, long long ld_t
     return kHostBadArg;
   }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool vec = ldx % 4 == 0 && ld_table % 4 == 0 &&
+                   !((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(x)) & 15);
   if (f32)
-    resid::embed_kernel<float><<<rows, 256, 0, s>>>(tokens, static_cast<const float*>(table), ld_table, x, ldx, d, vocab);
+    resid::embed_kernel<float><<<rows, 256, 0, s>>>(tokens, static_cast<const float*>(table), ld_table, x, ldx, d, vocab, vec);
   else
     resid::embed_kernel<__nv_bfloat16>
-        <<<rows, 256, 0, s>>>(tokens, static_cast<const __nv_bfloat16*>(table), ld_table, x, ldx, d, vocab);
+        <<<rows, 256, 0, s>>>(tokens, static_cast<const __nv_bfloat16*>(table), ld_table, x, ldx, d, vocab, vec);
   return check_launch("embed_kernel");
 }
 
