@@ -8,11 +8,13 @@
 //                       read-outs of a token (with k and with q) are taken from the decayed state before the write,
 //                       o = S'^T q + (q.k) u, so a token costs one reduction over eight lanes.
 //   delta_out_kernel  : per-head RMS norm of o, gain, silu gate.
-//   delta_step_kernel : all of it for one token per sequence (decode), one CTA per value head.
+//   delta_step_kernel : all of it for one token per sequence (decode), a cluster of four CTAs per value head.
 // The convolution's history is a ring of `taps` rows per sequence, the row of position p at p % taps, kept in fp32: a
 // step reads the rows of the taps - 1 tokens before it and writes the rows of its own last tokens. The state is stored
 // transposed, (dv, dk), so that the eight lanes of a column read 128 contiguous bytes.
 // Everything here is fp32 except the projections that come in.
+#include <cooperative_groups.h>
+
 #include "delta_common.cuh"
 
 RA_BOUNDS_TRANSLATION_UNIT()
@@ -204,40 +206,71 @@ __global__ void __launch_bounds__(256) delta_out_vec_kernel(const Params p) {
   }
 }
 
-// One token per sequence: grid (H, B). The convolution ring is only read at the rows of earlier tokens and only written
-// at the row of this one (taps rows apart), so the CTAs that share a q/k head need no order among themselves.
-constexpr int STEP_THREADS = 512;
+// One token per sequence: grid (4 H, B), clusters of four CTAs per value head. Every CTA takes a quarter of the head's value
+// channels (columns of S; eight lanes per column), starts by loading them, and makes q and k for itself; the sum of squares
+// of o meets through distributed shared memory. The convolution ring is only read at the rows of earlier tokens and only
+// written at the row of this one (taps rows apart), so the CTAs that share a q/k head need no order among themselves.
+constexpr int STEP_THREADS = 256, STEP_CTAS = 4;
+constexpr int STEP_COLS = STEP_THREADS / 8;  // columns per round
 template <typename T, int NJ>
-__global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p) {
+__global__ void __cluster_dims__(STEP_CTAS, 1, 1) __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p) {
   constexpr int DKP = 32 * NJ;
-  extern __shared__ float step_smem[];  // q[DKP], k[DKP], v[dv], o[dv]
+  namespace cg = cooperative_groups;
+  cg::cluster_group cluster = cg::this_cluster();
+  extern __shared__ float step_smem[];  // q[DKP], k[DKP], v[nv], o[nv]
   __shared__ float red[32];
-  __shared__ float scal[4];             // 1 / |q| * scale, 1 / |k|
-  float *sq = step_smem, *sk = sq + DKP, *sv = sk + DKP, *so = sv + p.dv;
-  const int h = blockIdx.x, b = blockIdx.y, kvh = h / (p.H / p.G);
+  __shared__ float scal[4];             // 1 / |q| * scale, 1 / |k|, g, beta
+  __shared__ float sums[STEP_CTAS];
+  const int part = static_cast<int>(cluster.block_rank()), h = blockIdx.x / STEP_CTAS, b = blockIdx.y, kvh = h / (p.H / p.G);
+  const int nv = (p.dv + STEP_CTAS - 1) / STEP_CTAS, v0 = min(p.dv, part * nv), v1 = min(p.dv, v0 + nv);
+  float *sq = step_smem, *sk = sq + DKP, *sv = sk + DKP, *so = sv + nv;
   const int tid = threadIdx.x, l = tid & 7, lane = tid & 31, warp = tid >> 5;
+  float* st = p.state + (static_cast<long long>(b) * p.H + h) * p.dv * p.dk;
+  const bool vec = (p.dk & 3) == 0;
+  float4 S[NJ];
+  auto load_cols = [&](int c0) {
+    const int col = c0 + (tid >> 3);
+    const float* sc = st + static_cast<long long>(col < v1 ? col : 0) * p.dk;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int i = 32 * j + 4 * l, n = col < v1 ? p.dk : 0;
+      if (vec) {
+        S[j] = i < n ? load4(sc + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      } else {
+        S[j].x = i < n ? sc[i] : 0.f;
+        S[j].y = i + 1 < n ? sc[i + 1] : 0.f;
+        S[j].z = i + 2 < n ? sc[i + 2] : 0.f;
+        S[j].w = i + 3 < n ? sc[i + 3] : 0.f;
+      }
+    }
+  };
+  load_cols(v0);
+
   const long long pos = *p.pos;
   const int C = 2 * p.G * p.dk + p.H * p.dv;
   const T* proj_b = static_cast<const T*>(p.proj) + static_cast<long long>(b) * p.ldp;
   float* ring_b = p.ring + static_cast<long long>(b) * p.taps * C;
   float* ring_now = ring_b + static_cast<long long>(ring_slot(pos, p.taps)) * C;
-  const bool first_of_group = h % (p.H / p.G) == 0;
-
-  float* st = p.state + (static_cast<long long>(b) * p.H + h) * p.dv * p.dk;
-  for (int i = tid; i < 2 * DKP + p.dv; i += STEP_THREADS) {
+  const bool first_of_group = part == 0 && h % (p.H / p.G) == 0;
+  for (int i = tid; i < 2 * DKP + (v1 - v0); i += STEP_THREADS) {
     const int kind = i < DKP ? 0 : (i < 2 * DKP ? 1 : 2);
     const int e = kind == 0 ? i : (kind == 1 ? i - DKP : i - 2 * DKP);
     float x = 0.f;
     if (kind == 2 || e < p.dk) {
-      const int nq = p.G * p.dk;
-      const int c = kind == 2 ? 2 * nq + h * p.dv + e : kind * nq + kvh * p.dk + e;
-      const int col = kind == 2 ? p.off_v + h * p.dv + e : (kind == 0 ? p.off_q : p.off_k) + kvh * p.dk + e;
+      const int nq = p.G * p.dk, hv = h * p.dv + v0 + e;
+      const int c = kind == 2 ? 2 * nq + hv : kind * nq + kvh * p.dk + e;
+      const int col = kind == 2 ? p.off_v + hv : (kind == 0 ? p.off_q : p.off_k) + kvh * p.dk + e;
       const T* w = static_cast<const T*>(kind == 0 ? p.conv_q : (kind == 1 ? p.conv_k : p.conv_v)) +
-                   static_cast<long long>(kind == 2 ? h * p.dv + e : kvh * p.dk + e) * p.taps;
+                   static_cast<long long>(kind == 2 ? hv : kvh * p.dk + e) * p.taps;
       x = conv_silu(p, proj_b, ring_b, w, 0, pos, C, c, col);
       if (kind == 2 || first_of_group) ring_now[c] = to_f(proj_b[col]);
     }
     step_smem[i] = x;
+  }
+  if (tid == STEP_THREADS - 1) {
+    const float* ba = p.ba + b * p.ldba;
+    scal[2] = expf(log_decay(ba[p.off_a + h], to_f(static_cast<const T*>(p.a_log)[h]), to_f(static_cast<const T*>(p.dt_bias)[h])));
+    scal[3] = sigmoid_f(ba[h]);
   }
   __syncthreads();
   if (warp < 2) {
@@ -246,10 +279,6 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p
     for (int i = lane; i < DKP; i += 32) ss += s[i] * s[i];
     ss = sum_warp(ss);
     if (lane == 0) scal[warp] = (warp == 0 ? p.q_scale : 1.f) / sqrtf(ss + 1e-6f);
-  } else if (tid == 64) {
-    const float* ba = p.ba + b * p.ldba;
-    scal[2] = expf(log_decay(ba[p.off_a + h], to_f(static_cast<const T*>(p.a_log)[h]), to_f(static_cast<const T*>(p.dt_bias)[h])));
-    scal[3] = sigmoid_f(ba[h]);
   }
   __syncthreads();
   const float qm = scal[0], km = scal[1], g = scal[2], beta = scal[3];
@@ -265,27 +294,14 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p
   }
 #pragma unroll
   for (int o = 4; o > 0; o >>= 1) qk += __shfl_xor_sync(0xffffffffu, qk, o);
-  const bool vec = (p.dk & 3) == 0;
   float ss = 0.f;
   // the trip count is the same for every thread: the shuffles below see whole warps
-  for (int c0 = 0; c0 < p.dv; c0 += STEP_THREADS / 8) {
+  for (int c0 = v0; c0 < v1; c0 += STEP_COLS) {
+    if (c0 > v0) load_cols(c0);
     const int col = c0 + (tid >> 3);
-    const bool in = col < p.dv;
+    const bool in = col < v1;
     float* sc = st + static_cast<long long>(in ? col : 0) * p.dk;
-    float4 S[NJ];
     float a = 0.f, c = 0.f;
-#pragma unroll
-    for (int j = 0; j < NJ; ++j) {
-      const int i = 32 * j + 4 * l;
-      if (vec) {
-        S[j] = (in && i < p.dk) ? load4(sc + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-      } else {
-        S[j].x = (in && i < p.dk) ? sc[i] : 0.f;
-        S[j].y = (in && i + 1 < p.dk) ? sc[i + 1] : 0.f;
-        S[j].z = (in && i + 2 < p.dk) ? sc[i + 2] : 0.f;
-        S[j].w = (in && i + 3 < p.dk) ? sc[i + 3] : 0.f;
-      }
-    }
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
       a += S[j].x * kk[j].x + S[j].y * kk[j].y + S[j].z * kk[j].z + S[j].w * kk[j].w;
@@ -296,7 +312,7 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p
       a += __shfl_xor_sync(0xffffffffu, a, o);
       c += __shfl_xor_sync(0xffffffffu, c, o);
     }
-    const float u = beta * ((in ? sv[col] : 0.f) - g * a);
+    const float u = beta * ((in ? sv[col - v0] : 0.f) - g * a);
     const float ov = fmaf(qk, u, g * c);
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
@@ -314,15 +330,19 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_step_kernel(const Params p
       }
     }
     if (in && l == 0) {
-      so[col] = ov;
+      so[col - v0] = ov;
       ss += ov * ov;
     }
   }
-  const float rs = 1.f / sqrtf(sum_block(ss, red) / p.dv + p.eps);
+  ss = sum_block(ss, red);
+  cluster.sync();  // every CTA of the cluster has started: its shared memory can be written
+  if (tid < STEP_CTAS) cluster.map_shared_rank(sums, tid)[part] = ss;
+  cluster.sync();
+  const float rs = 1.f / sqrtf((sums[0] + sums[1] + sums[2] + sums[3]) / p.dv + p.eps);
   const T* gate = proj_b + p.off_g + h * p.dv;
   T* out = static_cast<T*>(p.out) + b * p.ldo + h * p.dv;
-  for (int i = tid; i < p.dv; i += STEP_THREADS)
-    from_f(out[i], so[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
+  for (int i = v0 + tid; i < v1; i += STEP_THREADS)
+    from_f(out[i], so[i - v0] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
 }
 
 template <typename T>
@@ -359,8 +379,9 @@ int launch_out(const Params& p, cudaStream_t s) {
 
 template <typename T>
 int launch_step(const Params& p, cudaStream_t s) {
-  const dim3 grid(p.H, p.B);
-#define RA_STEP(NJ) delta_step_kernel<T, NJ><<<grid, STEP_THREADS, (64 * NJ + 2 * p.dv) * sizeof(float), s>>>(p)
+  const dim3 grid(STEP_CTAS * p.H, p.B);
+  const int nv = (p.dv + STEP_CTAS - 1) / STEP_CTAS;
+#define RA_STEP(NJ) delta_step_kernel<T, NJ><<<grid, STEP_THREADS, (64 * NJ + 2 * nv) * sizeof(float), s>>>(p)
   if (p.dk <= 32) RA_STEP(1);
   else if (p.dk <= 64) RA_STEP(2);
   else if (p.dk <= 96) RA_STEP(3);

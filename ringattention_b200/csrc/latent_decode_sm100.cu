@@ -6,6 +6,8 @@
 //                          query fragments in registers, the tile's rows divided over the warps; row maxima meet in shared memory;
 //                          P goes through shared memory; O += P C with the latent columns divided over the warps
 //   latent_output_kernel : merge of the splits, sink, value projection, output gate
+#include <cooperative_groups.h>
+
 #include "common/mma_sync.cuh"
 #include "common/sm100.cuh"
 #include "latent_common.cuh"
@@ -17,53 +19,66 @@ namespace latent {
 
 using bf16 = __nv_bfloat16;
 
-// grid (H + 1, rows). Head CTAs: eight latent columns per thread, the head's unrotated dimensions divided over groups of
-// threads, 16-byte weight loads; block H appends the row.
+// grid (H + 1, rows, ceil(r / 128)). Head CTAs take 128 latent columns: eight per thread, the head's unrotated dimensions
+// divided over 32 groups of threads; the first weights are on their way before the query is read. Block H appends the row.
 constexpr int QRY_THREADS = 512;
+constexpr int QRY_COLS = 128;
+constexpr int QRY_GROUPS = QRY_THREADS / (QRY_COLS / 8);
+constexpr int QRY_AHEAD = 4;  // weight rows per thread that are loaded up front
 __global__ void __launch_bounds__(QRY_THREADS) latent_query_kernel(const Params p) {
-  extern __shared__ float qry_smem[];  // q[dn], partial sums [groups][r]
+  extern __shared__ float sq[];  // q[dn]
+  __shared__ __align__(16) float part[QRY_GROUPS][QRY_COLS];
   __shared__ float red[32];
-  const int h = blockIdx.x;
+  const int h = blockIdx.x, c0 = blockIdx.z * QRY_COLS;
   const long long row = blockIdx.y;
   const int b = blockIdx.y / p.T, t = blockIdx.y - b * p.T;
-  const long long pos = *p.pos + t;
   if (h == p.H) {
-    append_row<bf16>(p, row, b, pos, red);
+    if (blockIdx.z == 0) append_row<bf16>(p, row, b, *p.pos + t, red);
     return;
   }
-  float* sq = qry_smem;
-  float* part = qry_smem + ((p.dn + 3) & ~3);
+  const int cg = threadIdx.x % (QRY_COLS / 8), grp = threadIdx.x / (QRY_COLS / 8);
+  const bool in = c0 + cg * 8 < p.r;
+  const bf16* w = static_cast<const bf16*>(p.w_uk) + static_cast<long long>(h) * p.dn * p.ldw + (in ? c0 + cg * 8 : 0);
+  uint4 u[QRY_AHEAD];
+#pragma unroll
+  for (int k = 0; k < QRY_AHEAD; ++k) {
+    const int i = grp + k * QRY_GROUPS;
+    u[k] = i < p.dn ? __ldg(reinterpret_cast<const uint4*>(w + i * p.ldw)) : make_uint4(0u, 0u, 0u, 0u);
+  }
   const bf16* q = static_cast<const bf16*>(p.proj) + row * p.ldp + p.off_q + h * (p.dn + p.dr);
   bf16* dst = static_cast<bf16*>(p.q_lat) + (row * p.H + h) * p.row_w;
   for (int i = threadIdx.x; i < p.dn; i += QRY_THREADS) sq[i] = to_f(q[i]);
-  for (int j = threadIdx.x; j < p.dr / 2; j += QRY_THREADS) rotate_pair(p, q + p.dn, dst + p.r_pad, j, pos);
-  for (int i = p.r_pad + p.dr + threadIdx.x; i < p.row_w; i += QRY_THREADS) dst[i] = __float2bfloat16(0.f);
-  __syncthreads();
-  const int ncg = p.r / 8, groups = QRY_THREADS / ncg;
-  const int cg = threadIdx.x % ncg, grp = threadIdx.x / ncg;
-  if (grp < groups) {
-    float a[8] = {};
-    const bf16* w = static_cast<const bf16*>(p.w_uk) + static_cast<long long>(h) * p.dn * p.ldw + cg * 8;
-#pragma unroll 8
-    for (int i = grp; i < p.dn; i += groups) {
-      const uint4 u = __ldg(reinterpret_cast<const uint4*>(w + i * p.ldw));
-      const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&u);
-      const float x = sq[i];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(b2[e]);
-        a[2 * e] = fmaf(x, f.x, a[2 * e]);
-        a[2 * e + 1] = fmaf(x, f.y, a[2 * e + 1]);
-      }
-    }
-    store4(part + grp * p.r + cg * 8, make_float4(a[0], a[1], a[2], a[3]));
-    store4(part + grp * p.r + cg * 8 + 4, make_float4(a[4], a[5], a[6], a[7]));
+  if (blockIdx.z == 0) {
+    const long long pos = *p.pos + t;
+    for (int j = threadIdx.x; j < p.dr / 2; j += QRY_THREADS) rotate_pair(p, q + p.dn, dst + p.r_pad, j, pos);
+    for (int i = p.r_pad + p.dr + threadIdx.x; i < p.row_w; i += QRY_THREADS) dst[i] = __float2bfloat16(0.f);
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < p.r; c += QRY_THREADS) {
+  float a[8] = {};
+  auto add = [&](int i, const uint4& v) {
+    const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&v);
+    const float x = sq[i];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(b2[e]);
+      a[2 * e] = fmaf(x, f.x, a[2 * e]);
+      a[2 * e + 1] = fmaf(x, f.y, a[2 * e + 1]);
+    }
+  };
+#pragma unroll
+  for (int k = 0; k < QRY_AHEAD; ++k)
+    if (grp + k * QRY_GROUPS < p.dn) add(grp + k * QRY_GROUPS, u[k]);
+  for (int i = grp + QRY_AHEAD * QRY_GROUPS; i < p.dn; i += QRY_GROUPS)
+    add(i, __ldg(reinterpret_cast<const uint4*>(w + i * p.ldw)));
+  store4(&part[grp][cg * 8], make_float4(a[0], a[1], a[2], a[3]));
+  store4(&part[grp][cg * 8 + 4], make_float4(a[4], a[5], a[6], a[7]));
+  __syncthreads();
+  const int c = threadIdx.x;
+  if (c < QRY_COLS && c0 + c < p.r) {
     float s = 0.f;
-    for (int k = 0; k < groups; ++k) s += part[k * p.r + c];
-    dst[c] = __float2bfloat16(s);
+#pragma unroll
+    for (int k = 0; k < QRY_GROUPS; ++k) s += part[k][c];
+    dst[c0 + c] = __float2bfloat16(s);
   }
 }
 
@@ -87,8 +102,9 @@ struct KvSmem {
   static constexpr int TOTAL = BAR + 64 + 1024 /*align*/;
 };
 
-// KS: k-steps of 16 columns that cover a cached row; MT: query tiles of 16 rows per CTA (1 or 2). r <= 16 * KS.
-template <int KS, int MT>
+// KS: k-steps of 16 columns that cover a cached row; MT: query tiles of 16 rows per CTA (1 or 2). r <= 16 * KS. FULL: the
+// latent columns are exactly those of the warps' pairs (no tests in the product loop).
+template <int KS, int MT, bool FULL>
 __global__ void __launch_bounds__(KV_THREADS, 1)
 latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
   using SM = KvSmem<KS>;
@@ -129,18 +145,24 @@ latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
     if (j0 + 1 < j1) fill(j0 + 1);
   }
 
-  // ---- query fragments of this warp's 16 rows
+  // ---- query fragments of this warp's 16 rows, through the third stage's buffer (first filled in the first round)
   uint32_t qa[KS][4];
-#pragma unroll
-  for (int ks = 0; ks < KS; ++ks)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = row0 + mt * 16 + g + 8 * (e & 1), c = ks * 16 + 8 * (e >> 1) + 2 * t;
-      qa[ks][e] = (r < n_q && c < p.row_w)
-                      ? *reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(p.q_lat) +
-                                                           (static_cast<long long>(b) * n_q + r) * p.row_w + c)
-                      : 0u;
+  {
+    uint8_t* sq = smem + 2 * SM::STAGE;  // (16 MT, 64 SLABS) in slabs like a tile
+    constexpr int PIECES = SM::SLABS * 8;
+    const bf16* q = static_cast<const bf16*>(p.q_lat) + static_cast<long long>(b) * n_q * p.row_w;
+    for (int i = tid; i < 16 * MT * PIECES; i += KV_THREADS) {
+      const int r = i / PIECES, pc = i % PIECES;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (row0 + r < n_q && pc * 8 < p.row_w)
+        v = __ldg(reinterpret_cast<const uint4*>(q + static_cast<long long>(row0 + r) * p.row_w + pc * 8));
+      *reinterpret_cast<uint4*>(const_cast<uint8_t*>(slab_piece(sq, r, pc))) = v;
     }
+    __syncthreads();
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) ldmatrix_x4(qa[ks], slab_piece(sq, mt * 16 + (mat & 1) * 8 + rr, 2 * ks + (mat >> 1)));
+    fence_proxy_async_smem();  // these generic accesses before the bulk copy that refills the buffer
+  }
   // last visible row (exclusive) of the two score rows of this thread
   int lim[2];
 #pragma unroll
@@ -230,7 +252,7 @@ latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
           v = fmaxf(v, fmaxf(fmaxf(f.x, f.y), fmaxf(f.z, f.w)));
         }
         const float mu = v == -INFINITY ? 0.f : v;
-        alpha[i][k] = exp2f(m[i][k] - mu);
+        alpha[i][k] = exp2_approx(m[i][k] - mu);
         m[i][k] = v;
       }
     float mrow[2], arow[2];
@@ -245,7 +267,7 @@ latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
     for (int i = 0; i < MT; ++i)
 #pragma unroll
       for (int k = 0; k < 2; ++k) {
-        const float p0 = exp2f(x[i][2 * k] - mrow[k]), p1 = exp2f(x[i][2 * k + 1] - mrow[k]);
+        const float p0 = exp2_approx(x[i][2 * k] - mrow[k]), p1 = exp2_approx(x[i][2 * k + 1] - mrow[k]);
         l[k] += p0 + p1;
         const int row = mt * 16 + g + 8 * k, pc = ng * MT + i;
         *reinterpret_cast<uint32_t*>(sP + row * 128 + ((pc ^ (row & 7)) << 4) + 4 * t) = pack_bf16x2(p0, p1);
@@ -272,7 +294,7 @@ latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
 #pragma unroll
       for (int q = 0; q < PAIRS; ++q) {
         const int pair = warp + 8 * q;
-        if (pair * 16 >= p.r) continue;
+        if (!FULL && pair * 16 >= p.r) continue;
         uint32_t bf[4];
         ldmatrix_x4_trans(bf, slab_piece(tile, ks * 16 + (mat & 1) * 8 + rr, 2 * pair + (mat >> 1)));
 #pragma unroll
@@ -316,18 +338,34 @@ latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
   if (*abort_flag) bounded_drain_pause();
 }
 
-// grid (H, rows): the splits of one head and row, then the head's value projection. r a multiple of 16.
-constexpr int OUT_THREADS = 512;
-__global__ void __launch_bounds__(OUT_THREADS) latent_output_kernel(const Params p) {
-  extern __shared__ float out_smem[];  // weights [splits, padded to 4], partial sums [groups][r]
+// grid (4 H, rows), clusters of four CTAs per head and row. CTA k of a cluster merges the splits of a quarter of the latent
+// columns, hands its quarter to the other three through distributed shared memory, and multiplies a quarter of the head's
+// value projection with the whole; the first weights are on their way meanwhile. r a multiple of 16.
+constexpr int OUT_THREADS = 256, OUT_CTAS = 4, OUT_WARPS = OUT_THREADS / 32;
+constexpr int OUT_MAX_R = 512;
+__global__ void __cluster_dims__(OUT_CTAS, 1, 1) __launch_bounds__(OUT_THREADS) latent_output_kernel(const Params p) {
+  extern __shared__ float sw[];  // weights of the splits
+  __shared__ __align__(16) float o_lat[OUT_MAX_R], part[OUT_THREADS][4];
   __shared__ float red[32];
-  const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  namespace cg = cooperative_groups;
+  cg::cluster_group cluster = cg::this_cluster();
+  const int k = static_cast<int>(cluster.block_rank()), h = blockIdx.x / OUT_CTAS;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long row = blockIdx.y;
-  float* sw = out_smem;
-  float* part = out_smem + ((p.splits + 3) & ~3);
+  // ---- this CTA's rows of the value projection: v0 + warp, + OUT_WARPS, ...; the first two rows of a warp up front
+  const int nv = (p.dv + OUT_CTAS - 1) / OUT_CTAS, v0 = k * nv, v1 = min(p.dv, v0 + nv);
+  const bf16* wv = static_cast<const bf16*>(p.w_uv) + static_cast<long long>(h) * p.dv * p.ldw;
+  constexpr int AHEAD = 4;
+  uint4 u[AHEAD][OUT_MAX_R / 256];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i)
+#pragma unroll
+    for (int j = 0; j < OUT_MAX_R / 256; ++j) {
+      const int v = v0 + warp + i * OUT_WARPS, c = j * 256 + lane * 8;
+      u[i][j] = v < v1 && c < p.r ? __ldg(reinterpret_cast<const uint4*>(wv + v * p.ldw + c)) : make_uint4(0u, 0u, 0u, 0u);
+    }
   const float* lp = p.lse_part + (row * p.H + h) * p.splits;
   const float* op = p.o_part + (row * p.H + h) * p.splits * p.r;
-  const bf16* proj = static_cast<const bf16*>(p.proj) + row * p.ldp;
   float mx = p.sink ? p.sink[h] : -INFINITY;
   for (int s = lane; s < p.splits; s += 32) mx = fmaxf(mx, lp[s]);  // every warp takes them all
 #pragma unroll
@@ -338,50 +376,65 @@ __global__ void __launch_bounds__(OUT_THREADS) latent_output_kernel(const Params
     den += sw[s];
   }
   den = sum_block(den, red) + (p.sink ? expf(p.sink[h] - mx) : 0.f);
-  const float mul = sigmoid_f(to_f(proj[p.off_g + h])) / den;
-  const int nc = p.r / 4, groups = OUT_THREADS / nc, c4 = threadIdx.x % nc, grp = threadIdx.x / nc;
+  const float mul = sigmoid_f(to_f(static_cast<const bf16*>(p.proj)[row * p.ldp + p.off_g + h])) / den;
+  // ---- a quarter of the columns: nc groups of four, the splits divided over the thread groups
+  const int nc = p.r / 16, groups = OUT_THREADS / nc, c4 = threadIdx.x % nc, grp = threadIdx.x / nc;
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
   if (grp < groups) {
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
     for (int s = grp; s < p.splits; s += groups) {
       const float w = sw[s];
-      const float4 v = load4(op + static_cast<long long>(s) * p.r + 4 * c4);
+      const float4 v = load4(op + static_cast<long long>(s) * p.r + k * (p.r / 4) + 4 * c4);
       a.x = fmaf(w, v.x, a.x);
       a.y = fmaf(w, v.y, a.y);
       a.z = fmaf(w, v.z, a.z);
       a.w = fmaf(w, v.w, a.w);
     }
-    store4(part + grp * p.r + 4 * c4, a);
   }
-  __syncthreads();
-  for (int c = threadIdx.x; c < p.r; c += OUT_THREADS) {
+  store4(part[threadIdx.x], a);
+  cluster.sync();  // also: every CTA of the cluster has started, its shared memory can be written
+  for (int c = threadIdx.x; c < p.r / 4; c += OUT_THREADS) {
     float s = 0.f;
-    for (int k = 0; k < groups; ++k) s += part[k * p.r + c];
-    part[c] = s * mul;  // column c of group 0 belongs to this thread alone
-  }
-  __syncthreads();
-  bf16* out = static_cast<bf16*>(p.out) + row * p.ldo + h * p.dv;
-#pragma unroll 4
-  for (int v = warp; v < p.dv; v += OUT_THREADS / 32) {
-    const bf16* w = static_cast<const bf16*>(p.w_uv) + (static_cast<long long>(h) * p.dv + v) * p.ldw;
-    float a = 0.f;
-    for (int c = lane * 8; c < p.r; c += 256) {
-      const uint4 u = __ldg(reinterpret_cast<const uint4*>(w + c));
-      const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+    for (int q = 0; q < groups; ++q) s += part[q * nc + (c >> 2)][c & 3];
+    s *= mul;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(b2[e]);
-        a = fmaf(part[c + 2 * e], f.x, fmaf(part[c + 2 * e + 1], f.y, a));
-      }
+    for (int q = 0; q < OUT_CTAS; ++q) cluster.map_shared_rank(o_lat, q)[k * (p.r / 4) + c] = s;
+  }
+  cluster.sync();
+  bf16* out = static_cast<bf16*>(p.out) + row * p.ldo + h * p.dv;
+  auto dot = [&](const uint4& v, int c) {
+    const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&v);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(b2[e]);
+      s = fmaf(o_lat[c + 2 * e], f.x, fmaf(o_lat[c + 2 * e + 1], f.y, s));
     }
-    a = sum_warp(a);
-    if (lane == 0) out[v] = __float2bfloat16(a);
+    return s;
+  };
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i) {
+    const int v = v0 + warp + i * OUT_WARPS;
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < OUT_MAX_R / 256; ++j) {
+      const int c = j * 256 + lane * 8;
+      if (c < p.r) s += dot(u[i][j], c);
+    }
+    s = sum_warp(s);
+    if (lane == 0 && v < v1) out[v] = __float2bfloat16(s);
+  }
+  for (int v = v0 + warp + AHEAD * OUT_WARPS; v < v1; v += OUT_WARPS) {
+    float s = 0.f;
+    for (int c = lane * 8; c < p.r; c += 256) s += dot(__ldg(reinterpret_cast<const uint4*>(wv + v * p.ldw + c)), c);
+    s = sum_warp(s);
+    if (lane == 0) out[v] = __float2bfloat16(s);
   }
 }
 
 template <int KS, int MT>
 int launch_splitkv(const CUtensorMap& tma, const Params& p, cudaStream_t s) {
-  auto kern = latent_splitkv_kernel<KS, MT>;
+  auto kern = p.r == 512 ? latent_splitkv_kernel<KS, MT, (KS > 32)> : latent_splitkv_kernel<KS, MT, false>;
   constexpr int smem = KvSmem<KS>::TOTAL;
   static_assert(smem <= 227 * 1024, "the tile ring does not fit in shared memory");
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
@@ -414,9 +467,8 @@ extern "C" int ra_latent_few_query(const ra::latent::Params* p, void* stream) {
   using namespace ra::latent;
   const int rc = check_few(p);
   if (rc) return rc;
-  const int groups = QRY_THREADS / (p->r / 8);
-  const int smem = (((p->dn + 3) & ~3) + groups * p->r) * static_cast<int>(sizeof(float));
-  latent_query_kernel<<<dim3(p->H + 1, p->B * p->T), QRY_THREADS, smem, static_cast<cudaStream_t>(stream)>>>(*p);
+  const dim3 grid(p->H + 1, p->B * p->T, (p->r + QRY_COLS - 1) / QRY_COLS);
+  latent_query_kernel<<<grid, QRY_THREADS, p->dn * sizeof(float), static_cast<cudaStream_t>(stream)>>>(*p);
   return ra::check_launch("latent_query_kernel");
 }
 
@@ -441,8 +493,7 @@ extern "C" int ra_latent_few_output(const ra::latent::Params* p, void* stream) {
   using namespace ra::latent;
   const int rc = check_few(p);
   if (rc) return rc;
-  const int groups = OUT_THREADS / (p->r / 4);
-  const int smem = (((p->splits + 3) & ~3) + groups * p->r) * static_cast<int>(sizeof(float));
-  latent_output_kernel<<<dim3(p->H, p->B * p->T), OUT_THREADS, smem, static_cast<cudaStream_t>(stream)>>>(*p);
+  latent_output_kernel<<<dim3(OUT_CTAS * p->H, p->B * p->T), OUT_THREADS, p->splits * sizeof(float),
+                         static_cast<cudaStream_t>(stream)>>>(*p);
   return ra::check_launch("latent_output_kernel");
 }
