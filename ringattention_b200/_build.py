@@ -84,10 +84,31 @@ def _compile_one(src: Path, hdr_digest: str, force: bool, verbose: bool) -> tupl
     return obj, True, log
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile (if stale) and link the kernel library; returns the path of the shared object."""
+def _is_current(src: Path, hdr: str) -> bool:
+    stamp = OBJ_DIR / (src.stem + ".stamp")
+    return ((OBJ_DIR / (src.stem + ".o")).exists() and stamp.exists()
+            and stamp.read_text() == hashlib.sha1(src.read_bytes() + hdr.encode()).hexdigest())
+
+
+def is_current() -> bool:
+    """Whether the whole library is there and up to date."""
+    hdr = _headers_digest()
+    return LIB_PATH.exists() and all(_is_current(s, hdr) for s in sources())
+
+
+def build(force: bool = False, verbose: bool = False, only: "tuple[str, ...] | None" = None) -> Path:
+    """Compile (if stale) and link the kernel library; returns the path of the shared object. ``only``: the stems of the
+    sources one engine needs (the shared host code comes along). Then nothing else is compiled and a library of just
+    those is linked beside the whole one, unless the whole one is up to date already. The objects are shared."""
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
-    srcs = sources()
+    srcs, lib_path = sources(), LIB_PATH
+    if only is not None and (force or not is_current()):
+        missing = set(only) - {p.stem for p in srcs}
+        if missing:
+            raise ValueError(f"no such sources: {sorted(missing)}")
+        srcs = [p for p in srcs if p.stem in only or p.parent != CSRC]
+        tag = hashlib.sha1(" ".join(sorted(only)).encode()).hexdigest()[:8]
+        lib_path = LIB_PATH.with_name(f"{LIB_PATH.stem}_{tag}.so")
     if not srcs:
         raise RuntimeError(f"no CUDA sources under {CSRC}")
     # one builder at a time: the ranks of a job all come through here at start-up
@@ -95,10 +116,10 @@ def build(force: bool = False, verbose: bool = False) -> Path:
 
     with open(OBJ_DIR / ".lock", "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
-        return _build_locked(srcs, force, verbose)
+        return _build_locked(srcs, lib_path, force, verbose)
 
 
-def _build_locked(srcs, force: bool, verbose: bool) -> Path:
+def _build_locked(srcs, lib_path: Path, force: bool, verbose: bool) -> Path:
     hdr = _headers_digest()
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         results = list(ex.map(lambda s: _compile_one(s, hdr, force, verbose), srcs))
@@ -107,13 +128,14 @@ def _build_locked(srcs, force: bool, verbose: bool) -> Path:
         for (_, c, log), s in zip(results, srcs):
             if c:
                 print(f"--- {s.name}\n{log}")
-    if changed or not LIB_PATH.exists():
-        cmd = [_nvcc(), "-shared", "-o", str(LIB_PATH), *[str(o) for o, _, _ in results],
+    newest = max(o.stat().st_mtime for o, _, _ in results)
+    if changed or not lib_path.exists() or lib_path.stat().st_mtime < newest:  # objects may come from another build
+        cmd = [_nvcc(), "-shared", "-o", str(lib_path), *[str(o) for o, _, _ in results],
                "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         if proc.returncode != 0:
             raise RuntimeError(f"link failed:\n{proc.stdout}{proc.stderr}")
-    return LIB_PATH
+    return lib_path
 
 
 def main(argv=None) -> int:

@@ -79,6 +79,10 @@ enum BoundsTag : int {
   kTagDecodeMask = 42,
   kTagSmallMLinear = 43,
   kTagPeerCopy = 50,
+  kTagDelta = 60,
+  kTagDeltaWork = 61,
+  kTagLatent = 62,
+  kTagLatentWork = 63,
 };
 
 }  // namespace ra

@@ -218,7 +218,8 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) delta_chunk_prep_kernel(const
     if (write) {  // the four tiles are contiguous and already have the image's layout
       const uint4* src = reinterpret_cast<const uint4*>(smem);
       uint4* dst = reinterpret_cast<uint4*>(g_qk);
-      for (int i = tid; i < 4 * SM::QK / 16; i += PREP_THREADS) dst[i] = src[i];
+      for (int i = tid; i < 4 * SM::QK / 16; i += PREP_THREADS)
+        if (RA_IN_BOUNDS(chunk, 1, p.n_chunks, kTagDeltaWork)) dst[i] = src[i];
     }
   }
 
@@ -461,7 +462,7 @@ __global__ void __launch_bounds__(NW * 32) delta_chunk_scan_kernel(const Params 
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int tok = c * CH + 8 * j + 2 * t + e;
-        if (tok < p.T) {
+        if (tok < p.T && RA_IN_BOUNDS(v0 + g + 8, 1, p.dv, kTagDelta)) {
           float* dst = p.o + ((static_cast<long long>(b) * p.T + tok) * p.H + h) * p.dv + v0 + g;
           dst[0] = O[j][e];
           dst[8] = O[j][2 + e];

@@ -142,7 +142,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const Params p) {
         S[j][2] = fmaf(kk[j].z, u, g * S[j][2]);
         S[j][3] = fmaf(kk[j].w, u, g * S[j][3]);
       }
-      if (l == 0 && in) p.o[((static_cast<long long>(b) * p.T + t0 + t) * p.H + h) * p.dv + col] = fmaf(qk, u, g * c);
+      if (l == 0 && in && RA_IN_BOUNDS(col, 1, p.dv, kTagDelta)) p.o[((static_cast<long long>(b) * p.T + t0 + t) * p.H + h) * p.dv + col] = fmaf(qk, u, g * c);
     }
   }
 #pragma unroll
@@ -174,7 +174,8 @@ __global__ void __launch_bounds__(128) delta_out_kernel(const Params p) {
   const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.off_g + h * p.dv;
   T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dv;
   for (int i = lane; i < p.dv; i += 32)
-    from_f(out[i], o[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * gate_f<T>(to_f(gate[i])));
+    if (RA_IN_BOUNDS(h * p.dv + i, 1, p.H * p.dv, kTagDelta))
+      from_f(out[i], o[i] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * gate_f<T>(to_f(gate[i])));
 }
 // dv = 4 * LANES: LANES lanes per (row, head), four values each, and four rows' heads per lane with all loads in flight;
 // everything starts at multiples of four elements
@@ -199,7 +200,7 @@ __global__ void __launch_bounds__(256) delta_out_vec_kernel(const Params p) {
     for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const float rs = 1.f / sqrtf(ss / p.dv + p.eps);
     const unsigned u = u0 + k * UPB, row = u / H, h = u - row * H;
-    if (u < n)
+    if (u < n && RA_IN_BOUNDS(h * p.dv + i, 4, p.H * p.dv, kTagDelta))
       store4(static_cast<T*>(p.out) + row * p.ldo + h * p.dv + i,
              make_float4(x[k].x * rs * w.x * gate_f<T>(g[k].x), x[k].y * rs * w.y * gate_f<T>(g[k].y),
                          x[k].z * rs * w.z * gate_f<T>(g[k].z), x[k].w * rs * w.w * gate_f<T>(g[k].w)));
@@ -342,7 +343,7 @@ __global__ void __cluster_dims__(STEP_CTAS, 1, 1) __launch_bounds__(STEP_THREADS
   const T* gate = proj_b + p.off_g + h * p.dv;
   T* out = static_cast<T*>(p.out) + b * p.ldo + h * p.dv;
   for (int i = v0 + tid; i < v1; i += STEP_THREADS)
-    from_f(out[i], so[i - v0] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
+    if (RA_IN_BOUNDS(h * p.dv + i, 1, p.H * p.dv, kTagDelta)) from_f(out[i], so[i - v0] * rs * to_f(static_cast<const T*>(p.norm_w)[i]) * silu_f(to_f(gate[i])));
 }
 
 template <typename T>

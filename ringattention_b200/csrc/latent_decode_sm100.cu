@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(QRY_THREADS) latent_query_kernel(const Params 
     float s = 0.f;
 #pragma unroll
     for (int k = 0; k < QRY_GROUPS; ++k) s += part[k][c];
-    dst[c0 + c] = __float2bfloat16(s);
+    if (RA_IN_BOUNDS(c0 + c, 1, p.row_w, kTagLatentWork)) dst[c0 + c] = __float2bfloat16(s);
   }
 }
 
@@ -328,7 +328,7 @@ latent_splitkv_kernel(const __grid_constant__ CUtensorMap tma, const Params p) {
 #pragma unroll
       for (int q = 0; q < PAIRS; ++q) {
         const int c = (warp + 8 * q) * 16 + 2 * t;
-        if (c >= p.r) continue;
+        if (c >= p.r || !RA_IN_BOUNDS(pi * p.r + c, 10, static_cast<long long>(p.B) * n_q * p.splits * p.r, kTagLatentWork)) continue;
         float* dst = p.o_part + pi * p.r + c;
         *reinterpret_cast<float2*>(dst) = make_float2(o[i][2 * q][2 * k] * inv, o[i][2 * q][2 * k + 1] * inv);
         *reinterpret_cast<float2*>(dst + 8) = make_float2(o[i][2 * q + 1][2 * k] * inv, o[i][2 * q + 1][2 * k + 1] * inv);
@@ -422,13 +422,13 @@ __global__ void __cluster_dims__(OUT_CTAS, 1, 1) __launch_bounds__(OUT_THREADS) 
       if (c < p.r) s += dot(u[i][j], c);
     }
     s = sum_warp(s);
-    if (lane == 0 && v < v1) out[v] = __float2bfloat16(s);
+    if (lane == 0 && v < v1 && RA_IN_BOUNDS(h * p.dv + v, 1, p.H * p.dv, kTagLatent)) out[v] = __float2bfloat16(s);
   }
   for (int v = v0 + warp + AHEAD * OUT_WARPS; v < v1; v += OUT_WARPS) {
     float s = 0.f;
     for (int c = lane * 8; c < p.r; c += 256) s += dot(__ldg(reinterpret_cast<const uint4*>(wv + v * p.ldw + c)), c);
     s = sum_warp(s);
-    if (lane == 0) out[v] = __float2bfloat16(s);
+    if (lane == 0 && RA_IN_BOUNDS(h * p.dv + v, 1, p.H * p.dv, kTagLatent)) out[v] = __float2bfloat16(s);
   }
 }
 

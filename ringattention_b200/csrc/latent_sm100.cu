@@ -116,7 +116,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) latent_attend_kernel(const Par
     float o = 0.f;
 #pragma unroll
     for (int w = 0; w < ATT_WARPS; ++w) o += sm_o[w * p.r + c] * f[w];
-    p.o_part[pi * p.r + c] = lt > 0.f ? o / lt : 0.f;
+    if (RA_IN_BOUNDS(pi * p.r + c, 1, static_cast<long long>(p.B) * p.T * p.H * p.splits * p.r, kTagLatentWork))
+      p.o_part[pi * p.r + c] = lt > 0.f ? o / lt : 0.f;
   }
   if (threadIdx.x == 0) p.lse_part[pi] = lt > 0.f ? mx + logf(lt) : -INFINITY;
 }
@@ -148,7 +149,7 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const Params p) {
     float a = 0.f;
     for (int c = lane; c < p.r; c += 32) a = fmaf(so[c], to_f(w[c]), a);
     a = sum_warp(a);
-    if (lane == 0) from_f(out[v], a);
+    if (lane == 0 && RA_IN_BOUNDS(h * p.dv + v, 1, p.H * p.dv, kTagLatent)) from_f(out[v], a);
   }
 }
 

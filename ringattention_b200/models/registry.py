@@ -18,6 +18,7 @@ class Family:
     named: Callable[..., Any]                       # preset name -> config
     from_dict: Callable[[Mapping[str, Any]], Any]   # config.json -> config
     dtypes: tuple                                   # what the engine computes in
+    sources: tuple                                  # kernel sources the inference engine on one GPU needs
 
 
 def _llama_from_dict(c: Mapping[str, Any]) -> LlamaConfig:
@@ -26,9 +27,12 @@ def _llama_from_dict(c: Mapping[str, Any]) -> LlamaConfig:
 
 
 FAMILIES = {
-    "Llama": Family("llama", LlamaConfig.named, _llama_from_dict, (torch.bfloat16,)),
+    "Llama": Family("llama", LlamaConfig.named, _llama_from_dict, (torch.bfloat16,),
+                    ("attn_fwd_sm100", "decode_sm100", "elementwise", "gemm_sm100")),
     HybridConfig.ARCHITECTURE: Family("dafelorn", HybridConfig.named, HybridConfig.from_dict,
-                                      (torch.bfloat16, torch.float32)),
+                                      (torch.bfloat16, torch.float32),
+                                      ("attn_fwd_sm100", "decode_sm100", "delta_chunk_sm100", "delta_sm100", "gemm_sm100",
+                                       "latent_decode_sm100", "latent_sm100", "linear_f32", "residual_f32")),
 }
 
 

@@ -43,6 +43,16 @@ def available() -> bool:
     return LIB_PATH.exists()
 
 
+_ONLY: "tuple[str, ...] | None" = None
+
+
+def need_only(sources: "tuple[str, ...]") -> None:
+    """Say, before the library is loaded, which sources this process needs: a program that serves one model then compiles
+    no more than that in a fresh checkout. No effect once the library is loaded or when all of it is up to date."""
+    global _ONLY
+    _ONLY = tuple(sources)
+
+
 def lib() -> ctypes.CDLL:
     """Load (once) and return the kernel library. Unless ``RINGATTN_B200_NO_AUTOBUILD=1``, the incremental build
     runs first (it compares source digests and does nothing when the library is current), so that a stale
@@ -62,7 +72,7 @@ def lib() -> ctypes.CDLL:
                 raise KernelError(f"{path} is missing; run python -m ringattention_b200._build")
         else:
             try:
-                _build.build()
+                path = _build.build(only=_ONLY)
             except _build.NvccMissing as e:  # an installed wheel on a machine without the toolkit
                 if not path.exists():
                     raise KernelError(f"cannot build {path}: {e}") from e
@@ -102,7 +112,8 @@ BOUNDS_TAGS = {1: "gemm store", 2: "gemm residual", 10: "attention forward out",
                20: "attention backward dK/dV", 21: "attention backward prep", 30: "rmsnorm", 31: "rope",
                32: "swiglu", 33: "embedding token id", 34: "embedding row", 35: "cross-entropy target",
                36: "cross-entropy row", 37: "adamw", 38: "cast", 39: "mask packing", 40: "decode cache row",
-               41: "decode merge", 42: "decode mask", 43: "small-M linear", 50: "peer copy"}
+               41: "decode merge", 42: "decode mask", 43: "small-M linear", 50: "peer copy", 60: "delta output or state",
+               61: "delta workspace", 62: "latent output", 63: "latent workspace"}
 
 
 def bounds_report(reset: bool = True) -> dict:

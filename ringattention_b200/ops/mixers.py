@@ -151,7 +151,7 @@ def latent_mixer(proj, out, *, B: int, T: int, m, offs, w, cache, n_rows: int, e
     a.out, a.ldo, a.eps, a.scale, a.pos = _p(out), out.stride(0), eps, m.scale, _p(pos)
     a.splits, is32 = 1, int(proj.dtype == torch.float32)
     expand = T >= EXPAND_MIN_TOKENS and two_part_fits(m, proj, out, offs)
-    if not expand and T < EXPAND_MIN_TOKENS and latent_few_fits(m, proj, cache, w):
+    if not expand and latent_few_fits(m, proj, cache, w):
         return _latent_few(a, m, rows, B, T, n_rows, proj.device)
     _lib.call("ra_latent_prep", ctypes.byref(a), is32, _lib.stream_ptr())
     if expand:

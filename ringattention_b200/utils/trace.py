@@ -88,7 +88,7 @@ def main(argv=None) -> int:
     if dtype not in registry.family_of(cfg).dtypes:
         print(f"trace_run: this model does not run in {args.dtype}", file=sys.stderr)
         return 3
-    torch.backends.cuda.matmul.allow_tf32 = False
+    _lib.need_only(registry.family_of(cfg).sources)
     engine = registry.make_engine(cfg, max(1, args.max_tokens), source=registry.checkpoint_source(args.model), dtype=dtype)
     runner = TraceRunner(engine)
     for text in sys.stdin:

@@ -106,6 +106,32 @@ def main():
     qkv = canary((B, 1, 3, H, D), bf, fill=torch.randn(B, 1, 3, H, D, device=dev).to(bf))
     K.rope_append(qkv, ck, cv, torch.tensor([S - 1, 0], device=dev, dtype=torch.int64), 10000.0)
     K.rope_append(qkv, ck, cv, torch.tensor([S + 5, 0], device=dev, dtype=torch.int64), 10000.0)  # not on this shard
+    # ---- hybrid decoders: linear epilogues into row-strided views, and every mixer kernel through whole steps
+    wide = canary((3, 208), bf)
+    K.linear_segments(xs_, ws_[:192].contiguous(), x2=xs_, y=wide[:, :64], y32=canary((3, 32), torch.float32),
+                      ya=wide[:, 80:176], n32_from=64, act_from=96)
+    K.linear_ex(torch.randn(77, 520, device=dev).to(bf), ws_[:192].contiguous(), canary((77, 64), bf),
+                tail=canary((77, 128), torch.float32), n_split=64)
+    K.linear_ex(torch.randn(77, 70, device=dev), torch.randn(51, 70, device=dev), canary((77, 51), torch.float32), relu2=True)
+    import dafelorn_torch as R
+    from hybrid_configs import CONFIGS
+    from ringattention_b200.config import HybridConfig
+    from ringattention_b200.models import registry
+
+    for raw in CONFIGS.values():
+        w = R.random_model(raw, seed=2)
+        for dt in (bf, torch.float32):
+            eng = registry.make_engine(HybridConfig.from_dict(raw), 200, source=w, dtype=dt, batch=2)
+            for c in eng.caches:  # caches and states inside canaries
+                for name in ("data", "state", "ring"):
+                    if hasattr(c, name):
+                        t = getattr(c, name)
+                        setattr(c, name, canary(tuple(t.shape), t.dtype, fill=t))
+            ids = torch.randint(0, raw["vocab"], (2, 200), device=dev)
+            for lo, hi in ((0, 130), (130, 133), (133, 134), (134, 199), (199, 200)):
+                part = ids[:, lo:hi]
+                got = eng.decode_step(part[:, 0])[:, None] if hi - lo == 1 else eng.step(part)
+                assert torch.isfinite(got).all()
     torch.cuda.synchronize()
     _lib.check_status()
     clean = _lib.bounds_report(reset=True)

@@ -21,6 +21,31 @@ def test_build_and_symbols():
 
 
 @pytest.mark.skipif(shutil.which("nvcc") is None, reason="nvcc not installed")
+@pytest.mark.parametrize("family", ["Dafelorn", "Llama"])
+def test_build_of_one_engines_sources(family, tmp_path, monkeypatch):
+    """A library of only the sources an engine names exports what the engine calls and nothing of training."""
+    from ringattention_b200 import _build
+    from ringattention_b200.models import registry
+
+    _build.build()
+    monkeypatch.setattr(_build, "is_current", lambda: False)      # as in a fresh checkout; the objects are reused
+    monkeypatch.setattr(_build, "LIB_PATH", tmp_path / "libpart.so")
+    path = _build.build(only=registry.FAMILIES[family].sources)
+    assert path.parent == tmp_path and path != _build.LIB_PATH
+    lib = ctypes.CDLL(str(path))
+    want = ["ra_last_error", "ra_decode_advance", "ra_small_m_linear", "ra_attn_fwd"]
+    want += (["ra_attn_two_part", "ra_delta_step", "ra_delta_chunk_scan", "ra_latent_few_attend", "ra_latent_prep",
+              "ra_linear_f32", "ra_norm_f32", "ra_embed_f32", "ra_gemm_bf16_ex", "ra_small_m_linear_segments"]
+             if family == "Dafelorn" else ["ra_rmsnorm_fwd", "ra_rope_append", "ra_gemm_bf16_swiglu"])
+    for sym in want:
+        assert hasattr(lib, sym), sym
+    for sym in ("ra_attn_bwd", "ra_adamw" if family == "Dafelorn" else "ra_delta_step"):
+        assert not hasattr(lib, sym), sym
+    with pytest.raises(ValueError, match="no such sources"):
+        _build.build(only=("nothing",))
+
+
+@pytest.mark.skipif(shutil.which("nvcc") is None, reason="nvcc not installed")
 def test_wheel_is_self_contained(tmp_path):
     """A wheel built from the tree, installed elsewhere, carries the kernel sources and the compiled library and
     loads it without the source tree."""
