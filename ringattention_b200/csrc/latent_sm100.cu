@@ -15,20 +15,59 @@ RA_BOUNDS_TRANSLATION_UNIT()
 namespace ra {
 namespace latent {
 
-// grid (rows): the row's latent and keys go to the cache, its queries are rotated in place
-template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(const Params p) {
+// a pair of neighbouring elements (aligned to both), loaded and stored together
+__device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
+  return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+__device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float2 v) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y);
+}
+
+// grid (rows): the row's latent and keys go to the cache, its queries are rotated in place. The sines and cosines of the
+// row's position are made once for all heads; a warp walks heads, its lanes the pairs. PAIRED: every pair starts at an
+// even element.
+constexpr int PREP_THREADS = 128;
+template <typename T, bool PAIRED>
+__global__ void __launch_bounds__(PREP_THREADS, 12) latent_prep_kernel(const Params p) {
+  extern __shared__ float2 turn[];  // (rot_dims / 2) cosine, sine
   __shared__ float red[32];
   const long long row = blockIdx.x;
   const int b = blockIdx.x / p.T, t = blockIdx.x - b * p.T;
   const long long pos = *p.pos + t;
-  append_row<T>(p, row, b, pos, red);
-  const int pairs = (p.dr + 1) / 2;
-  for (int i = threadIdx.x; i < p.H * pairs; i += 128) {
-    const int h = i / pairs, j = i - h * pairs;
-    T* q = static_cast<T*>(p.proj) + row * p.ldp + p.off_q + h * (p.dn + p.dr) + p.dn;
-    rotate_pair(p, q, q, j, pos);
+  const int pairs = p.rot_dims / 2, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, hd = p.dn + p.dr;
+  for (int j = threadIdx.x; j < pairs; j += PREP_THREADS) {
+    float sn, cs;
+    sincosf(static_cast<float>(pos) * p.inv_freq[j], &sn, &cs);
+    turn[j] = make_float2(cs, sn);
   }
+  append_row<T>(p, row, b, pos, red);  // its sums synchronise the CTA
+  T* q0 = static_cast<T*>(p.proj) + row * p.ldp + p.off_q + p.dn;
+  for (int j = lane; j < pairs; j += 32) {
+    const float2 f = turn[j];
+    T* q = q0 + warp * hd + 2 * j;
+#pragma unroll 4
+    for (int h = warp; h < p.H; h += PREP_THREADS / 32, q += (PREP_THREADS / 32) * hd) {
+      const float2 x = PAIRED ? load2(q) : make_float2(to_f(q[0]), to_f(q[1]));
+      const float2 y = make_float2(x.x * f.x - x.y * f.y, x.y * f.x + x.x * f.y);
+      if (PAIRED) {
+        store2(q, y);
+      } else {
+        from_f(q[0], y.x);
+        from_f(q[1], y.y);
+      }
+    }
+  }
+}
+
+template <typename T>
+int launch_prep(const Params& p, cudaStream_t s) {
+  const int smem = (p.rot_dims / 2) * static_cast<int>(sizeof(float2));
+  const bool paired = !((p.dn | p.dr | p.off_q | p.ldp) & 1) && !(reinterpret_cast<uintptr_t>(p.proj) & 7);
+  if (paired) latent_prep_kernel<T, true><<<p.B * p.T, PREP_THREADS, smem, s>>>(p);
+  else latent_prep_kernel<T, false><<<p.B * p.T, PREP_THREADS, smem, s>>>(p);
+  return check_launch("latent_prep_kernel");
 }
 
 // grid (rows, H, ceil(row_w / 128)): one thread per latent column
@@ -182,7 +221,7 @@ int run_absorbed(const Params& p, cudaStream_t s) {
 
 int check(const Params* p) {
   if (p->B < 1 || p->T < 1 || p->H < 1 || p->H > 65535 || p->dn < 0 || p->dr < 0 || p->dv < 1 || p->r < 1 || p->row_w > 1280 ||
-      p->r_pad < p->r || p->row_w < p->r_pad + p->dr || p->rot_dims > p->dr || p->rot_dims % 2 || p->splits < 1 ||
+      p->r_pad < p->r || p->row_w < p->r_pad + p->dr || p->rot_dims > p->dr || p->rot_dims > 4096 || p->rot_dims % 2 || p->splits < 1 ||
       static_cast<long long>(p->B) * p->T > 65535) {
     set_error("ra_latent: bad shape (a cached row has at most 1280 columns, a call at most 65535 rows)");
     return kHostBadArg;
@@ -198,9 +237,7 @@ extern "C" int ra_latent_prep(const ra::latent::Params* p, int f32, void* stream
   int rc = latent::check(p);
   if (rc) return rc;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (f32) latent::latent_prep_kernel<float><<<p->B * p->T, 128, 0, s>>>(*p);
-  else latent::latent_prep_kernel<__nv_bfloat16><<<p->B * p->T, 128, 0, s>>>(*p);
-  return check_launch("latent_prep_kernel");
+  return f32 ? latent::launch_prep<float>(*p, s) : latent::launch_prep<__nv_bfloat16>(*p, s);
 }
 
 // after ra_latent_prep: attention of the step's rows over the cache in the absorbed form
