@@ -23,7 +23,7 @@ sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__.splitlines()[0])
     ap.add_argument("--model", default="llama-7b",
-                    help="a preset (llama-*, dafelorn-*) or a folder with config.json and model.safetensors")
+                    help="a preset (llama-*, dafelorn-*, kalonex-*) or a folder with config.json and model.safetensors")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: hybrid decoders only")
     ap.add_argument("--context", type=int, default=131072, help="tokens of cached context to prefill")
     ap.add_argument("--chunk", type=int, default=32768)
@@ -52,7 +52,7 @@ def main() -> int:
     max_ctx = (args.context + args.new_tokens + 128 * world - 1) // (128 * world) * (128 * world)
     dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}[args.dtype]
     if isinstance(cfg, HybridConfig):
-        kv_gb = args.batch * max_ctx * cfg.cache_bytes_per_token(dtype.itemsize) / 1e9
+        kv_gb = args.batch * cfg.cache_bytes(max_ctx, dtype.itemsize, max_step=8192) / 1e9
     else:
         kv_gb = args.batch * max_ctx / world * 2 * cfg.d_model * 2 * cfg.n_layers / 1e9
     free_gb = torch.cuda.mem_get_info(dev)[0] / 1e9

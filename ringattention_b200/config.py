@@ -250,8 +250,8 @@ class LlamaConfig:
 
 @dataclass(frozen=True)
 class RotaryConfig:
-    """Rotary positions on the first ``dims`` dimensions of a vector, pairs (2i, 2i + 1), frequencies
-    ``base ** (-2i / dims)``."""
+    """Rotary positions on the first ``dims`` dimensions of a vector, frequencies ``base ** (-2i / dims)``. The mixer that
+    uses it fixes the pairs: (2i, 2i + 1) in latent attention, (i, i + dims / 2) in windowed attention."""
 
     base: float
     dims: int
@@ -295,13 +295,62 @@ class GatedDeltaConfig:
 
 
 @dataclass(frozen=True)
+class WindowAttentionConfig:
+    """Attention of ``heads`` query heads over ``kv_heads`` key/value heads (query head h reads head ``h // (heads //
+    kv_heads)``) with biases in the projections, RMS norms over the whole query and key projections, rotary positions on
+    the first dimensions of a head and a learned sink per head. A query sees itself and the ``window - 1`` tokens before it
+    (None: everything before it)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotaryConfig
+    window: Optional[int] = None
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        if self.rot.dims % 2 or not 0 <= self.rot.dims <= self.dim:
+            raise ValueError("rotary dims must be even and at most dim")
+        if self.window is not None and self.window < 1:
+            raise ValueError("a window holds at least the token itself")
+
+
+@dataclass(frozen=True)
 class DenseConfig:
-    """Two-matrix feed-forward ``down(relu(up x)^2)``."""
+    """Feed-forward: ``down(relu(up x)^2)``, or with ``gated`` ``down(silu(gate x) * (up x))``."""
 
     ff: int
+    gated: bool = False
 
 
-MixerConfig = Union[LatentAttentionConfig, GatedDeltaConfig]
+@dataclass(frozen=True)
+class MoEConfig:
+    """Routed experts: of ``experts`` gated feed-forwards of width ``ff`` a token uses the ``top`` with the largest sigmoid
+    scores; the score multiplies the expert's input. A ``shared_ff`` wide one runs for every token (None: there is none)."""
+
+    experts: int
+    top: int
+    ff: int
+    shared_ff: Optional[int] = None
+
+    def __post_init__(self):
+        if not 1 <= self.top <= self.experts:
+            raise ValueError("a token uses at least one and at most all experts")
+
+
+MixerConfig = Union[LatentAttentionConfig, GatedDeltaConfig, WindowAttentionConfig]
+
+
+@dataclass(frozen=True)
+class LoopConfig:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same tensors; every pass has caches of its own."""
+
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
@@ -310,26 +359,74 @@ class LayerConfig:
     the layer whose tensors it uses (its cache or state is its own all the same)."""
 
     mixer: MixerConfig
-    mlp: Optional[DenseConfig] = None
+    mlp: Union[DenseConfig, MoEConfig, None] = None
     weights_of: Optional[int] = None
 
 
 @dataclass(frozen=True)
+class Design:
+    """What an architecture fixes for all its models."""
+
+    norm_gain_offset: float   # 1: norm gains are stored around zero
+    parallel: bool            # mixer and feed-forward read the same stream and are added together; else one after the other
+    gated: bool               # dense feed-forwards are gated
+    mixers: tuple             # mixer types of a config.json
+
+
+DESIGNS = {
+    "Dafelorn": Design(norm_gain_offset=1.0, parallel=True, gated=False, mixers=("latent_attention", "delta")),
+    "Kalonex": Design(norm_gain_offset=0.0, parallel=False, gated=True, mixers=("attention",)),
+}
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer: ``enter`` is the number of the pass that begins with it, None inside a pass or outside
+    the loop."""
+
+    layer: int
+    enter: Optional[int] = None
+
+
+@dataclass(frozen=True)
 class HybridConfig:
-    """Decoder whose layers are listed one by one, each with a mixer of its own kind. Mixer and feed-forward of a layer
-    read the same residual stream through norms of their own and are added to it together (the Dafelorn design)."""
+    """Decoder whose layers are listed one by one, each with a mixer and a feed-forward of its own kind. ``architecture``
+    names the design: in Dafelorn mixer and feed-forward of a layer read the same residual stream and are added to it
+    together; in Kalonex they follow one another, and some layers run several times (``loop``)."""
 
     vocab_size: int
     d_model: int
     layers: tuple
     rms_eps: float
-    norm_gain_offset: float = 1.0     # gains of the layer and final norms are stored around zero
+    architecture: str = "Dafelorn"
+    loop: Optional[LoopConfig] = None
+    logit_scale: float = 1.0
 
-    ARCHITECTURE = "Dafelorn"
+    def __post_init__(self):
+        l = self.loop
+        if l is not None and not (0 <= l.start < l.stop <= len(self.layers) and l.times >= 1):
+            raise ValueError("the loop does not lie within the layers")
+
+    @property
+    def design(self) -> Design:
+        return DESIGNS[self.architecture]
+
+    @property
+    def norm_gain_offset(self) -> float:
+        return self.design.norm_gain_offset
 
     @property
     def n_layers(self) -> int:
         return len(self.layers)
+
+    @property
+    def runs(self) -> tuple:
+        """The layer runs in the order of execution; every run has a cache or state of its own."""
+        l = self.loop
+        if l is None:
+            return tuple(LayerRun(i) for i in range(self.n_layers))
+        looped = [LayerRun(i, t if i == l.start else None) for t in range(l.times) for i in range(l.start, l.stop)]
+        return tuple([LayerRun(i) for i in range(l.start)] + looped + [LayerRun(i) for i in range(l.stop, self.n_layers)])
 
     def owner(self, i: int) -> int:
         """The layer whose tensors layer ``i`` uses."""
@@ -343,47 +440,78 @@ class HybridConfig:
 
     def n_params(self, include_embedding: bool = True) -> int:
         d = self.d_model
-        n = self.vocab_size * d * (2 if include_embedding else 1)
+        n = self.vocab_size * d * (2 if include_embedding else 1) + (2 * d * d if self.loop is not None else 0)
         for i, layer in enumerate(self.layers):
             if self.owner(i) != i:
                 continue
-            m = layer.mixer
+            m, f = layer.mixer, layer.mlp
             if isinstance(m, LatentAttentionConfig):
                 n += d * (m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim + m.heads + m.heads * m.vdim)
                 n += m.kv_rank * m.heads * (m.dim + m.vdim)
+            elif isinstance(m, WindowAttentionConfig):
+                n += d * (m.heads + m.kv_heads) * (m.dim + m.vdim)
             else:
                 n += d * (2 * m.kv_heads * m.dim + 3 * m.heads * m.vdim + 2 * m.heads)
-            if layer.mlp is not None:
-                n += 2 * d * layer.mlp.ff
+            if isinstance(f, MoEConfig):
+                n += d * (f.experts + 3 * f.experts * f.ff + 3 * (f.shared_ff or 0))
+            elif f is not None:
+                n += (3 if f.gated else 2) * d * f.ff
         return n
 
-    def cache_bytes_per_token(self, element_bytes: int = 2) -> int:
-        return sum((l.mixer.kv_rank + l.mixer.rot_dim) * element_bytes for l in self.layers
-                   if isinstance(l.mixer, LatentAttentionConfig))
+    def cache_bytes(self, context: int, element_bytes: int = 2, max_step: int = 1 << 30) -> int:
+        """Bytes that the caches of one sequence of ``context`` tokens take (recurrent states aside)."""
+        n = 0
+        for r in self.runs:
+            m = self.layers[r.layer].mixer
+            if isinstance(m, LatentAttentionConfig):
+                n += context * (m.kv_rank + m.rot_dim)
+            elif isinstance(m, WindowAttentionConfig):
+                rows = context if m.window is None else min(context, m.window + min(max_step, context))
+                n += rows * m.kv_heads * (m.dim + m.vdim)
+        return n * element_bytes
+
+    @staticmethod
+    def _mixer_from_dict(kind: str, m: Mapping[str, Any]) -> MixerConfig:
+        if kind == "latent_attention":
+            return LatentAttentionConfig(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"],
+                                         kv_rank=m["kv_rank"], scale=m["scale"],
+                                         rot=RotaryConfig(base=m["rot"]["base"], dims=m["rot"]["dims"]))
+        if kind == "attention":
+            mask = m.get("mask")
+            return WindowAttentionConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
+                                         scale=m["scale"], rot=RotaryConfig(base=m["rot"]["base"], dims=m["rot"]["dims"]),
+                                         window=None if mask is None else mask["size"])
+        return GatedDeltaConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], conv=m["conv"])
 
     @classmethod
     def from_dict(cls, c: Mapping[str, Any]) -> "HybridConfig":
-        """Parse a ``config.json`` of this design."""
+        """Parse a ``config.json`` of one of the designs."""
+        arch = c.get("architecture", "Dafelorn")
+        design = DESIGNS[arch]
         layers = []
         for i, e in enumerate(c["layers"]):
-            m = e["mixer"]
-            if e["type"] == "latent_attention":
-                mixer = LatentAttentionConfig(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"],
-                                              kv_rank=m["kv_rank"], scale=m["scale"],
-                                              rot=RotaryConfig(base=m["rot"]["base"], dims=m["rot"]["dims"]))
-            elif e["type"] == "delta":
-                mixer = GatedDeltaConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
-                                         conv=m["conv"])
-            else:
+            if e["type"] not in design.mixers:
                 raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
-            mlp = e.get("mlp")
-            if mlp is not None and mlp["kind"] != "dense":
-                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            mixer = cls._mixer_from_dict(e["type"], e["mixer"])
+            f = e.get("mlp")
+            if f is None:
+                mlp = None
+            elif f["kind"] == "dense":
+                mlp = DenseConfig(ff=f["ff"], gated=design.gated)
+            elif f["kind"] == "moe" and design.gated:
+                shared = f.get("shared")
+                mlp = MoEConfig(experts=f["router"]["experts"], top=f["router"]["top"], ff=f["expert"]["ff"],
+                                shared_ff=None if shared is None else shared["ff"])
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
             w = e.get("weights_of")
             if w is not None and not 0 <= w < len(c["layers"]):
                 raise ValueError(f"layer {i}: weights_of {w} is not a layer")
-            layers.append(LayerConfig(mixer, None if mlp is None else DenseConfig(ff=mlp["ff"]), w))
-        out = cls(vocab_size=c["vocab"], d_model=c["width"], layers=tuple(layers), rms_eps=c["norm"]["eps"])
+            layers.append(LayerConfig(mixer, mlp, w))
+        loop = c.get("loop")
+        out = cls(vocab_size=c["vocab"], d_model=c["width"], layers=tuple(layers), rms_eps=c["norm"]["eps"],
+                  architecture=arch, logit_scale=float(c.get("logit_scale", 1.0)),
+                  loop=None if loop is None else LoopConfig(loop["start"], loop["stop"], loop["times"]))
         for i in range(out.n_layers):
             j = out.owner(i)
             if (out.layers[i].mixer, out.layers[i].mlp) != (out.layers[j].mixer, out.layers[j].mlp):
@@ -392,12 +520,24 @@ class HybridConfig:
 
     @classmethod
     def named(cls, name: str, **over) -> "HybridConfig":
-        """Presets of LLaMA-like sizes, three delta layers to one latent-attention layer."""
-        def stack(n, heads, dim, rot, rank, ff, dk):
+        """Presets of LLaMA-like sizes."""
+        def dafelorn(n, heads, dim, rot, rank, ff, dk):
+            """Three delta layers to one latent-attention layer."""
             lat = LatentAttentionConfig(heads=heads, dim=dim, rot_dim=rot, vdim=dim, kv_rank=rank,
                                         scale=(dim + rot) ** -0.5, rot=RotaryConfig(10000.0, rot))
             dl = GatedDeltaConfig(heads=heads, kv_heads=heads // 2, dim=dk, vdim=dk, conv=4)
-            return tuple(LayerConfig(lat if i % 4 == 3 else dl, DenseConfig(ff)) for i in range(n))
+            return dict(layers=tuple(LayerConfig(lat if i % 4 == 3 else dl, DenseConfig(ff)) for i in range(n)))
+
+        def kalonex(n, heads, kv_heads, dim, window, ff, experts, top, expert_ff, shared_ff):
+            """``n`` layer runs: a dense layer, (n - 2) / 2 passes over a routed and a dense layer, a routed layer. The
+            routed layers' active feed-forward (top experts and the shared one) is as wide as the dense one."""
+            if n < 4 or n % 2:
+                raise ValueError("this preset has an even number of layer runs, at least four")
+            at = WindowAttentionConfig(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5,
+                                       rot=RotaryConfig(10000.0, dim // 2), window=window)
+            dense, moe = DenseConfig(ff, gated=True), MoEConfig(experts, top, expert_ff, shared_ff)
+            return dict(layers=tuple(LayerConfig(at, f) for f in (dense, moe, dense, moe)),
+                        loop=LoopConfig(1, 3, (n - 2) // 2))
 
         presets = {
             "dafelorn-7b": dict(vocab_size=32000, d_model=4096, rms_eps=1e-6,
@@ -406,14 +546,24 @@ class HybridConfig:
                                 stack=dict(n=16, heads=16, dim=128, rot=64, rank=512, ff=8256, dk=128)),
             "dafelorn-tiny": dict(vocab_size=1024, d_model=256, rms_eps=1e-6,
                                   stack=dict(n=4, heads=2, dim=64, rot=32, rank=64, ff=768, dk=64)),
+            "kalonex-7b": dict(vocab_size=32000, d_model=4096, rms_eps=1e-6,
+                               stack=dict(n=32, heads=32, kv_heads=8, dim=128, window=4096, ff=11008, experts=64, top=8,
+                                          expert_ff=1152, shared_ff=1792)),
+            "kalonex-1b": dict(vocab_size=32000, d_model=2048, rms_eps=1e-6,
+                               stack=dict(n=16, heads=16, kv_heads=4, dim=128, window=2048, ff=5504, experts=32, top=4,
+                                          expert_ff=1024, shared_ff=1408)),
+            "kalonex-tiny": dict(vocab_size=1024, d_model=256, rms_eps=1e-6,
+                                 stack=dict(n=4, heads=4, kv_heads=2, dim=64, window=128, ff=512, experts=8, top=2,
+                                            expert_ff=128, shared_ff=256)),
         }
         if name not in presets:
             raise KeyError(f"unknown model {name!r}; have {sorted(presets)}")
         kw = dict(presets[name])
+        arch = name.split("-")[0].capitalize()
         st = dict(kw.pop("stack"))
         if "n_layers" in over:
             st["n"] = over.pop("n_layers")
-        kw["layers"] = stack(**st)
+        kw.update({"dafelorn": dafelorn, "kalonex": kalonex}[name.split("-")[0]](**st), architecture=arch)
         kw.update(over)
         return cls(**kw)
 

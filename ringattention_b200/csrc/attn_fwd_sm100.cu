@@ -45,13 +45,24 @@ struct FwdParams {
   long long copy_n16;
   int copy_ctas;
   int* status;
-  // Two-part keys (NR > 0): width of the values that is stored (the tile's columns past it are zero), per-head attention
-  // sink (one more entry exp(sink) in the denominator, without a value), per-head output gate sigmoid(gate[row, h])
+  // EXT: width of the values that is stored (the tile's columns past it are zero), per-head attention sink (one more entry
+  // exp(sink) in the denominator, without a value), per-head output gate sigmoid(gate[row, h])
   int dv;
   const float* sink;            // (H), or null
   const __nv_bfloat16* gate;    // (B * Sq, gate_ld), or null
   long long gate_ld;
+  // EXT: a query sees keys at distances 0 .. window - 1 (0: no limit); kv_share query heads read one key/value head (0 or 1:
+  // each its own); keys and values lie in a ring of k_rows rows (a multiple of 128): key 0 in row k_row0 (0 rows: no ring)
+  int window, kv_share, k_row0, k_rows;
 };
+
+// Window rules for a 128 x 128 tile: some entry lies inside the window; every entry does.
+__device__ __forceinline__ bool tile_in_window(const MaskParams& m, int window, int qi0, int k0) {
+  return !window || m.qmap(qi0) - m.kmap(min(k0 + 127, m.Sk - 1)) < window;
+}
+__device__ __forceinline__ bool tile_window_plain(const MaskParams& m, int window, int qi0, int k0) {
+  return !window || m.qmap(min(qi0 + 127, m.Sq - 1)) - m.kmap(k0) < window;
+}
 
 // NS: 64-wide slabs of the query/key width, DV: value width of the tile. The second K stage is given up where it does not
 // fit beside two tiles of wide queries; V keeps two.
@@ -73,8 +84,9 @@ struct FwdSmem {
 };
 
 // NQ: slabs of the query/key part that every head has of its own; NR: slabs of a second part (maps tma_q2, tma_k2) whose
-// keys all heads share; DV: value width. NR = 0 is plain attention with head dim 64 NQ = DV.
-template <int NQ, int NR, int DV>
+// keys all heads share; DV: value width. EXT adds the options of an inference layer (see FwdParams); without it NR = 0 and
+// the head dim is 64 NQ = DV.
+template <int NQ, int NR, int DV, bool EXT>
 __global__ void __launch_bounds__(FWD_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                 const __grid_constant__ CUtensorMap tma_v, const __grid_constant__ CUtensorMap tma_q2,
@@ -137,8 +149,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
   const int qp = n_qpairs - 1 - (idx - bh * n_qpairs);
   const int h = bh % p.H;
   const int b = bh / p.H;
+  const int h_kv = EXT && p.kv_share > 1 ? h / p.kv_share : h;
   const int q0 = qp * 256;
   const int nk = (mk.Sk + 127) / 128;
+  // row of a key tile (tiles never straddle the end of the ring)
+  auto kv_row = [&](int k0) -> int {
+    if (!EXT || !p.k_rows) return k0;
+    const int r = p.k_row0 + k0;
+    return r >= p.k_rows ? r - p.k_rows : r;
+  };
+  auto visible = [&](int w, int j) -> bool {
+    return tile_visible(mk, b, q0 + w * 128, j * 128) && (!EXT || tile_in_window(mk, p.window, q0 + w * 128, j * 128));
+  };
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -174,13 +196,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
 #pragma unroll
     for (int w = 0; w < 2; ++w)
       fill_visibility(sVis + w * VIS_WORDS, nk, static_cast<int>(threadIdx.x), FWD_THREADS,
-                      [&](int j) { return tile_visible(mk, b, q0 + w * 128, j * 128); });
+                      [&](int j) { return visible(w, j); });
   }
   // next kv tile at or after j that q tile w sees, or nk
   auto next_vis = [&](int w, int j) -> int {
     if (use_vis) return vis_next(sVis + w * VIS_WORDS, j, nk);
     for (; j < nk; ++j)
-      if (tile_visible(mk, b, q0 + w * 128, j * 128)) break;
+      if (visible(w, j)) break;
     return j;
   };
   tc_fence_before();
@@ -214,13 +236,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
 #pragma unroll
         for (int s = 0; s < NSLAB; ++s)
           tma_load_4d(sK + kst * SM::K_TILE_BYTES + s * SM::SLAB_BYTES, s < NQ ? &tma_k : &tma_k2, &k_full[kst],
-                      (s < NQ ? s : s - NQ) * 64, s < NQ ? h : 0, k0, b);
+                      (s < NQ ? s : s - NQ) * 64, s < NQ ? h_kv : 0, kv_row(k0), b);
         if (!mbar_wait_relaxed(&v_empty[st], ph ^ 1u, wc, kTimeoutSmemEmpty)) break;
         mbar_arrive_expect_tx(&v_full[st], SM::V_TILE_BYTES);
 #pragma unroll
         for (int s = 0; s < VSLAB; ++s)
           tma_load_4d(sV + st * SM::V_TILE_BYTES + s * SM::SLAB_BYTES, &tma_v, &v_full[st], s * 64,
-                      h, k0, b);
+                      h_kv, kv_row(k0), b);
         ++it;
       }
     }
@@ -344,7 +366,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
     // every role walks the same visibility mask, so skips stay consistent
     for (int j = next_vis(w, 0); j < nk && alive; j = next_vis(w, j + 1)) {
       const int k0 = j * 128;
-      const bool plain = tile_plain(mk, b, qi0, k0);
+      const bool plain = tile_plain(mk, b, qi0, k0) && (!EXT || tile_window_plain(mk, p.window, qi0, k0));
       if (!plain && (mk.seg_k || mk.bias)) {
         const int buf = cnt & 1;
         const int kc = k0 + wg_tid;
@@ -389,6 +411,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
         for (int c = 0; c < 4; ++c) {
           const int n = limit - 32 * c;
           keep[c] = n >= 32 ? 0xffffffffu : (n <= 0 ? 0u : ((1u << n) - 1u));
+        }
+        if (EXT && p.window) {
+          const int first = qpos - p.window + 1 - mk.kmap(k0);  // columns before it are too far away
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const int n = first - 32 * c;
+            keep[c] &= n >= 32 ? 0u : (n <= 0 ? 0xffffffffu : ~((1u << n) - 1u));
+          }
         }
         if (mk.keep) {
           uint4 kb = make_uint4(0u, 0u, 0u, 0u);
@@ -521,11 +551,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
         lse = mxl + __logf(tot);
       }
     }
-    if ((!NR || p.lse_out) && row_valid &&
+    if ((!EXT || p.lse_out) && row_valid &&
         RA_IN_BOUNDS(lse_idx, 1, static_cast<long long>(p.B) * p.H * mk.Sq, kTagAttnFwdLse))
       p.lse_out[lse_idx] = lse;
     float mul = inv_l * w_this;
-    if (NR && row_valid) {
+    if (EXT && row_valid) {
       if (p.sink) mul /= 1.f + expf(p.sink[h] - lse);
       if (p.gate)
         mul /= 1.f + expf(-__bfloat162float(p.gate[(static_cast<long long>(b) * mk.Sq + qi) * p.gate_ld + h]));
@@ -567,7 +597,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + o_off + c * 32;
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            if (NR && c * 32 + i * 8 >= p.dv) continue;
+            if (EXT && c * 32 + i * 8 >= p.dv) continue;
             uint4 v;
             v.x = pack_bf16x2(f[8 * i], f[8 * i + 1]);
             v.y = pack_bf16x2(f[8 * i + 2], f[8 * i + 3]);
@@ -605,11 +635,11 @@ int make_bshd_map(CUtensorMap* m, const void* base, int B, int S, int H, int D, 
   return ra::make_tmap_bf16_sw128(m, base, 4, dims, str, box);
 }
 
-template <int NQ, int NR, int DV>
+template <int NQ, int NR, int DV, bool EXT = (NR > 0)>
 int launch_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq2,
                const CUtensorMap& tk2, const ra::attn::FwdParams& p, long long grid, cudaStream_t s) {
   using namespace ra::attn;
-  auto kern = attn_fwd_kernel<NQ, NR, DV>;
+  auto kern = attn_fwd_kernel<NQ, NR, DV, EXT>;
   constexpr int smem = FwdSmem<NQ + NR, DV>::TOTAL;
   static_assert(smem <= 227 * 1024, "tile buffers do not fit in shared memory");
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
@@ -704,6 +734,7 @@ extern "C" int ra_attn_fwd(const RaAttnFwdArgs* a) {
   p.sink = nullptr;
   p.gate = nullptr;
   p.gate_ld = 0;
+  p.window = p.kv_share = p.k_row0 = p.k_rows = 0;
   const long long grid = static_cast<long long>((a->Sq + 255) / 256) * a->H * a->B + p.copy_ctas;
   cudaStream_t s = static_cast<cudaStream_t>(a->stream);
   return a->D == 128 ? launch_fwd<2, 0, 128>(tq, tk, tv, tq, tk, p, grid, s)
@@ -774,4 +805,74 @@ extern "C" int ra_attn_two_part(const RaAttnTwoPartArgs* a) {
                       : launch_fwd<2, 1, 64>(tq, tk, tv, tq2, tk2, p, grid, s);
   return a->dv > 64 ? launch_fwd<1, 1, 128>(tq, tk, tv, tq2, tk2, p, grid, s)
                     : launch_fwd<1, 1, 64>(tq, tk, tv, tq2, tk2, p, grid, s);
+}
+
+// Causal attention over the last `window` keys with grouped heads, a sink per head and keys and values in a ring: query i sits
+// at position q_pos0 + i and sees the keys at distances 0 .. window - 1; position j lies in row j % k_rows, k_rows a multiple
+// of 128. Head h reads key/value head h / (H / G). q (B, Sq, H, dk), k (B, k_rows, G, dk), v (B, k_rows, G, dv), out (B, Sq,
+// H, dv): bf16, element strides, innermost contiguous; dk and dv multiples of 8 up to 128. `sink` (H) fp32.
+struct RaAttnWindowArgs {
+  const void* q; long long q_sb, q_ss, q_sh;
+  const void* k; long long k_sb, k_ss, k_sh;
+  const void* v; long long v_sb, v_ss, v_sh;
+  void* out; long long o_sb, o_ss, o_sh;
+  const float* sink;
+  int B, H, G, Sq, dk, dv, window, k_rows;
+  float scale;
+  long long q_pos0;
+  int* status;
+  void* stream;
+};
+
+extern "C" int ra_attn_window(const RaAttnWindowArgs* a) {
+  using namespace ra;
+  using namespace ra::attn;
+  const long long odd = (a->q_sb | a->q_ss | a->q_sh | a->k_sb | a->k_ss | a->k_sh | a->v_sb | a->v_ss | a->v_sh | a->o_sb |
+                         a->o_ss | a->o_sh) & 7;
+  if (a->B < 1 || a->G < 1 || a->H < 1 || a->H % a->G || a->Sq < 1 || a->q_pos0 < 0 || a->window < 1 || a->dk < 8 ||
+      a->dk > 128 || a->dk % 8 || a->dv < 8 || a->dv > 128 || a->dv % 8 || a->k_rows < 128 || a->k_rows % 128 || odd ||
+      ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k) | reinterpret_cast<uintptr_t>(a->v) |
+        reinterpret_cast<uintptr_t>(a->out)) & 15)) {
+    set_error("ra_attn_window: bad shape or alignment");
+    return kHostBadArg;
+  }
+  // the first tile with a visible key; everything below counts keys from there
+  const long long lo = a->q_pos0 - a->window + 1, base = lo > 0 ? lo / 128 * 128 : 0;
+  const long long n_keys = a->q_pos0 + a->Sq - base;
+  if (n_keys > a->k_rows || n_keys > (1 << 30)) {
+    set_error("ra_attn_window: the ring does not hold the window of this step");
+    return kHostBadArg;
+  }
+  CUtensorMap tq, tk, tv;
+  int rc;
+  if ((rc = make_bshd_map(&tq, a->q, a->B, a->Sq, a->H, a->dk, a->q_sb, a->q_ss, a->q_sh))) return rc;
+  if ((rc = make_bshd_map(&tk, a->k, a->B, a->k_rows, a->G, a->dk, a->k_sb, a->k_ss, a->k_sh))) return rc;
+  if ((rc = make_bshd_map(&tv, a->v, a->B, a->k_rows, a->G, a->dv, a->v_sb, a->v_ss, a->v_sh))) return rc;
+  FwdParams p = {};
+  p.B = a->B;
+  p.H = a->H;
+  p.mask.Sq = a->Sq;
+  p.mask.Sk = static_cast<int>(n_keys);
+  p.mask.cbs = 1;
+  p.mask.qmap = PosMap{static_cast<int>(a->q_pos0 - base), 0, 1 << 30};
+  p.mask.kmap = PosMap{0, 0, 1 << 30};
+  p.scale_log2 = a->scale * kLog2e;
+  p.out = a->out;
+  p.o_stride_b = a->o_sb;
+  p.o_stride_s = a->o_ss;
+  p.o_stride_h = a->o_sh;
+  p.status = a->status;
+  p.dv = a->dv;
+  p.sink = a->sink;
+  p.window = a->window;
+  p.kv_share = a->H / a->G;
+  p.k_row0 = static_cast<int>(base % a->k_rows);
+  p.k_rows = a->k_rows;
+  const long long grid = static_cast<long long>((a->Sq + 255) / 256) * a->H * a->B;
+  cudaStream_t s = static_cast<cudaStream_t>(a->stream);
+  if (a->dk > 64)
+    return a->dv > 64 ? launch_fwd<2, 0, 128, true>(tq, tk, tv, tq, tk, p, grid, s)
+                      : launch_fwd<2, 0, 64, true>(tq, tk, tv, tq, tk, p, grid, s);
+  return a->dv > 64 ? launch_fwd<1, 0, 128, true>(tq, tk, tv, tq, tk, p, grid, s)
+                    : launch_fwd<1, 0, 64, true>(tq, tk, tv, tq, tk, p, grid, s);
 }

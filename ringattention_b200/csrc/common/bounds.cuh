@@ -83,6 +83,8 @@ enum BoundsTag : int {
   kTagDeltaWork = 61,
   kTagLatent = 62,
   kTagLatentWork = 63,
+  kTagWindow = 64,
+  kTagMoe = 65,
 };
 
 }  // namespace ra

@@ -24,6 +24,7 @@
 #include "common/bounds.cuh"
 #include "common/host_util.h"
 #include "common/mma_sync.cuh"
+#include "common/numeric.cuh"
 #include "common/sm100.cuh"
 
 RA_BOUNDS_TRANSLATION_UNIT()
@@ -905,7 +906,9 @@ constexpr int LM_STAGE = LM_WTILE + LM_XTILE;
 // Columns of the product fall into up to three segments with outputs of their own (an inference layer's projections in
 // one launch): [0, n32_from) bf16 to y, [n32_from, act_from) fp32 to y32 (added to what is there when `add32`: the 32-bit
 // residual stream), [act_from, N) squared relu in bf16 to ya; the last segment multiplies x2 instead of x (the same rows
-// through another norm). Segment borders are multiples of LM_COLS.
+// through another norm). Segment borders are multiples of LM_COLS. The first two segments are alpha * product + bias.
+// With gated_F > 0 there is one segment: w = [gate | up] (gated_F rows each, a multiple of 8), a CTA takes eight gate columns
+// and the matching up columns, and y gets silu(gate) * up.
 struct LmParams {
   const __nv_bfloat16 *x, *x2;
   long long ldx;
@@ -919,6 +922,9 @@ struct LmParams {
   long long ldya;
   int n32_from, act_from, add32;
   int M, N, K;
+  const float* bias;           // by column of the product, or null
+  float alpha;
+  int gated_F;
 };
 
 __global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const LmParams p) {
@@ -943,7 +949,8 @@ __global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const Lm
       const int row = piece >> 4, ch = piece & 15;
       const int col = col0 + row;
       const bool in = col < N && k0 + ch * 8 < K;
-      const __nv_bfloat16* src = w + static_cast<long long>(in ? col : 0) * K + (in ? k0 + ch * 8 : 0);
+      const int w_row = !p.gated_F ? col : (row < 8 ? 0 : p.gated_F) + (col0 >> 1) + (row & 7);
+      const __nv_bfloat16* src = w + static_cast<long long>(in ? w_row : 0) * K + (in ? k0 + ch * 8 : 0);
       cp_async16(wt + row * (LM_KC * 2) + ((ch ^ (row & 7)) << 4), src, in ? 16 : 0);
     }
 #pragma unroll
@@ -1004,6 +1011,20 @@ __global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const Lm
     red[warp][g][8 * nt + 2 * t + 1] = acc[nt][1];
   }
   __syncthreads();
+  if (p.gated_F) {
+    for (int i = threadIdx.x; i < M * 8; i += LM_THREADS) {
+      const int m = i >> 3, c = i & 7;
+      float gv = 0.f, uv = 0.f;
+#pragma unroll
+      for (int k = 0; k < LM_WARPS; ++k) {
+        gv += red[k][m][c];
+        uv += red[k][m][c + 8];
+      }
+      const int col = (col0 >> 1) + c;
+      if (RA_IN_BOUNDS(col, 1, p.gated_F, kTagSmallMLinear)) p.y[m * p.ldy + col] = __float2bfloat16(silu_fast(gv) * uv);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < M * LM_COLS; i += LM_THREADS) {
     const int m = i / LM_COLS, c = i % LM_COLS;
     if (col0 + c >= N) continue;
@@ -1012,6 +1033,7 @@ __global__ void __launch_bounds__(LM_THREADS) small_m_linear_mma_kernel(const Lm
     for (int k = 0; k < LM_WARPS; ++k) v += red[k][m][c];
     const int col = col0 + c;
     if (!RA_IN_BOUNDS(col, 1, N, kTagSmallMLinear)) continue;
+    if (col0 < p.act_from) v = fmaf(v, p.alpha, p.bias ? p.bias[col] : 0.f);
     if (col0 >= p.act_from) {
       v = fmaxf(v, 0.f);
       p.ya[m * p.ldya + col - p.act_from] = __float2bfloat16(v * v);
@@ -1377,6 +1399,7 @@ extern "C" int ra_small_m_linear_mma(const void* x, const void* w, void* y, cons
   p.res = static_cast<const __nv_bfloat16*>(res);
   p.n32_from = p.act_from = (N + LM_COLS - 1) / LM_COLS * LM_COLS;  // one segment
   p.M = M; p.N = N; p.K = K;
+  p.alpha = 1.f;
   return launch_small_m_mma(p, static_cast<cudaStream_t>(stream));
 }
 
@@ -1384,7 +1407,8 @@ extern "C" int ra_small_m_linear_mma(const void* x, const void* w, void* y, cons
 // of 16 (at least N when a segment is absent); ldx is a multiple of 8.
 extern "C" int ra_small_m_linear_segments(const void* x, const void* x2, long long ldx, const void* w, void* y,
                                           long long ldy, float* y32, long long ldy32, int add32, void* ya,
-                                          long long ldya, int n32_from, int act_from, int M, int N, int K, void* stream) {
+                                          long long ldya, int n32_from, int act_from, int M, int N, int K, const float* bias,
+                                          float alpha, void* stream) {
   using namespace ra::decode;
   if (M < 1 || M > 8 || K % 8 || N < 1 || ldx % 8 || n32_from % LM_COLS || act_from % LM_COLS || n32_from > act_from ||
       (n32_from > 0 && !y) || (n32_from < act_from && n32_from < N && !y32) || (act_from < N && (!ya || !x2)) ||
@@ -1404,6 +1428,29 @@ extern "C" int ra_small_m_linear_segments(const void* x, const void* x2, long lo
   p.ldya = ldya;
   p.n32_from = n32_from; p.act_from = act_from;
   p.M = M; p.N = N; p.K = K;
+  p.bias = bias; p.alpha = alpha;
+  return launch_small_m_mma(p, static_cast<cudaStream_t>(stream));
+}
+
+// y (M, ldy >= F) = silu(x Wg^T) * (x Wu^T) for w = [Wg | Wu] (2 F, K) dense, M <= 8; F and K multiples of 8.
+extern "C" int ra_small_m_linear_gated(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int F,
+                                       int K, void* stream) {
+  using namespace ra::decode;
+  if (M < 1 || M > 8 || K % 8 || F < 8 || F % 8 || ldx % 8 || ldy < F ||
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15)) {
+    set_error("ra_small_m_linear_gated: bad shape");
+    return kHostBadArg;
+  }
+  LmParams p = {};
+  p.x = p.x2 = static_cast<const __nv_bfloat16*>(x);
+  p.ldx = ldx;
+  p.w = static_cast<const __nv_bfloat16*>(w);
+  p.y = static_cast<__nv_bfloat16*>(y);
+  p.ldy = ldy;
+  p.n32_from = p.act_from = 2 * F;
+  p.M = M; p.N = 2 * F; p.K = K;
+  p.alpha = 1.f;
+  p.gated_F = F;
   return launch_small_m_mma(p, static_cast<cudaStream_t>(stream));
 }
 

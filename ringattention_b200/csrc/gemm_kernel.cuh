@@ -40,6 +40,10 @@ struct Params {
   float* C2;  // null = no tail
   long long ldc2;
   int n_split;
+  // Plain K-major products only, before everything else in the epilogue: v = alpha * v + bias[column] (fp32, at least N
+  // entries rounded up to a multiple of 32; null: neither)
+  const float* bias;
+  float alpha;
 };
 
 constexpr int MAX_SHARDS = 8;
@@ -360,6 +364,16 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
         tmem_ld_wait();
         const int col0 = n0 + c * 32;
         if (row < p.M && col0 < p.N) {
+          if (p.bias) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+              const float4 bv = *reinterpret_cast<const float4*>(p.bias + col0 + 4 * j);
+              r[4 * j] = __float_as_uint(fmaf(__uint_as_float(r[4 * j]), p.alpha, bv.x));
+              r[4 * j + 1] = __float_as_uint(fmaf(__uint_as_float(r[4 * j + 1]), p.alpha, bv.y));
+              r[4 * j + 2] = __float_as_uint(fmaf(__uint_as_float(r[4 * j + 2]), p.alpha, bv.z));
+              r[4 * j + 3] = __float_as_uint(fmaf(__uint_as_float(r[4 * j + 3]), p.alpha, bv.w));
+            }
+          }
           if (p.relu2) {
 #pragma unroll
             for (int e = 0; e < 32; ++e) {

@@ -107,17 +107,18 @@ extern "C" int ra_gemm_bf16_swiglu(const void* A, const void* W, void* Hout, int
 }
 
 
-// C[M,N] = act(A B^T (+ R)) with the epilogues of an inference layer: `relu2` squares the positive part (no addend then),
-// `C2` takes the columns [n_split, N) in fp32 (n_split a multiple of 32, N - n_split a multiple of 4). Both operands
+// C[M,N] = act(alpha A B^T + bias (+ R)) with the epilogues of an inference layer: `bias` is fp32 by column, padded to a
+// multiple of 32 entries (null: none, and alpha is not looked at); `relu2` squares the positive part (no addend then), `C2` takes the columns [n_split, N) in fp32 (n_split a multiple of 32, N - n_split a multiple of 4). Both operands
 // K-major; N a multiple of 8 (of 4 with an fp32 C); otherwise the rules of ra_gemm_bf16.
 extern "C" int ra_gemm_bf16_ex(const void* A, const void* B, void* C, const void* R, float* C2, int M, int N, int K,
                                long long lda, long long ldb, long long ldc, long long ldr, long long ldc2, int n_split,
-                               int relu2, int c_fp32, int group_m, int* status, void* stream) {
+                               int relu2, int c_fp32, const float* bias, float alpha, int group_m, int* status,
+                               void* stream) {
   using namespace ra;
   if (M <= 0 || N <= 0 || K <= 0 || (N % (c_fp32 ? 4 : 8)) || (lda % 8) || (ldb % 8) || (ldc % (c_fp32 ? 4 : 8)) ||
       (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) ||
       (reinterpret_cast<uintptr_t>(C) & 15) || (reinterpret_cast<uintptr_t>(R) & 15) ||
-      (reinterpret_cast<uintptr_t>(C2) & 15) || (R && (ldr % (c_fp32 ? 4 : 8))) || (R && relu2) ||
+      (reinterpret_cast<uintptr_t>(C2) & 15) || (reinterpret_cast<uintptr_t>(bias) & 15) || (R && (ldr % (c_fp32 ? 4 : 8))) || (R && relu2) ||
       (C2 && (n_split % 32 || n_split < 0 || n_split >= N || ldc2 % 4 || ldc2 < N - n_split))) {
     set_error("ra_gemm_bf16_ex: bad shape/alignment");
     return kHostBadArg;
@@ -132,6 +133,7 @@ extern "C" int ra_gemm_bf16_ex(const void* A, const void* B, void* C, const void
   dims[1] = N; box[1] = gemm::BN;
   str[0] = static_cast<uint64_t>(ldb) * 2;
   if ((rc = make_tmap_bf16_sw128(&tb, B, 2, dims, str, box)) != 0) return rc;
-  gemm::Params p{C, ldc, M, N, K, c_fp32, R, ldr, group_m > 0 ? group_m : 8, status, 0, relu2, C2, ldc2, n_split};
+  gemm::Params p{C, ldc, M, N, K, c_fp32, R, ldr, group_m > 0 ? group_m : 8, status, 0, relu2, C2, ldc2, n_split,
+                 bias, alpha};
   return gemm::launch<0, 0>(ta, tb, p, static_cast<cudaStream_t>(stream));
 }

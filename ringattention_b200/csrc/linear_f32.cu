@@ -1,5 +1,5 @@
 // Linear layers in true fp32 on the CUDA cores: C[M,N] = A[M,K] * B[N,K]^T with the same epilogues as the bf16 GEMM
-// (addend, squared relu, last columns to a second output). This is the matrix product of the engine's 32-bit mode; it
+// (scale and bias by column, addend, squared relu, last columns to a second output). This is the matrix product of the engine's 32-bit mode; it
 // never rounds an operand. 64 x 64 output tile per CTA, 4 x 4 outputs per thread, K in steps of 16 through shared memory.
 #include "common/bounds.cuh"
 #include "common/host_util.h"
@@ -18,6 +18,8 @@ struct Params {
   int M, N, K;
   int n_split;  // columns from here on go to C2 (N: none)
   int relu2;    // C = max(v, 0)^2
+  const float* bias;  // by column, or null
+  float alpha;        // v = alpha * v + bias
 };
 
 __global__ void __launch_bounds__(THREADS) linear_f32_kernel(const Params p) {
@@ -55,7 +57,8 @@ __global__ void __launch_bounds__(THREADS) linear_f32_kernel(const Params p) {
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= p.N) continue;
-      float v = acc[i][j];
+      float v = acc[i][j] * p.alpha;
+      if (p.bias) v += p.bias[n];
       if (n >= p.n_split) {
         p.C2[m * p.ldc2 + n - p.n_split] = v;
         continue;
@@ -76,13 +79,13 @@ __global__ void __launch_bounds__(THREADS) linear_f32_kernel(const Params p) {
 // R may be C (in-place accumulation). Leading dimensions in elements, no alignment rules.
 extern "C" int ra_linear_f32(const float* A, const float* B, float* C, const float* R, float* C2, int M, int N, int K,
                              long long lda, long long ldb, long long ldc, long long ldr, long long ldc2, int n_split,
-                             int relu2, void* stream) {
+                             int relu2, const float* bias, float alpha, void* stream) {
   using namespace ra;
   if (M < 1 || N < 1 || K < 1 || (n_split < N && !C2)) {
     set_error("ra_linear_f32: bad shape");
     return kHostBadArg;
   }
-  lin32::Params p{A, B, C, R, C2, lda, ldb, ldc, ldr, ldc2, M, N, K, n_split, relu2};
+  lin32::Params p{A, B, C, R, C2, lda, ldb, ldc, ldr, ldc2, M, N, K, n_split, relu2, bias, alpha};
   dim3 grid((N + lin32::TN - 1) / lin32::TN, (M + lin32::TM - 1) / lin32::TM);
   if (grid.y > 65535) {
     set_error("ra_linear_f32: too many rows");

@@ -1,6 +1,8 @@
 // The 32-bit residual stream: embedding lookup into it, and RMS norms out of it. A norm call writes one or two
 // normalised copies of the same rows (a layer whose mixer and feed-forward read the same input through norms of their
-// own needs two) and reads the rows once; gains are stored either as they are or around zero (`gain_offset` 1).
+// own needs two) and reads the rows once; gains are stored either as they are or around zero (`gain_offset` 1). Also the rows
+// that enter a pass over looped layers ([stream | embedding] side by side, one product's input), and the gated activation of
+// fp32 engines.
 #include "common/bounds.cuh"
 #include "common/host_util.h"
 #include "common/numeric.cuh"
@@ -26,6 +28,36 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const T* __restrict
   } else {
     for (int i = threadIdx.x; i < ldx; i += blockDim.x) dst[i] = i < d ? to_f(src[i]) : 0.f;
   }
+}
+
+// out (rows, 2 dp) = [x | table[token]], each half padded with zeros from d on
+template <typename T>
+__global__ void pair_kernel(const int* __restrict__ tokens, const T* __restrict__ table, long long ld_table,
+                            const float* __restrict__ x, long long ldx, T* __restrict__ out, int d, int dp, int vocab) {
+  const long long r = blockIdx.x;
+  const int tok = min(max(tokens[r], 0), vocab - 1);
+  const T* src = table + tok * ld_table;
+  T* dst = out + r * 2 * dp;
+  if (!RA_IN_BOUNDS(tokens[r], 1, vocab, kTagEmbeddingToken)) return;
+  if (ld_table % 4 == 0 && d % 4 == 0) {
+    for (int i = threadIdx.x * 4; i < dp; i += blockDim.x * 4) {
+      const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+      store4(dst + i, i < d ? load4(x + r * ldx + i) : z);
+      store4(dst + dp + i, i < d ? load4(src + i) : z);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < dp; i += blockDim.x) {
+    from_f(dst[i], i < d ? x[r * ldx + i] : 0.f);
+    dst[dp + i] = i < d ? src[i] : T(0.f);
+  }
+}
+
+// y (rows, F) = silu(gu[:, :F]) * gu[:, F:], fp32
+__global__ void gated_act_kernel(const float* __restrict__ gu, float* __restrict__ y, long long ldy, int F) {
+  const long long r = blockIdx.x;
+  for (int i = threadIdx.x; i < F; i += blockDim.x)
+    if (RA_IN_BOUNDS(i, 1, ldy, kTagSwiglu)) y[r * ldy + i] = silu_f(gu[r * 2 * F + i]) * gu[r * 2 * F + F + i];
 }
 
 struct NormParams {
@@ -120,4 +152,34 @@ extern "C" int ra_norm_f32(const float* x, const int* rows_idx, const void* w1, 
   resid::NormParams p{x, rows_idx, w1, w2, y1, y2, ldx, ldy, d, dp, eps, gain_offset};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   return f32 ? resid::launch_norm<float>(p, rows, s) : resid::launch_norm<__nv_bfloat16>(p, rows, s);
+}
+
+// out (rows, 2 dp) = [x | table[token]]: what enters a pass over looped layers. dp a multiple of 8; `f32`: table and out are
+// fp32, else bf16.
+extern "C" int ra_stream_pair(const int* tokens, const void* table, long long ld_table, const float* x, long long ldx,
+                              void* out, int rows, int d, int dp, int vocab, int f32, void* stream) {
+  using namespace ra;
+  if (rows < 1 || d < 1 || vocab < 1 || dp < d || dp % 8 || ldx % 4 || ldx < d || ld_table < d) {
+    set_error("ra_stream_pair: bad shape");
+    return kHostBadArg;
+  }
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (f32)
+    resid::pair_kernel<float><<<rows, 256, 0, s>>>(tokens, static_cast<const float*>(table), ld_table, x, ldx,
+                                                   static_cast<float*>(out), d, dp, vocab);
+  else
+    resid::pair_kernel<__nv_bfloat16><<<rows, 256, 0, s>>>(tokens, static_cast<const __nv_bfloat16*>(table), ld_table, x, ldx,
+                                                           static_cast<__nv_bfloat16*>(out), d, dp, vocab);
+  return check_launch("pair_kernel");
+}
+
+// y (rows, ldy >= F) = silu(gu[:, :F]) * gu[:, F:2F], fp32; gu dense.
+extern "C" int ra_gated_act_f32(const float* gu, float* y, long long ldy, int rows, int F, void* stream) {
+  using namespace ra;
+  if (rows < 1 || F < 1 || ldy < F) {
+    set_error("ra_gated_act_f32: bad shape");
+    return kHostBadArg;
+  }
+  resid::gated_act_kernel<<<rows, 256, 0, static_cast<cudaStream_t>(stream)>>>(gu, y, ldy, F);
+  return check_launch("gated_act_kernel");
 }

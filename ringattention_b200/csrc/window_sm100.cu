@@ -1,0 +1,251 @@
+// Attention over a sliding window with grouped key/value heads, a sink per head, RMS norms over the whole query and key
+// projections and rotary positions on the first dimensions of a head:
+//   window_prep_kernel   : norms, rotation (queries in place) and the new rows of the key/value ring. One CTA per token; in
+//                          16-byte pieces where the sizes allow it.
+//   window_attend_kernel : one warp per (token, head) on the CUDA cores; any sizes, bf16 or fp32 throughout. bf16 prompts of
+//                          the common sizes run on the tensor cores (attn_fwd_sm100.cu), single tokens in
+//                          window_decode_sm100.cu.
+#include "window_common.cuh"
+
+RA_BOUNDS_TRANSLATION_UNIT()
+
+namespace ra {
+namespace window {
+
+constexpr int PREP_THREADS = 256;
+constexpr int MAX_HALF = 256;
+
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&f)[8]) {
+  const float4 a = load4(p), b = load4(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+template <>
+__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 v = __bfloat1622float2(h[i]);
+    f[2 * i] = v.x;
+    f[2 * i + 1] = v.y;
+  }
+}
+__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
+  store4(p, make_float4(f[0], f[1], f[2], f[3]));
+  store4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
+  uint4 u;
+  uint32_t* w = reinterpret_cast<uint32_t*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+    w[i] = *reinterpret_cast<const uint32_t*>(&v);
+  }
+  *reinterpret_cast<uint4*>(p) = u;
+}
+
+// VEC: head sizes and rot_half are multiples of eight.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(PREP_THREADS) window_prep_kernel(const Params p) {
+  __shared__ float red[32], sn[MAX_HALF], cs[MAX_HALF];
+  const long long row = blockIdx.x;
+  const int b = static_cast<int>(row / p.T), t = static_cast<int>(row - static_cast<long long>(b) * p.T);
+  const long long pos = *p.pos + t;
+  const int r = static_cast<int>(pos % p.R), tid = threadIdx.x;
+  T* q = static_cast<T*>(p.proj) + row * p.ldp + p.off_q;
+  const T* k = static_cast<const T*>(p.proj) + row * p.ldp + p.off_k;
+  const T* v = static_cast<const T*>(p.proj) + row * p.ldp + p.off_v;
+  T* kc = static_cast<T*>(p.k_cache) + (static_cast<long long>(b) * p.G * p.R + r) * p.kw;  // head g: + g * R * kw
+  T* vc = static_cast<T*>(p.v_cache) + (static_cast<long long>(b) * p.G * p.R + r) * p.vw;
+  const T *qw = static_cast<const T*>(p.q_norm), *kw = static_cast<const T*>(p.k_norm);
+  const int nq = p.H * p.dk, nk = p.G * p.dk, half = p.rot_half;
+  for (int i = tid; i < half; i += PREP_THREADS) sincosf(static_cast<float>(pos) * p.inv_freq[i], &sn[i], &cs[i]);
+  float sq = 0.f, sk = 0.f;
+  if (VEC) {
+    for (int i = tid * 8; i < nq; i += PREP_THREADS * 8) {
+      float f[8];
+      load8(q + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sq += f[e] * f[e];
+    }
+    for (int i = tid * 8; i < nk; i += PREP_THREADS * 8) {
+      float f[8];
+      load8(k + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sk += f[e] * f[e];
+    }
+  } else {
+    for (int i = tid; i < nq; i += PREP_THREADS) sq += to_f(q[i]) * to_f(q[i]);
+    for (int i = tid; i < nk; i += PREP_THREADS) sk += to_f(k[i]) * to_f(k[i]);
+  }
+  const float rq = 1.f / sqrtf(sum_block(sq, red) / nq + p.eps);
+  const float rk = 1.f / sqrtf(sum_block(sk, red) / nk + p.eps);  // its barriers also cover the sines
+  if (!RA_IN_BOUNDS(row, 1, static_cast<long long>(p.B) * p.T, kTagWindow)) return;
+  if (VEC) {
+    const int h8 = half >> 3, units = (p.dk >> 3) - h8;  // a unit turns pieces u and u + h8, or copies piece u + h8
+    for (int i = tid; i < (p.H + p.G) * units; i += PREP_THREADS) {
+      const int head = i / units, u = i - head * units;
+      const bool is_q = head < p.H;
+      const int hh = is_q ? head : head - p.H;
+      const T* src = is_q ? q + hh * p.dk : k + hh * p.dk;
+      const T* gain = is_q ? qw + hh * p.dk : kw + hh * p.dk;
+      T* dst = is_q ? q + hh * p.dk : kc + static_cast<long long>(hh) * p.R * p.kw;
+      const float rs = is_q ? rq : rk;
+      float x[8], w[8];
+      const int hi = (u + h8) * 8;
+      load8(src + hi, x);
+      load8(gain + hi, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= rs * w[e];
+      if (u < h8) {
+        float y[8];
+        load8(src + u * 8, y);
+        load8(gain + u * 8, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float a = y[e] * rs * w[e], s = sn[u * 8 + e], c = cs[u * 8 + e];
+          y[e] = a * c - x[e] * s;
+          x[e] = x[e] * c + a * s;
+        }
+        store8(dst + u * 8, y);
+      }
+      store8(dst + hi, x);
+    }
+    const int v8 = p.dv >> 3;
+    for (int i = tid; i < p.G * v8; i += PREP_THREADS) {
+      const int g = i / v8, u = i - g * v8;
+      float x[8];
+      load8(v + g * p.dv + u * 8, x);
+      store8(vc + static_cast<long long>(g) * p.R * p.vw + u * 8, x);
+    }
+    return;
+  }
+  const int rest = p.dk - 2 * half, per = half + rest;  // pairs, then dimensions that pass
+  for (int i = tid; i < (p.H + p.G) * per; i += PREP_THREADS) {
+    const int head = i / per, u = i - head * per;
+    const bool is_q = head < p.H;
+    const int hh = is_q ? head : head - p.H;
+    const T* src = is_q ? q + hh * p.dk : k + hh * p.dk;
+    const T* gain = is_q ? qw + hh * p.dk : kw + hh * p.dk;
+    T* dst = is_q ? q + hh * p.dk : kc + static_cast<long long>(hh) * p.R * p.kw;
+    const float rs = is_q ? rq : rk;
+    if (u < half) {
+      const float a = to_f(src[u]) * rs * to_f(gain[u]), c = to_f(src[u + half]) * rs * to_f(gain[u + half]);
+      from_f(dst[u], a * cs[u] - c * sn[u]);
+      from_f(dst[u + half], c * cs[u] + a * sn[u]);
+    } else {
+      from_f(dst[u + half], to_f(src[u + half]) * rs * to_f(gain[u + half]));
+    }
+  }
+  for (int i = tid; i < p.G * p.dv; i += PREP_THREADS) {
+    const int g = i / p.dv, u = i - g * p.dv;
+    vc[static_cast<long long>(g) * p.R * p.vw + u] = v[i];
+  }
+}
+
+constexpr int ATT_WARPS = 4;
+
+// NR: dimensions per lane (dk and dv at most 32 NR).
+template <typename T, int NR>
+__global__ void __launch_bounds__(32 * ATT_WARPS) window_attend_kernel(const Params p) {
+  const long long row = blockIdx.x;
+  const int h = blockIdx.y * ATT_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= p.H) return;
+  const int b = static_cast<int>(row / p.T), t = static_cast<int>(row - static_cast<long long>(b) * p.T);
+  const long long pos = *p.pos + t;
+  const int g = h / (p.H / p.G);
+  const T* q = static_cast<const T*>(p.proj) + row * p.ldp + p.off_q + h * p.dk;
+  const T* kb = static_cast<const T*>(p.k_cache) + (static_cast<long long>(b) * p.G + g) * p.R * p.kw;
+  const T* vb = static_cast<const T*>(p.v_cache) + (static_cast<long long>(b) * p.G + g) * p.R * p.vw;
+  float qr[NR], o[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = lane + 32 * i;
+    qr[i] = d < p.dk ? to_f(q[d]) * p.scale : 0.f;
+    o[i] = 0.f;
+  }
+  float m = p.sink[h], l = 1.f;  // the sink comes first: weight 1 at the running maximum, no value
+  const int n = static_cast<int>(pos + 1 < p.window ? pos + 1 : p.window);
+  int r = static_cast<int>((pos - n + 1) % p.R);
+  for (int j = 0; j < n; ++j, r = r + 1 == p.R ? 0 : r + 1) {
+    const T* kr = kb + static_cast<long long>(r) * p.kw;
+    const T* vr = vb + static_cast<long long>(r) * p.vw;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = lane + 32 * i;
+      if (d < p.dk) s = fmaf(qr[i], to_f(kr[d]), s);
+    }
+    s = sum_warp(s);
+    if (s > m) {
+      const float a = expf(m - s);
+      l *= a;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) o[i] *= a;
+      m = s;
+    }
+    const float w = expf(s - m);
+    l += w;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = lane + 32 * i;
+      if (d < p.dv) o[i] = fmaf(w, to_f(vr[d]), o[i]);
+    }
+  }
+  T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dv;
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = lane + 32 * i;
+    if (d < p.dv && RA_IN_BOUNDS(h * p.dv + d, 1, p.ldo, kTagWindow)) from_f(out[d], o[i] / l);
+  }
+}
+
+int check(const Params* p) {
+  const char* why = nullptr;
+  if (p->B < 1 || p->T < 1 || p->H < 1 || p->G < 1 || p->H % p->G || p->dk < 1 || p->dv < 1) why = "window: bad shape";
+  else if (p->dk > 512 || p->dv > 512) why = "window: head sizes above 512";
+  else if (p->rot_half < 0 || 2 * p->rot_half > p->dk || p->rot_half > MAX_HALF) why = "window: bad rotary size";
+  else if (p->kw < p->dk || p->vw < p->dv || p->kw % 8 || p->vw % 8 || p->ldp % 8 || p->off_q % 8 || p->off_k % 8 || p->off_v % 8)
+    why = "window: bad row width";
+  else if (p->window < 1 || p->R < 1) why = "window: bad window";
+  if (!why) return kHostOk;
+  set_error(why);
+  return kHostBadArg;
+}
+
+template <typename T>
+int launch_attend(const Params& p, cudaStream_t s) {
+  const dim3 grid(p.B * p.T, (p.H + ATT_WARPS - 1) / ATT_WARPS);
+  const int d = p.dk > p.dv ? p.dk : p.dv;
+  if (d <= 64) window_attend_kernel<T, 2><<<grid, 32 * ATT_WARPS, 0, s>>>(p);
+  else if (d <= 128) window_attend_kernel<T, 4><<<grid, 32 * ATT_WARPS, 0, s>>>(p);
+  else window_attend_kernel<T, 16><<<grid, 32 * ATT_WARPS, 0, s>>>(p);
+  return check_launch("window_attend_kernel");
+}
+
+}  // namespace window
+}  // namespace ra
+
+extern "C" int ra_window_prep(const ra::window::Params* p, int f32, void* stream) {
+  using namespace ra;
+  if (const int rc = window::check(p)) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int rows = p->B * p->T;
+  const bool vec = !(p->dk % 8 || p->dv % 8 || p->rot_half % 8);
+  if (f32 && vec) window::window_prep_kernel<float, true><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else if (f32) window::window_prep_kernel<float, false><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else if (vec) window::window_prep_kernel<__nv_bfloat16, true><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else window::window_prep_kernel<__nv_bfloat16, false><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  return check_launch("window_prep_kernel");
+}
+
+// After ra_window_prep of the same step.
+extern "C" int ra_window_attend(const ra::window::Params* p, int f32, void* stream) {
+  using namespace ra;
+  if (const int rc = window::check(p)) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return f32 ? window::launch_attend<float>(*p, s) : window::launch_attend<__nv_bfloat16>(*p, s);
+}

@@ -6,7 +6,7 @@ from __future__ import annotations
 
 import torch
 
-from ..config import GatedDeltaConfig, LatentAttentionConfig
+from ..config import GatedDeltaConfig, LatentAttentionConfig, WindowAttentionConfig
 
 
 class KVCache:
@@ -38,6 +38,26 @@ class LatentCache:
 
     def clear(self) -> None:
         """Rows past the engine's length are never read: nothing to do."""
+
+
+class WindowCache:
+    """Keys and values of the last tokens in a ring per head: position p in row ``p % rows``, heads-major ``(B, G, rows, dim)``
+    with dims padded to multiples of eight. ``rows`` is a multiple of 128 (key tiles never straddle the end of the ring) that
+    holds the windows of all tokens of a step of ``max_step`` tokens, or the whole context where that is less."""
+
+    def __init__(self, m: WindowAttentionConfig, batch: int, context: int, max_step: int, device, dtype):
+        self.window = context if m.window is None else min(m.window, context)
+        whole, ring = (context + 127) // 128 * 128, (self.window - 1 + max_step + 127 + 127) // 128 * 128
+        self.rows = min(whole, ring)
+        pad = lambda n: (n + 7) // 8 * 8
+        self.k = torch.zeros(batch, m.kv_heads, self.rows, pad(m.dim), device=device, dtype=dtype)
+        self.v = torch.zeros(batch, m.kv_heads, self.rows, pad(m.vdim), device=device, dtype=dtype)
+
+    def bytes(self) -> int:
+        return (self.k.numel() + self.v.numel()) * self.k.element_size()
+
+    def clear(self) -> None:
+        """Rows of positions past the engine's length are never read: nothing to do."""
 
 
 class DeltaState:

@@ -29,15 +29,17 @@ def _llama_from_dict(c: Mapping[str, Any]) -> LlamaConfig:
 FAMILIES = {
     "Llama": Family("llama", LlamaConfig.named, _llama_from_dict, (torch.bfloat16,),
                     ("attn_fwd_sm100", "decode_sm100", "elementwise", "gemm_sm100")),
-    HybridConfig.ARCHITECTURE: Family("dafelorn", HybridConfig.named, HybridConfig.from_dict,
-                                      (torch.bfloat16, torch.float32),
-                                      ("attn_fwd_sm100", "decode_sm100", "delta_chunk_sm100", "delta_sm100", "gemm_sm100",
-                                       "latent_decode_sm100", "latent_sm100", "linear_f32", "residual_f32")),
+    "Dafelorn": Family("dafelorn", HybridConfig.named, HybridConfig.from_dict, (torch.bfloat16, torch.float32),
+                       ("attn_fwd_sm100", "decode_sm100", "delta_chunk_sm100", "delta_sm100", "gemm_sm100",
+                        "latent_decode_sm100", "latent_sm100", "linear_f32", "residual_f32")),
+    "Kalonex": Family("kalonex", HybridConfig.named, HybridConfig.from_dict, (torch.bfloat16, torch.float32),
+                      ("attn_fwd_sm100", "decode_sm100", "gemm_sm100", "linear_f32", "moe", "moe_gemm_sm100",
+                       "residual_f32", "window_decode_sm100", "window_sm100")),
 }
 
 
 def family_of(cfg) -> Family:
-    return FAMILIES[HybridConfig.ARCHITECTURE if isinstance(cfg, HybridConfig) else "Llama"]
+    return FAMILIES[cfg.architecture if isinstance(cfg, HybridConfig) else "Llama"]
 
 
 def load_config(spec: str, **over):

@@ -2,8 +2,9 @@
 
 Packing puts what a step reads together: the input projections of a mixer are one matrix (segments start at multiples of
 eight rows so that every part of the product is 16-byte aligned), the mixer's and the feed-forward's output projections
-are one matrix side by side (their sum is one product over the concatenated inputs), and every dimension is zero-padded
-to a multiple of eight."""
+are one matrix side by side where both read the same stream (their sum is one product over the concatenated inputs), gate
+and up projections are one matrix, the experts of a layer are stacked, and every dimension is zero-padded to a multiple of
+eight."""
 from __future__ import annotations
 
 import json
@@ -15,7 +16,7 @@ from typing import Callable, Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import GatedDeltaConfig, HybridConfig, LatentAttentionConfig
+from ..config import HybridConfig, LatentAttentionConfig, MoEConfig, WindowAttentionConfig
 
 _DTYPES = {"BF16": torch.bfloat16, "F32": torch.float32, "F16": torch.float16, "I32": torch.int32, "I64": torch.int64}
 
@@ -78,6 +79,14 @@ def write_safetensors(path: str, tensors: Dict[str, torch.Tensor]) -> None:
 def hybrid_tensor_shapes(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
     """Names and shapes of a checkpoint of this design."""
     d, out = cfg.d_model, {"embed": (cfg.vocab_size, cfg.d_model)}
+
+    def feed_forward(p: str, ff: int, gated: bool) -> None:
+        if gated:
+            out[p + "gate"] = (ff, d)
+        out.update({p + "up": (ff, d), p + "down": (d, ff)})
+
+    if cfg.loop is not None:
+        out.update({"loop.in": (d, 2 * d), "loop.step": (cfg.loop.times, d)})
     for i, layer in enumerate(cfg.layers):
         if cfg.owner(i) != i:
             continue
@@ -88,6 +97,11 @@ def hybrid_tensor_shapes(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
             out.update({p + "mix.q": (H * (m.dim + m.rot_dim), d), p + "mix.dkv": (m.kv_rank + m.rot_dim, d),
                         p + "mix.dkv.norm": (m.kv_rank,), p + "mix.uk": (H * m.dim, m.kv_rank),
                         p + "mix.uv": (H * m.vdim, m.kv_rank), p + "mix.sink": (H,), p + "mix.g": (H, d)})
+        elif isinstance(m, WindowAttentionConfig):
+            for n, rows in (("q", H * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                out.update({p + f"mix.{n}": (rows, d), p + f"mix.{n}.b": (rows,)})
+            out.update({p + "mix.q.norm": (H * m.dim,), p + "mix.k.norm": (m.kv_heads * m.dim,), p + "mix.sink": (H,),
+                        p + "mix.o.b": (d,)})
         else:
             for n, rows in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", H * m.vdim)):
                 out[p + f"mix.{n}"] = (rows, d)
@@ -96,7 +110,15 @@ def hybrid_tensor_shapes(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
                         p + "mix.norm": (m.vdim,), p + "mix.g": (H * m.vdim, d)})
         out[p + "mix.o"] = (d, H * m.vdim)
         if layer.mlp is not None:
-            out.update({p + "norm2": (d,), p + "mlp.up": (layer.mlp.ff, d), p + "mlp.down": (d, layer.mlp.ff)})
+            out[p + "norm2"] = (d,)
+        if isinstance(layer.mlp, MoEConfig):
+            for e in range(layer.mlp.experts):
+                feed_forward(f"{p}mlp.e{e}.", layer.mlp.ff, True)
+            out[p + "mlp.router"] = (layer.mlp.experts, d)
+            if layer.mlp.shared_ff is not None:
+                feed_forward(p + "mlp.shared.", layer.mlp.shared_ff, True)
+        elif layer.mlp is not None:
+            feed_forward(p + "mlp.", layer.mlp.ff, layer.mlp.gated)
     out["final.norm"] = (d,)
     out["head"] = (cfg.vocab_size, d)
     return out
@@ -105,16 +127,19 @@ def hybrid_tensor_shapes(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
 def random_source(cfg: HybridConfig, device, seed: int = 0) -> Callable[[str], torch.Tensor]:
     """Random weights of the design's shapes (generated on ``device``, tensor by tensor)."""
     shapes = hybrid_tensor_shapes(cfg)
+    number = {name: i for i, name in enumerate(shapes)}
     gen = torch.Generator(device=device)
 
     def get(name: str) -> torch.Tensor:
         shape = shapes[name]
-        gen.manual_seed(seed * 100003 + list(shapes).index(name))
+        gen.manual_seed(seed * 100003 + number[name])
         t = torch.randn(*shape, device=device, generator=gen)
-        if name.endswith((".conv",)) or (len(shape) == 2 and name != "embed"):
+        if name.endswith((".conv",)) or (len(shape) == 2 and name not in ("embed", "loop.step")):
             t /= math.sqrt(shape[1])
-        elif name.endswith((".dkv.norm", "mix.norm")):
+        elif name.endswith((".dkv.norm", "mix.norm", ".q.norm", ".k.norm")):
             t = 1.0 + 0.1 * t
+        elif name.endswith(("norm1", "norm2", "final.norm")):
+            t = 1.0 - cfg.norm_gain_offset + 0.1 * t
         elif name.endswith("dt_bias"):
             t -= 2.0
         elif name != "embed":
@@ -129,15 +154,21 @@ class LayerWeights:
 
     step_w: torch.Tensor                # [mixer input projections | up projection], one launch of a decode step
     in_w: torch.Tensor                  # the first part of it, zero rows up to a multiple of 16 included
+    in_b: Optional[torch.Tensor] = None  # fp32 biases of the first part
     offs: Tuple[int, ...]               # first column of each projection in the product
-    n_split: Optional[int]              # columns from here on leave in fp32 (decay and step-size projections)
-    off_a: int
-    up_w: Optional[torch.Tensor]        # the second part
+    n_split: Optional[int] = None       # columns from here on leave in fp32 (decay and step-size projections)
+    off_a: int = 0
+    up_w: Optional[torch.Tensor] = None  # the second part
     out_w: torch.Tensor                 # [mixer output projection | feed-forward down projection]
+    out_b: Optional[torch.Tensor] = None
     o_cols: int                         # columns of the mixer part (padded)
     mix: Dict[str, torch.Tensor]
     norm1: torch.Tensor
-    norm2: Optional[torch.Tensor]
+    norm2: Optional[torch.Tensor] = None
+    # layers whose feed-forward follows the mixer: [gate | up] and down, or the tensors of routed experts
+    gu_w: Optional[torch.Tensor] = None
+    down_w: Optional[torch.Tensor] = None
+    moe: Optional[Dict[str, torch.Tensor]] = None
 
 
 class HybridWeights:
@@ -148,7 +179,15 @@ class HybridWeights:
         self.d, self.dp = cfg.d_model, round8(cfg.d_model)
         self.embed = self._tensor("embed")
         self.head = self._rows([self._tensor("head")])[0]
+        # a scale of the logits goes into the product's epilogue beside a bias of zeros
+        self.head_b = self._bias([], self.head.shape[0]) if cfg.logit_scale != 1.0 else None
         self.final_norm = self._vec("final.norm")
+        if cfg.loop is not None:
+            w = self._tensor("loop.in")
+            self.loop_w = torch.zeros(self.dp, 2 * self.dp, device=self.device, dtype=dtype)
+            self.loop_w[:self.d, :self.d] = w[:, :self.d]
+            self.loop_w[:self.d, self.dp:self.dp + self.d] = w[:, self.d:]
+            self.loop_step = [self._bias([(0, t)], self.dp) for t in self._tensor("loop.step")]
         self.layers: Dict[int, LayerWeights] = {}
         for i, layer in enumerate(cfg.layers):
             if cfg.owner(i) == i:
@@ -181,12 +220,46 @@ class HybridWeights:
             out[o:o + t.shape[0], :t.shape[1]] = t
         return out, tuple(offs)
 
+    def _bias(self, parts, n: int) -> torch.Tensor:
+        """fp32 vector of ``n`` entries, up to a multiple of 32 of zeros: the vectors of ``parts`` at their offsets."""
+        out = torch.zeros((n + 31) // 32 * 32, device=self.device, dtype=torch.float32)
+        for o, t in parts:
+            out[o:o + t.numel()] = t.float()
+        return out
+
+    def _gate_up(self, p: str) -> torch.Tensor:
+        """``(2 F, dp)``: gate rows, then up rows, each padded to a multiple of eight."""
+        g, u = self._tensor(p + "gate"), self._tensor(p + "up")
+        out = torch.zeros(2, round8(g.shape[0]), self.dp, device=self.device, dtype=self.dtype)
+        out[0, :g.shape[0], :self.d], out[1, :g.shape[0], :self.d] = g, u
+        return out.view(-1, self.dp)
+
+    def _down(self, p: str) -> torch.Tensor:
+        return self._rows([self._tensor(p + "down")])[0]
+
+    def _experts(self, p: str, f: MoEConfig) -> Dict[str, torch.Tensor]:
+        F, kw = round8(f.ff), dict(device=self.device, dtype=self.dtype)
+        out = {"router": self._rows([self._tensor(p + "router")])[0], "gu": torch.empty(f.experts, 2 * F, self.dp, **kw),
+               "down": torch.empty(f.experts, self.dp, F, **kw)}
+        for e in range(f.experts):
+            out["gu"][e], out["down"][e] = self._gate_up(f"{p}e{e}."), self._down(f"{p}e{e}.")
+        if f.shared_ff is not None:
+            out["sh_gu"], out["sh_down"] = self._gate_up(p + "shared."), self._down(p + "shared.")
+        return out
+
     def _layer(self, i: int, layer) -> LayerWeights:
         p, m, L = f"l{i}.", layer.mixer, LayerWeights()
         t = lambda n: self._tensor(p + "mix." + n)
         L.norm1 = self._vec(p + "norm1")
-        L.n_split, L.off_a = None, 0
-        if isinstance(m, LatentAttentionConfig):
+        if isinstance(m, WindowAttentionConfig):
+            parts = ("q", "k", "v")
+            L.in_w, L.offs = self._rows([t(n) for n in parts])
+            L.in_b = self._bias([(o, t(n + ".b")) for o, n in zip(L.offs, parts)], L.in_w.shape[0])
+            L.out_b = self._bias([(0, t("o.b"))], self.dp)
+            inv = torch.tensor(m.rot.inv_freq(), dtype=torch.float64).to(self.device, torch.float32)
+            L.mix = {"q_norm": t("q.norm").contiguous(), "k_norm": t("k.norm").contiguous(), "inv_freq": inv,
+                     "sink": t("sink").float().contiguous()}
+        elif isinstance(m, LatentAttentionConfig):
             L.in_w, L.offs = self._rows([t("q"), t("dkv"), t("g")])
             uk, uv = t("uk"), t("uv")
             w, (ok, ov) = self._rows([uk, uv])
@@ -202,15 +275,22 @@ class HybridWeights:
                      "dt_bias": t("dt_bias").contiguous(), "norm": t("norm").contiguous()}
         o = t("o")
         L.o_cols = round8(o.shape[1])
-        ff = 0 if layer.mlp is None else layer.mlp.ff
+        f = layer.mlp
+        ff = f.ff if f is not None and self.cfg.design.parallel else 0
         L.out_w = torch.zeros(self.dp, L.o_cols + round8(ff), device=self.device, dtype=self.dtype)
         L.out_w[:self.d, :o.shape[1]] = o
-        L.step_w, L.up_w, L.norm2 = L.in_w, None, None
-        if layer.mlp is not None:
-            L.norm2 = self._vec(p + "norm2")
+        L.step_w = L.in_w
+        if f is None:
+            return L
+        L.norm2 = self._vec(p + "norm2")
+        if self.cfg.design.parallel:
             L.step_w, (_, up) = self._rows([L.in_w[:, :self.d], self._tensor(p + "mlp.up")], align=[8, 16])
             L.in_w, L.up_w = L.step_w[:up], L.step_w[up:]
             L.out_w[:self.d, L.o_cols:L.o_cols + ff] = self._tensor(p + "mlp.down")
+        elif isinstance(f, MoEConfig):
+            L.moe = self._experts(p + "mlp.", f)
+        else:
+            L.gu_w, L.down_w = self._gate_up(p + "mlp."), self._down(p + "mlp.")
         return L
 
     def bytes(self) -> int:
@@ -218,4 +298,5 @@ class HybridWeights:
         for L in self.layers.values():
             n += L.step_w.numel() + L.out_w.numel()
             n += L.mix["ukv"].numel() if "ukv" in L.mix else 0
+            n += sum(t.numel() for t in (L.gu_w, L.down_w, *(L.moe or {}).values()) if t is not None)
         return n * self.embed.element_size()

@@ -113,7 +113,7 @@ BOUNDS_TAGS = {1: "gemm store", 2: "gemm residual", 10: "attention forward out",
                32: "swiglu", 33: "embedding token id", 34: "embedding row", 35: "cross-entropy target",
                36: "cross-entropy row", 37: "adamw", 38: "cast", 39: "mask packing", 40: "decode cache row",
                41: "decode merge", 42: "decode mask", 43: "small-M linear", 50: "peer copy", 60: "delta output or state",
-               61: "delta workspace", 62: "latent output", 63: "latent workspace"}
+               61: "delta workspace", 62: "latent output", 63: "latent workspace", 64: "window attention", 65: "expert output or list"}
 
 
 def bounds_report(reset: bool = True) -> dict:

@@ -88,16 +88,20 @@ def linear_wgrad(dy, x, dw_acc):
     return gemm(dy, x, a_mn=True, b_mn=True, out=dw_acc, residual=dw_acc)
 
 
-def linear_ex(x, w, out, *, residual=None, tail=None, n_split: Optional[int] = None, relu2: bool = False):
-    """``out = act(x W^T (+ residual))`` with an inference layer's epilogues, in bf16 or true fp32 by the type of ``x``.
+def linear_ex(x, w, out, *, residual=None, tail=None, n_split: Optional[int] = None, relu2: bool = False, bias=None,
+              alpha: float = 1.0):
+    """``out = act(alpha x W^T + bias (+ residual))`` with an inference layer's epilogues, in bf16 or true fp32 by the type
+    of ``x``.
 
     ``x (M, K)`` and ``w (N, K)`` share a type; ``out`` (a row-strided view) is of that type or fp32. ``residual`` has
-    ``out``'s type and may be ``out``. ``tail``: an fp32 view that takes the columns from ``n_split`` on."""
+    ``out``'s type and may be ``out``. ``tail``: an fp32 view that takes the columns from ``n_split`` on. ``bias``: fp32 by
+    column, with entries up to a multiple of 32; ``alpha`` other than 1 needs one."""
     M, Kd = x.shape
     N = w.shape[0]
     assert w.shape[1] == Kd and x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1 and x.dtype == w.dtype
     n_split = N if tail is None else int(n_split)
-    assert out.shape[0] == M and out.shape[1] >= n_split
+    assert out.shape[0] == M and out.shape[1] >= n_split and (alpha == 1.0 or bias is not None)
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() >= (N + 31) // 32 * 32)
     if residual is not None:
         assert residual.dtype == out.dtype and residual.stride(1) == 1 and not relu2
     if tail is not None:
@@ -107,26 +111,44 @@ def linear_ex(x, w, out, *, residual=None, tail=None, n_split: Optional[int] = N
     if x.dtype == torch.float32:
         assert out.dtype == torch.float32
         _lib.call("ra_linear_f32", ptr(x), ptr(w), ptr(out), ptr(residual), ptr(tail), M, N, Kd, c_ll(x.stride(0)),
-                  c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2), stream_ptr())
+                  c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2), ptr(bias), c_f(alpha),
+                  stream_ptr())
         return out
     if M <= 8 and w.is_contiguous() and (residual is None or (residual.data_ptr() == out.data_ptr() and
                                                               out.dtype == torch.float32)):
         if out.dtype == torch.float32:
-            return linear_segments(x, w, y32=out, add32=residual is not None)
+            return linear_segments(x, w, y32=out, add32=residual is not None, bias=bias, alpha=alpha)
         if relu2:
             return linear_segments(x, w, x2=x, ya=out, act_from=0)
-        return linear_segments(x, w, y=out, y32=tail, n32_from=None if tail is None else n_split)
+        return linear_segments(x, w, y=out, y32=tail, n32_from=None if tail is None else n_split, bias=bias, alpha=alpha)
     _lib.call("ra_gemm_bf16_ex", ptr(x), ptr(w), ptr(out), ptr(residual), ptr(tail), M, N, Kd, c_ll(x.stride(0)),
               c_ll(w.stride(0)), c_ll(out.stride(0)), c_ll(ldr), c_ll(ld2), n_split, int(relu2),
-              int(out.dtype == torch.float32), 8, _status(), stream_ptr())
+              int(out.dtype == torch.float32), ptr(bias), c_f(alpha), 8, _status(), stream_ptr())
+    return out
+
+
+def linear_gated(x, wgu, out):
+    """``out = silu(x Wg^T) * (x Wu^T)`` for ``wgu = [Wg ; Wu]`` ``(2F, K)``, in bf16 or true fp32 by the type of ``x``."""
+    M, F = x.shape[0], wgu.shape[0] // 2
+    assert x.stride(1) == 1 and wgu.is_contiguous() and wgu.shape[1] == x.shape[1] and out.stride(1) == 1
+    assert out.shape[0] == M and out.shape[1] >= F and x.dtype == wgu.dtype == out.dtype
+    if x.dtype == torch.float32:
+        gu = torch.empty(M, 2 * F, device=x.device, dtype=torch.float32)
+        linear_ex(x, wgu, gu)
+        _lib.call("ra_gated_act_f32", ptr(gu), ptr(out), c_ll(out.stride(0)), M, F, stream_ptr())
+    elif M <= 8:
+        _lib.call("ra_small_m_linear_gated", ptr(x), c_ll(x.stride(0)), ptr(wgu), ptr(out), c_ll(out.stride(0)), M, F,
+                  x.shape[1], stream_ptr())
+    else:
+        linear_swiglu(x, wgu, out=out[:, :F])
     return out
 
 
 def linear_segments(x, w, *, x2=None, y=None, y32=None, ya=None, n32_from: Optional[int] = None,
-                    act_from: Optional[int] = None, add32: bool = False):
-    """At most 8 rows: ``x W^T`` in one launch with the columns in up to three segments, each with an output of its own:
+                    act_from: Optional[int] = None, add32: bool = False, bias=None, alpha: float = 1.0):
+    """At most 8 rows: ``alpha x W^T + bias`` in one launch with the columns in up to three segments, each with an output of its own:
     bf16 to ``y``, from ``n32_from`` on fp32 to ``y32`` (added to it with ``add32``), from ``act_from`` on the squared relu
-    of ``x2 W^T`` in bf16 to ``ya``. Borders are multiples of 16; outputs are row-strided views. Without ``y`` the fp32
+    of ``x2 W^T`` in bf16 to ``ya`` (without ``alpha`` and ``bias``). Borders are multiples of 16; outputs are row-strided views. Without ``y`` the fp32
     segment starts at 0. Returns ``y``, ``y32`` or ``ya``, the first that is there."""
     M, Kd = x.shape
     N = w.shape[0]
@@ -139,7 +161,8 @@ def linear_segments(x, w, *, x2=None, y=None, y32=None, ya=None, n32_from: Optio
         assert t is None or (t.shape[0] == M and t.stride(1) == 1 and t.shape[1] >= n)
     ld = lambda t: c_ll(0 if t is None else t.stride(0))
     _lib.call("ra_small_m_linear_segments", ptr(x), ptr(x2), c_ll(x.stride(0)), ptr(w), ptr(y), ld(y), ptr(y32), ld(y32),
-              int(add32), ptr(ya), ld(ya), n32_from, act_from, M, N, Kd, stream_ptr())
+              int(add32), ptr(ya), ld(ya), n32_from, act_from, M, N, Kd, ptr(bias), c_f(alpha),
+              stream_ptr())
     return y if y is not None else (y32 if y32 is not None else ya)
 
 
@@ -206,6 +229,16 @@ def embed_f32(tokens, table, d: int, out):
     assert tokens.dtype == torch.int32 and tokens.is_contiguous() and out.dtype == torch.float32 and out.is_contiguous()
     _lib.call("ra_embed_f32", ptr(tokens), ptr(table), c_ll(table.stride(0)), ptr(out), c_ll(out.stride(0)),
               tokens.numel(), d, table.shape[0], int(table.dtype == torch.float32), stream_ptr())
+    return out
+
+
+def stream_pair(tokens, table, x, d: int):
+    """``(rows, 2 dp)`` in ``table``'s type: the fp32 rows of ``x (rows, dp)`` beside the tokens' rows of ``table``."""
+    rows, dp = x.shape
+    assert tokens.dtype == torch.int32 and tokens.numel() == rows and x.dtype == torch.float32 and x.stride(1) == 1
+    out = torch.empty(rows, 2 * dp, device=x.device, dtype=table.dtype)
+    _lib.call("ra_stream_pair", ptr(tokens), ptr(table), c_ll(table.stride(0)), ptr(x), c_ll(x.stride(0)), ptr(out), rows, d,
+              dp, table.shape[0], int(table.dtype == torch.float32), stream_ptr())
     return out
 
 

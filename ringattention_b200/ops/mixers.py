@@ -1,5 +1,5 @@
-"""Bindings of the token mixers of hybrid decoders: the gated delta rule (``delta_sm100.cu``) and latent attention
-(``latent_sm100.cu``). Activations and weights are bf16 or fp32 throughout (one type per call); states, decays, scores
+"""Bindings of the token mixers of hybrid decoders: the gated delta rule (``delta_sm100.cu``), latent attention
+(``latent_sm100.cu``) and windowed attention (``window_sm100.cu``). Activations and weights are bf16 or fp32 throughout (one type per call); states, decays, scores
 and softmax are fp32 in both."""
 from __future__ import annotations
 
@@ -222,3 +222,73 @@ def _latent_expanded(proj, out, B: int, T: int, m, offs, w, cache, n: int) -> No
     two_part_attention(q, kv[:, :, :H * dn].view(B, n, H, dn), cache[:, :n, r_pad:r_pad + dr],
                        kv[:, :, w["uv_off"]:w["uv_off"] + H * dv].view(B, n, H, dv), o, scale=m.scale, q_pos0=n - T,
                        sink=w["sink"], gate=proj[:, offs[2]:offs[2] + H])
+
+
+# --------------------------------------------------------------------------------------------- windowed attention
+class _WindowParams(ctypes.Structure):
+    _fields_ = [("B", c_i), ("T", c_i), ("H", c_i), ("G", c_i), ("dk", c_i), ("dv", c_i), ("rot_half", c_i),
+                ("proj", c_vp), ("ldp", c_ll), ("off_q", c_i), ("off_k", c_i), ("off_v", c_i),
+                ("q_norm", c_vp), ("k_norm", c_vp), ("inv_freq", c_vp), ("k_cache", c_vp), ("v_cache", c_vp),
+                ("R", c_i), ("kw", c_i), ("vw", c_i), ("window", c_i), ("sink", c_vp), ("out", c_vp), ("ldo", c_ll),
+                ("eps", c_f), ("scale", c_f), ("pos", c_vp), ("splits", c_i), ("n_max", c_ll)]
+
+
+class _WindowArgs(ctypes.Structure):
+    _fields_ = [("q", c_vp), ("q_sb", c_ll), ("q_ss", c_ll), ("q_sh", c_ll),
+                ("k", c_vp), ("k_sb", c_ll), ("k_ss", c_ll), ("k_sh", c_ll),
+                ("v", c_vp), ("v_sb", c_ll), ("v_ss", c_ll), ("v_sh", c_ll),
+                ("out", c_vp), ("o_sb", c_ll), ("o_ss", c_ll), ("o_sh", c_ll), ("sink", c_vp),
+                ("B", c_i), ("H", c_i), ("G", c_i), ("Sq", c_i), ("dk", c_i), ("dv", c_i), ("window", c_i), ("k_rows", c_i),
+                ("scale", c_f), ("q_pos0", c_ll), ("status", c_vp), ("stream", c_vp)]
+
+
+def window_attention(q, k_ring, v_ring, out, *, scale: float, q_pos0: int, window: int, sink) -> None:
+    """Causal attention over the last ``window`` keys on the tensor cores. ``q (B, Sq, H, dk)`` at positions ``q_pos0 ..``,
+    ``k_ring (B, G, R, dk)`` and ``v_ring (B, G, R, dv)`` with position p in row ``p % R``, ``out (B, Sq, H, dv)``: bf16 views,
+    innermost contiguous; ``sink (H,)`` fp32. The ring has to hold the window of every query of the step."""
+    B, Sq, H, dk = q.shape
+    a = _WindowArgs()
+    a.q, (a.q_sb, a.q_ss, a.q_sh) = _p(q), q.stride()[:3]
+    a.k, (a.k_sb, a.k_sh, a.k_ss) = _p(k_ring), k_ring.stride()[:3]
+    a.v, (a.v_sb, a.v_sh, a.v_ss) = _p(v_ring), v_ring.stride()[:3]
+    a.out, (a.o_sb, a.o_ss, a.o_sh) = _p(out), out.stride()[:3]
+    a.sink, a.B, a.H, a.G, a.Sq, a.dk, a.dv = _p(sink), B, H, k_ring.shape[1], Sq, dk, v_ring.shape[3]
+    a.window, a.k_rows, a.scale, a.q_pos0 = window, k_ring.shape[2], scale, q_pos0
+    a.status, a.stream = _lib.status_tensor(q.device).data_ptr(), torch.cuda.current_stream().cuda_stream
+    _lib.call("ra_attn_window", ctypes.byref(a))
+
+
+def window_tensor_core_fits(m, proj, out) -> bool:
+    """Sizes the tensor-core kernels take (every head starts at a multiple of 16 bytes)."""
+    return (proj.dtype == torch.bfloat16 and m.dim <= 128 and m.vdim <= 128 and not (m.dim % 8 or m.vdim % 8)
+            and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)
+
+
+def window_mixer(proj, out, *, B: int, T: int, m, offs, w, cache, length: int, eps: float, pos) -> None:
+    """Windowed attention of ``T`` new tokens of each of ``B`` sequences.
+
+    ``proj (B*T, ld)``: query, key and value projections at columns ``offs`` (queries are normed and turned in place).
+    ``cache``: a :class:`~ringattention_b200.models.cache.WindowCache`, which the new tokens join. ``length``: tokens before
+    this step (for a single token an upper bound that sizes grids; the kernels take positions from ``pos``). ``w``: ``q_norm``,
+    ``k_norm``, ``inv_freq``, ``sink``. ``m``: a :class:`~ringattention_b200.config.WindowAttentionConfig`."""
+    rows, H, G, dk, dv = B * T, m.heads, m.kv_heads, m.dim, m.vdim
+    assert proj.shape[0] == rows and proj.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype
+    assert cache.k.is_contiguous() and cache.v.is_contiguous() and cache.k.dtype == proj.dtype
+    a = _WindowParams()
+    a.B, a.T, a.H, a.G, a.dk, a.dv, a.rot_half = B, T, H, G, dk, dv, m.rot.dims // 2
+    a.proj, a.ldp = _p(proj), proj.stride(0)
+    a.off_q, a.off_k, a.off_v = offs
+    a.q_norm, a.k_norm, a.inv_freq, a.sink = _p(w["q_norm"]), _p(w["k_norm"]), _p(w["inv_freq"]), _p(w["sink"])
+    a.k_cache, a.v_cache, a.R, a.kw, a.vw = _p(cache.k), _p(cache.v), cache.rows, cache.k.shape[3], cache.v.shape[3]
+    a.window = min(cache.window, 1 << 30)
+    a.out, a.ldo, a.eps, a.scale, a.pos, a.n_max = _p(out), out.stride(0), eps, m.scale, _p(pos), length + 1
+    is32, fits = int(proj.dtype == torch.float32), window_tensor_core_fits(m, proj, out)
+    if T == 1 and fits:
+        return _lib.call("ra_window_decode", ctypes.byref(a), _lib.stream_ptr())
+    _lib.call("ra_window_prep", ctypes.byref(a), is32, _lib.stream_ptr())
+    if not fits:
+        return _lib.call("ra_window_attend", ctypes.byref(a), is32, _lib.stream_ptr())
+    ld = proj.stride(0)
+    q = proj.as_strided((B, T, H, dk), (T * ld, ld, dk, 1), proj.storage_offset() + offs[0])
+    o = out.as_strided((B, T, H, dv), (T * out.stride(0), out.stride(0), dv, 1), out.storage_offset())
+    window_attention(q, cache.k, cache.v, o, scale=m.scale, q_pos0=length, window=a.window, sink=w["sink"])
