@@ -69,9 +69,10 @@ def checkpoint_source(spec: str):
 
 
 def make_engine(cfg, max_context: int, *, source=None, dtype: torch.dtype = torch.bfloat16, batch: int = 1, device="cuda",
-                seed: int = 0, axis=None, streams: int = 0, max_new_tokens: int = 512):
+                seed: int = 0, axis=None, streams: int = 0, max_new_tokens: int = 512, max_step: int = 8192):
     """The inference engine of a configuration. ``source``: tensor name -> tensor (random weights when None). A context
-    is rounded up to what the engine needs."""
+    is rounded up to what the engine needs. ``max_step``: tokens of a sequence that a hybrid decoder with windowed attention
+    runs at once."""
     if dtype not in family_of(cfg).dtypes:
         raise ValueError(f"this model does not run in {dtype}")
     if isinstance(cfg, HybridConfig):
@@ -81,7 +82,7 @@ def make_engine(cfg, max_context: int, *, source=None, dtype: torch.dtype = torc
             raise ValueError("hybrid decoders have no shared-prefix streams")
         from .hybrid_infer import HybridInference
 
-        return HybridInference(cfg, max_context, batch=batch, device=device, seed=seed, dtype=dtype,
+        return HybridInference(cfg, max_context, batch=batch, device=device, seed=seed, dtype=dtype, max_step=max_step,
                                source=None if source is None else source.__getitem__)
     from .llama_infer import LlamaInference
     from .params import FlatParams

@@ -1,9 +1,9 @@
 """Serving benchmark of hybrid decoders beside the LLaMA engine at equal width, depth and feed-forward parameters.
 
-    python bench.py --serve [--serve-models dafelorn-1b,dafelorn-7b] [--serve-layers 8] ...
+    python bench.py --serve [--serve-models dafelorn-1b,dafelorn-7b,kalonex-1b,kalonex-7b] [--serve-layers 8] ...
     python -m ringattention_b200.utils.servebench --kernels          # device time per launcher of one prefill chunk
 
-For every model: prefill tokens/s (chunks of ``--chunk`` tokens up to ``--context``) and decode tokens/s at that context
+A model whose layers run several times counts layer runs. For every model: prefill tokens/s (chunks of ``--chunk`` tokens up to ``--context``) and decode tokens/s at that context
 (replayed CUDA graph), with random weights and tokens. All device times are CUDA events. The working set of a step (the
 weights) exceeds the L2 by far, so no flush is needed between steps.
 """
@@ -16,7 +16,7 @@ from collections import defaultdict
 
 import torch
 
-PARTNER = {"dafelorn-1b": "llama-1b", "dafelorn-7b": "llama-7b", "dafelorn-tiny": "llama-tiny"}
+PARTNER = {f"{d}-{n}": f"llama-{n}" for d in ("dafelorn", "kalonex") for n in ("tiny", "1b", "7b")}
 
 
 def build(model: str, layers, max_context: int, batch: int):
@@ -24,6 +24,10 @@ def build(model: str, layers, max_context: int, batch: int):
 
     cfg = registry.load_config(model, **({} if layers is None else {"n_layers": layers}))
     return cfg, registry.make_engine(cfg, max_context, batch=batch)
+
+
+def n_runs(cfg) -> int:
+    return len(cfg.runs) if hasattr(cfg, "runs") else cfg.n_layers
 
 
 def run_model(model: str, layers, context: int, chunk: int, batch: int, new_tokens: int, warmup: int = 3) -> dict:
@@ -60,7 +64,7 @@ def run_model(model: str, layers, context: int, chunk: int, batch: int, new_toke
         lat.append(a.elapsed_time(b))
     _lib.check_status()
     ms = statistics.median(lat)
-    out = {"model": model, "n_layers": cfg.n_layers, "params_b": round(cfg.n_params() / 1e9, 3), "batch": batch,
+    out = {"model": model, "n_layers": n_runs(cfg), "params_b": round(cfg.n_params() / 1e9, 3), "batch": batch,
            "context": context, "chunk": chunk, "prefill_tokens_per_s": round(batch * context / prefill_ms * 1e3),
            "prefill_ms": round(prefill_ms, 2), "decode_ms": round(ms, 4), "decode_tokens_per_s": round(batch / ms * 1e3, 1),
            "decode_steps": len(lat)}
@@ -113,14 +117,14 @@ def kernels(model: str, layers, context: int, chunk: int, batch: int) -> dict:
         with CallTimer() as d:
             eng.decode_step(nxt)
         eng.reset()
-    return {"model": model, "context": context, "chunk": chunk, "batch": batch, "n_layers": cfg.n_layers,
+    return {"model": model, "context": context, "chunk": chunk, "batch": batch, "n_layers": n_runs(cfg),
             "prefill_chunk": t.rows, "decode_step_eager": d.rows}
 
 
 def add_arguments(ap: argparse.ArgumentParser) -> None:
-    ap.add_argument("--serve-models", default="dafelorn-1b,dafelorn-7b",
+    ap.add_argument("--serve-models", default="dafelorn-1b,dafelorn-7b,kalonex-1b,kalonex-7b",
                     help="hybrid presets; each is followed by the LLaMA preset of equal size")
-    ap.add_argument("--serve-layers", type=int, default=None, help="override the layer count (a multiple of 4)")
+    ap.add_argument("--serve-layers", type=int, default=None, help="override the number of layer runs (a multiple of 4)")
     ap.add_argument("--serve-context", type=int, default=32768)
     ap.add_argument("--serve-chunk", type=int, default=8192)
     ap.add_argument("--serve-batches", default="1,4")

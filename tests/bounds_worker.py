@@ -113,17 +113,22 @@ def main():
     K.linear_ex(torch.randn(77, 520, device=dev).to(bf), ws_[:192].contiguous(), canary((77, 64), bf),
                 tail=canary((77, 128), torch.float32), n_split=64)
     K.linear_ex(torch.randn(77, 70, device=dev), torch.randn(51, 70, device=dev), canary((77, 51), torch.float32), relu2=True)
-    import dafelorn_torch as R
-    from hybrid_configs import CONFIGS
+    K.linear_gated(xs_, ws_[:144].contiguous(), canary((3, 72), bf))
+    K.linear_gated(torch.randn(77, 520, device=dev).to(bf), ws_[:144].contiguous(), canary((77, 72), bf))
+    import dafelorn_torch
+    import hybrid_configs
+    import kalonex_configs
+    import kalonex_torch
     from ringattention_b200.config import HybridConfig
     from ringattention_b200.models import registry
 
-    for raw in CONFIGS.values():
+    for raw in [*hybrid_configs.CONFIGS.values(), *kalonex_configs.CONFIGS.values()]:
+        R = dafelorn_torch if raw["architecture"] == "Dafelorn" else kalonex_torch
         w = R.random_model(raw, seed=2)
         for dt in (bf, torch.float32):
-            eng = registry.make_engine(HybridConfig.from_dict(raw), 200, source=w, dtype=dt, batch=2)
+            eng = registry.make_engine(HybridConfig.from_dict(raw), 200, source=w, dtype=dt, batch=2, max_step=64)
             for c in eng.caches:  # caches and states inside canaries
-                for name in ("data", "state", "ring"):
+                for name in ("data", "state", "ring", "k", "v"):
                     if hasattr(c, name):
                         t = getattr(c, name)
                         setattr(c, name, canary(tuple(t.shape), t.dtype, fill=t))

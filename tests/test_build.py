@@ -21,7 +21,7 @@ def test_build_and_symbols():
 
 
 @pytest.mark.skipif(shutil.which("nvcc") is None, reason="nvcc not installed")
-@pytest.mark.parametrize("family", ["Dafelorn", "Llama"])
+@pytest.mark.parametrize("family", ["Dafelorn", "Kalonex", "Llama"])
 def test_build_of_one_engines_sources(family, tmp_path, monkeypatch):
     """A library of only the sources an engine names exports what the engine calls and nothing of training."""
     from ringattention_b200 import _build
@@ -34,12 +34,17 @@ def test_build_of_one_engines_sources(family, tmp_path, monkeypatch):
     assert path.parent == tmp_path and path != _build.LIB_PATH
     lib = ctypes.CDLL(str(path))
     want = ["ra_last_error", "ra_decode_advance", "ra_small_m_linear", "ra_attn_fwd"]
-    want += (["ra_attn_two_part", "ra_delta_step", "ra_delta_chunk_scan", "ra_latent_few_attend", "ra_latent_prep",
-              "ra_linear_f32", "ra_norm_f32", "ra_embed_f32", "ra_gemm_bf16_ex", "ra_small_m_linear_segments"]
-             if family == "Dafelorn" else ["ra_rmsnorm_fwd", "ra_rope_append", "ra_gemm_bf16_swiglu"])
+    hybrid = ["ra_linear_f32", "ra_norm_f32", "ra_embed_f32", "ra_gemm_bf16_ex", "ra_small_m_linear_segments"]
+    want += {"Dafelorn": hybrid + ["ra_attn_two_part", "ra_delta_step", "ra_delta_chunk_scan", "ra_latent_few_attend",
+                                   "ra_latent_prep"],
+             "Kalonex": hybrid + ["ra_attn_window", "ra_window_prep", "ra_window_attend", "ra_window_decode", "ra_moe_few",
+                                  "ra_moe_route", "ra_moe_gemm", "ra_moe_combine", "ra_stream_pair", "ra_gated_act_f32",
+                                  "ra_small_m_linear_gated", "ra_gemm_bf16_swiglu"],
+             "Llama": ["ra_rmsnorm_fwd", "ra_rope_append", "ra_gemm_bf16_swiglu"]}[family]
     for sym in want:
         assert hasattr(lib, sym), sym
-    for sym in ("ra_attn_bwd", "ra_adamw" if family == "Dafelorn" else "ra_delta_step"):
+    for sym in ("ra_attn_bwd", "ra_adamw" if family != "Llama" else "ra_delta_step",
+                "ra_moe_gemm" if family != "Kalonex" else "ra_latent_prep"):
         assert not hasattr(lib, sym), sym
     with pytest.raises(ValueError, match="no such sources"):
         _build.build(only=("nothing",))
