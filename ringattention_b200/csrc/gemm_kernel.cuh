@@ -321,6 +321,17 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
       tn = (tn + tn_rot) % tiles_n;
       const int row = tm * BM + quad * 32 + lane;
       const int n0 = tn * BN;
+      // The fp32 addend is loaded one chunk of 32 columns ahead, the first while the tile's products still run: with a
+      // short K the epilogue would otherwise be a chain of memory round trips longer than the main loop.
+      const bool add32 = p.c_fp32 && p.R && row < p.M;
+      float4 ahead[8];
+      auto load_addend = [&](int c) {
+        const float* src = reinterpret_cast<const float*>(p.R) + static_cast<long long>(row) * p.ldr + n0 + c * 32;
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (n0 + c * 32 + j * 4 < p.N) ahead[j] = *reinterpret_cast<const float4*>(src + 4 * j);
+      };
+      if (add32) load_addend(0);
       if (!mbar_wait(&tfull[acc], acc_phase, wc, kTimeoutTmemFull)) break;
       tc_fence_after();
       const uint32_t t_row = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) +
@@ -391,15 +402,19 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
                                 __uint_as_float(r[4 * j + 3]));
           } else if (p.c_fp32) {
             float* dst = reinterpret_cast<float*>(p.C) + static_cast<long long>(row) * p.ldc + col0;
+            float4 now[8];
+            if (add32) {
+#pragma unroll
+              for (int j = 0; j < 8; ++j) now[j] = ahead[j];
+              if (c + 1 < BN / 32) load_addend(c + 1);
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
               if (col0 + j * 4 < p.N) {
                 float4 v = make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]),
                                        __uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3]));
-                if (p.R) {
-                  const float4 o = *reinterpret_cast<const float4*>(
-                      reinterpret_cast<const float*>(p.R) + static_cast<long long>(row) * p.ldr + col0 + 4 * j);
-                  v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
+                if (add32) {
+                  v.x += now[j].x; v.y += now[j].y; v.z += now[j].z; v.w += now[j].w;
                 }
                 if (RA_IN_BOUNDS(row, 1, p.M, kTagGemmStore) && RA_IN_BOUNDS(col0 + 4 * j, 4, p.N, kTagGemmStore))
                   *reinterpret_cast<float4*>(dst + 4 * j) = v;

@@ -19,7 +19,7 @@ struct Params {
   const void *sh_gu, *sh_down; // (2 Fs, dp); (dp, Fs)
   int* ids;                    // (rows, top) chosen experts
   float* weight;               // (rows, top) their scores
-  void* act;                   // few rows: (rows, top * F + Fs); many rows: (rows * top, F)
+  void* act;                   // few rows: (rows, top * F + Fs); many rows: (128 row tiles, F), see moe_gemm_sm100.cu
   float* x;                    // (rows, ldx) residual stream
   long long ldx;
   // many rows: entries t * top + k by expert, list[e * rows + i], i < count[e]

@@ -1,11 +1,12 @@
-// Matrix products of routed experts for many rows: a persistent tcgen05 GEMM over the tiles of all experts. The rows of A are
-// gathered by TMA (tile::gather4, four rows a copy, one copy per lane of the producer warp) from the entries in an expert's
-// list, the outputs are scattered by the same list, so nothing is sorted or copied in memory:
-//   UP   : act[entry] = silu(w g) * (w u) with g, u = the gate and up products of token entry / top, w = its score
-//   DOWN : y[entry] = W_down act[entry]
-// Tile order: column tiles of one row tile first, expert after expert. Each CTA finds its tiles from the experts' counts,
-// which it sums up itself. Pipeline and accumulators as in gemm_kernel.cuh: 128 x 256 x 64 tiles, four stages, two
-// accumulators; a gate/up tile is 128 gate columns and the 128 matching up columns.
+// Matrix products of routed experts for many rows: a persistent tcgen05 GEMM over the row tiles of all experts.
+//   UP   : act[128 tile + i] = silu(w g) * (w u) with g, u = the gate and up products of the token of the tile's i-th entry
+//          and w = its score. Four warps gather the tokens' rows with cp.async straight into the swizzled tile (a TMA gather
+//          of four rows a copy ran at a third of this speed), so no sorted copy of the input is made.
+//   DOWN : y[entry] = W_down act[128 tile + i]; tiles of act are plain TMA boxes, the rows are scattered by the list.
+// Row tiles are numbered expert after expert; column tiles of one row tile run first. Each CTA finds its tiles from the
+// experts' counts, which it sums up itself. Pipeline and accumulators as in gemm_kernel.cuh: 128 x 256 x 64 tiles, four
+// stages, two accumulators; a gate/up tile is 128 gate columns and the 128 matching up columns.
+#include "common/mma_sync.cuh"
 #include "common/sm100.cuh"
 #include "moe_common.cuh"
 
@@ -14,7 +15,9 @@ RA_BOUNDS_TRANSLATION_UNIT()
 namespace ra {
 namespace moe {
 
-constexpr int BM = 128, BN = 256, BK = 64, STAGES = 4, NUM_ACC = 2, GEMM_THREADS = 192;
+constexpr int BM = 128, BN = 256, BK = 64, STAGES = 4, NUM_ACC = 2, GATHER = 128;
+constexpr int GEMM_THREADS = 192;      // TMA, MMA and four epilogue warps; UP has GATHER threads more
+constexpr int IN_FLIGHT = 2;           // stages of gathered rows on their way per thread
 constexpr int A_BYTES = BM * BK * 2, B_BYTES = BN * BK * 2;
 constexpr int GEMM_SMEM = STAGES * (A_BYTES + B_BYTES) + 1024 + 256 + MAX_EXPERTS * 4 + 16;
 
@@ -30,18 +33,14 @@ struct TileWalk {
   }
 };
 
-// Four rows of a K-major operand (one 128-byte row segment each) to 512 consecutive bytes.
-__device__ __forceinline__ void tma_gather4(void* dst, const CUtensorMap* m, uint64_t* bar, int x, int y0, int y1, int y2,
-                                            int y3) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, "
-      "%6, %7}], [%2];" ::"r"(smem_u32(dst)),
-      "l"(m), "r"(smem_u32(bar)), "r"(x), "r"(y0), "r"(y1), "r"(y2), "r"(y3)
-      : "memory");
+// Rows of act: every expert may leave its last row tile partly empty.
+__host__ __device__ __forceinline__ long long act_rows(const Params& p) {
+  const long long n = static_cast<long long>(p.rows) * p.top;
+  return BM * (n / BM + (n < p.E ? n : p.E));
 }
 
 template <bool UP>
-__global__ void __launch_bounds__(GEMM_THREADS, 1)
+__global__ void __launch_bounds__(GEMM_THREADS + (UP ? GATHER : 0), 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b, const Params p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -59,7 +58,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
   const WaitCtx wc{abort_flag, p.status};
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; ++s) {
-      mbar_init(&full[s], 1);
+      mbar_init(&full[s], UP ? 1 + GATHER : 1);
       mbar_init(&empty[s], 1);
     }
     for (int a = 0; a < NUM_ACC; ++a) {
@@ -100,7 +99,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
   TileWalk walk{0, 0};
 
   if (warp == 0) {
-    // ------------------------------------------------------------------ TMA producer (all lanes: four rows of A each)
+    // ------------------------------------------------------------------ TMA producer (warp-uniform flow)
     const bool leader = elect_one();
     int stage = 0;
     uint32_t phase = 0;
@@ -108,33 +107,22 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
     for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
       const int mt = tile / tiles_n, tn = tile - mt * tiles_n;
       if (!walk.find(tile_end, p.E, mt)) break;
-      const int cnt = min(p.count[walk.e], p.rows), m0 = (mt - walk.first) * BM;
-      const int* list = p.list + static_cast<long long>(walk.e) * p.rows;
-      int src[4];
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {  // rows past the end repeat the last one; their outputs are not stored
-        const int entry = list[min(m0 + 4 * lane + i, cnt - 1)];
-        src[i] = min(max(UP ? entry / p.top : entry, 0), (UP ? p.rows : p.rows * p.top) - 1);
-      }
+      const int row = UP ? walk.e * 2 * p.F + tn * (BN / 2) : walk.e * p.dp + tn * BN;
       for (int kb = 0; kb < num_kb; ++kb) {
         const int k0 = kb * BK;
-        // (the lanes agree: a lane alone that gave up would leave a stage half filled)
-        if (!__all_sync(0xffffffffu, mbar_wait(&empty[stage], phase ^ 1u, wc, kTimeoutSmemEmpty))) {
+        if (!mbar_wait(&empty[stage], phase ^ 1u, wc, kTimeoutSmemEmpty)) {
           ok = false;
           break;
         }
-        uint8_t* a_dst = sA + stage * A_BYTES;
         uint8_t* b_dst = sB + stage * B_BYTES;
-        if (leader) mbar_arrive_expect_tx(&full[stage], A_BYTES + B_BYTES);
-        __syncwarp();
-        tma_gather4(a_dst + lane * 512, &tma_a, &full[stage], k0, src[0], src[1], src[2], src[3]);
         if (leader) {
+          mbar_arrive_expect_tx(&full[stage], B_BYTES + (UP ? 0 : A_BYTES));
           if (UP) {
-            const int r = walk.e * 2 * p.F + tn * (BN / 2);
-            tma_load_2d(b_dst, &tma_b, &full[stage], k0, r);
-            tma_load_2d(b_dst + B_BYTES / 2, &tma_b, &full[stage], k0, r + p.F);
+            tma_load_2d(b_dst, &tma_b, &full[stage], k0, row);
+            tma_load_2d(b_dst + B_BYTES / 2, &tma_b, &full[stage], k0, row + p.F);
           } else {
-            tma_load_2d(b_dst, &tma_b, &full[stage], k0, walk.e * p.dp + tn * BN);
+            tma_load_2d(sA + stage * A_BYTES, &tma_a, &full[stage], k0, mt * BM);
+            tma_load_2d(b_dst, &tma_b, &full[stage], k0, row);
           }
         }
         if (++stage == STAGES) {
@@ -182,6 +170,52 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
       }
     }
     __syncwarp();
+  } else if (UP && warp >= 6) {
+    // ------------------------------------------------------------------ gather (4 warps)
+    // Thread t copies 16-byte piece t % 8 of rows t / 8 + 16 j. A stage is handed over when its copies have landed, which
+    // is known IN_FLIGHT stages later; the fence makes them visible to the tensor core.
+    const int t = threadIdx.x - GEMM_THREADS, piece = t & 7, r0 = t >> 3;
+    int stage = 0, issued = 0;
+    uint32_t phase = 0;
+    bool ok = true;
+    const __nv_bfloat16* h = static_cast<const __nv_bfloat16*>(p.h);
+    for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
+      const int mt = tile / tiles_n;
+      if (!walk.find(tile_end, p.E, mt)) break;
+      const int cnt = min(p.count[walk.e], p.rows), m0 = (mt - walk.first) * BM;
+      const int* list = p.list + static_cast<long long>(walk.e) * p.rows;
+      const __nv_bfloat16* src[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {  // rows past the end repeat the last one; their outputs are not stored
+        const int token = list[min(m0 + r0 + 16 * j, cnt - 1)] / p.top;
+        src[j] = h + static_cast<long long>(min(max(token, 0), p.rows - 1)) * p.dp + piece * 8;
+      }
+      for (int kb = 0; kb < num_kb; ++kb) {
+        const int k0 = kb * BK;
+        if (!mbar_wait(&empty[stage], phase ^ 1u, wc, kTimeoutSmemEmpty)) {
+          ok = false;
+          break;
+        }
+        const bool in = k0 + piece * 8 < K;
+        uint8_t* dst = sA + stage * A_BYTES + r0 * 128 + ((piece ^ (r0 & 7)) << 4);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) cp_async16(dst + j * 16 * 128, src[j] + (in ? k0 : -piece * 8), in ? 16 : 0);
+        cp_async_commit();
+        if (++issued > IN_FLIGHT) {
+          cp_async_wait<IN_FLIGHT>();
+          fence_proxy_async_smem();
+          mbar_arrive(&full[(stage + STAGES - IN_FLIGHT) % STAGES]);
+        }
+        if (++stage == STAGES) {
+          stage = 0;
+          phase ^= 1u;
+        }
+      }
+    }
+    cp_async_wait<0>();
+    fence_proxy_async_smem();
+    if (ok)
+      for (int i = min(issued, IN_FLIGHT); i > 0; --i) mbar_arrive(&full[(stage + STAGES - i) % STAGES]);
   } else {
     // ------------------------------------------------------------------ epilogue (4 warps)
     const int quad = warp & 3;
@@ -194,8 +228,9 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
       const bool valid = i < cnt;
       const int entry = valid ? p.list[static_cast<long long>(walk.e) * p.rows + i] : 0;
       const float w = UP && valid ? p.weight[entry] : 0.f;
-      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(UP ? p.act : p.y) + static_cast<long long>(entry) * N;
-      const bool store = valid && RA_IN_BOUNDS(entry, 1, static_cast<long long>(p.rows) * p.top, kTagMoe);
+      const long long out_row = UP ? static_cast<long long>(mt) * BM + quad * 32 + lane : entry;
+      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(UP ? p.act : p.y) + out_row * N;
+      const bool store = valid && RA_IN_BOUNDS(out_row, 1, UP ? act_rows(p) : static_cast<long long>(p.rows) * p.top, kTagMoe);
       if (!mbar_wait(&tfull[acc], acc_phase, wc, kTimeoutTmemFull)) break;
       tc_fence_after();
       const uint32_t t_row = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + static_cast<uint32_t>(acc * BN);
@@ -246,7 +281,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
 
 template <bool UP>
 int launch_gemm(const Params& p, cudaStream_t s) {
-  const long long K = UP ? p.dp : p.F, a_rows = UP ? p.rows : static_cast<long long>(p.rows) * p.top;
+  const long long K = UP ? p.dp : p.F, a_rows = UP ? p.rows : act_rows(p);
   const long long b_rows = static_cast<long long>(p.E) * (UP ? 2 * p.F : p.dp);
   const void *A = UP ? p.h : p.act, *B = UP ? p.gu : p.down;
   if (b_rows > (1ll << 31) - 1 || a_rows > (1ll << 31) - 1 ||
@@ -257,7 +292,7 @@ int launch_gemm(const Params& p, cudaStream_t s) {
   }
   CUtensorMap ta, tb;
   uint64_t dims[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(a_rows)}, str[1] = {static_cast<uint64_t>(K) * 2};
-  uint32_t box[2] = {BK, 1};
+  uint32_t box[2] = {BK, BM};
   if (int rc = make_tmap_bf16_sw128(&ta, A, 2, dims, str, box)) return rc;
   dims[1] = static_cast<uint64_t>(b_rows);
   box[1] = UP ? BN / 2 : BN;
@@ -268,14 +303,14 @@ int launch_gemm(const Params& p, cudaStream_t s) {
     set_error("moe_gemm: smem attribute");
     return kHostLaunchFail;
   }
-  kern<<<sm_count(), GEMM_THREADS, GEMM_SMEM, s>>>(ta, tb, p);
+  kern<<<sm_count(), GEMM_THREADS + (UP ? GATHER : 0), GEMM_SMEM, s>>>(ta, tb, p);
   return check_launch("moe_gemm_kernel");
 }
 
 }  // namespace moe
 }  // namespace ra
 
-// After ra_moe_route: act (rows * top, F) and y (rows * top, dp) by entry, bf16. Two launches.
+// After ra_moe_route: act (act_rows, F) by row tile and y (rows * top, dp) by entry, bf16. Two launches.
 extern "C" int ra_moe_gemm(const ra::moe::Params* p, void* stream) {
   using namespace ra;
   if (const int rc = moe::check(p)) return rc;
@@ -283,3 +318,4 @@ extern "C" int ra_moe_gemm(const ra::moe::Params* p, void* stream) {
   if (int rc = moe::launch_gemm<true>(*p, s)) return rc;
   return moe::launch_gemm<false>(*p, s);
 }
+

@@ -28,6 +28,73 @@ struct Params {
   long long n_max;             // decode: upper bound of the visible keys
 };
 
+// eight consecutive bf16 numbers (16-byte aligned)
+struct Piece {
+  uint4 u;
+};
+__device__ __forceinline__ Piece load_piece(const __nv_bfloat16* p) { return {*reinterpret_cast<const uint4*>(p)}; }
+__device__ __forceinline__ void unpack(const Piece& s, float (&f)[8]) {
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&s.u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 v = __bfloat1622float2(h[i]);
+    f[2 * i] = v.x;
+    f[2 * i + 1] = v.y;
+  }
+}
+__device__ __forceinline__ Piece pack(const float (&f)[8]) {
+  Piece s;
+  uint32_t* w = reinterpret_cast<uint32_t*>(&s.u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+    w[i] = *reinterpret_cast<const uint32_t*>(&v);
+  }
+  return s;
+}
+__device__ __forceinline__ float square_sum(const Piece& s) {
+  float f[8], a = 0.f;
+  unpack(s, f);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) a += f[e] * f[e];
+  return a;
+}
+// A head's pieces in units: unit u < half / 8 is the pair of pieces u and u + half / 8, which turn; the units after it are
+// pieces u + half / 8 that pass. `lo` (turning units) and `hi` are normed by rs and the gains and turned.
+__device__ __forceinline__ void norm_turn(Piece& lo, Piece& hi, const __nv_bfloat16* gain, float rs, int u, int h8,
+                                          const float* sn, const float* cs) {
+  float x[8], y[8], w[8];
+  unpack(hi, x);
+  unpack(load_piece(gain + (u + h8) * 8), w);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) x[e] *= rs * w[e];
+  if (u < h8) {
+    unpack(lo, y);
+    unpack(load_piece(gain + u * 8), w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float a = y[e] * rs * w[e], s = sn[u * 8 + e], c = cs[u * 8 + e];
+      y[e] = a * c - x[e] * s;
+      x[e] = x[e] * c + a * s;
+    }
+    lo = pack(y);
+  }
+  hi = pack(x);
+}
+// Two sums over the CTA at once; `red` holds 64 floats. Every thread gets the results.
+__device__ __forceinline__ float2 sum_block2(float a, float b, float* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  a = sum_warp(a);
+  b = sum_warp(b);
+  __syncthreads();
+  if (lane == 0) {
+    red[warp] = a;
+    red[32 + warp] = b;
+  }
+  __syncthreads();
+  return make_float2(sum_warp(lane < nw ? red[lane] : 0.f), sum_warp(lane < nw ? red[32 + lane] : 0.f));
+}
+
 int check(const Params* p);  // window_sm100.cu
 
 }  // namespace window

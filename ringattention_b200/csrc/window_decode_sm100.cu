@@ -20,7 +20,7 @@ namespace window {
 
 namespace cg = cooperative_groups;
 
-constexpr int WARPS = 4, THREADS = 128, ST = 3, ROWS = 16;
+constexpr int WARPS = 8, THREADS = 256, ST = 3, ROWS = 16, MAX_CLUSTER = 8;
 
 // D: padded head size of keys and values in shared memory; FULL: more than eight query rows.
 template <int D, bool FULL>
@@ -41,7 +41,7 @@ __global__ void __launch_bounds__(THREADS) window_decode_kernel(const Params p) 
   constexpr int NQ = SM::NQ, TILE = SM::TILE, RB = D * 2, PPR = D / 8, NT = D / 8;
   constexpr float kLog2e = 1.4426950408889634f;
   extern __shared__ __align__(16) uint8_t smem[];
-  __shared__ float red[32], sn[D / 2], cs[D / 2], part_m[NQ + 1], part_l[NQ], warp_m[WARPS][NQ], warp_l[WARPS][NQ];
+  __shared__ float red[64], sn[D / 2], cs[D / 2], part_m[NQ + 1], part_l[NQ], warp_m[WARPS][NQ], warp_l[WARPS][NQ];
   __shared__ float new_s[NQ];
   float* part_o = reinterpret_cast<float*>(smem + SM::OUT_OFF);
   float* new_kv = reinterpret_cast<float*>(smem + SM::NEW_OFF);
@@ -85,60 +85,75 @@ __global__ void __launch_bounds__(THREADS) window_decode_kernel(const Params p) 
     cp_async_commit();
   }
 
-  // ---- norms over the whole projections, sines, this cluster's query rows
-  const int nq = p.H * p.dk, nk = p.G * p.dk, half = p.rot_half;
+  // ---- norms over the whole projections, sines, this cluster's query rows and (first CTA) the new key and value
+  const int nq = p.H * p.dk, nk = p.G * p.dk, half = p.rot_half, h8 = half >> 3;
+  const bool turn8 = !(half & 7);
+  uint8_t* sq_rows = smem + SM::Q_OFF;
   float sq = 0.f, sk = 0.f;
-  for (int i = tid * 8; i < nq; i += THREADS * 8) {
-    const uint4 u = *reinterpret_cast<const uint4*>(x + p.off_q + i);
-    const __nv_bfloat162* hp = reinterpret_cast<const __nv_bfloat162*>(&u);
+  for (int i = tid * 8; i < nq; i += THREADS * 8) sq += square_sum(load_piece(x + p.off_q + i));
+  if (rank == 0)
+    for (int i = tid * 8; i < nk; i += THREADS * 8) sk += square_sum(load_piece(x + p.off_k + i));
+  for (int i = tid; i < half; i += THREADS) sincosf(static_cast<float>(pos) * p.inv_freq[i], &sn[i], &cs[i]);
+  for (int i = tid; i < 16 * PPR; i += THREADS) reinterpret_cast<uint4*>(sq_rows)[i] = make_uint4(0u, 0u, 0u, 0u);
+  for (int i = tid; i < 2 * D; i += THREADS) new_kv[i] = 0.f;
+  const float2 ss = sum_block2(sq, sk, red);
+  const float rq = 1.f / sqrtf(ss.x / nq + p.eps), rk = 1.f / sqrtf(ss.y / nk + p.eps);
+  const bool writer = rank == 0 && blockIdx.y % blocks == 0;
+  const int new_row = static_cast<int>(pos % p.R);
+  // dimensions d .. d + 7 of query head h0 + r, or (r = nh) of the new key
+  auto put = [&](int r, int d, const Piece& v) {
+    if (r < nh) {
+      *reinterpret_cast<uint4*>(sq_rows + r * RB + (((d >> 3) ^ (r & 7)) << 4)) = v.u;
+      return;
+    }
+    float f[8];
+    unpack(v, f);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float2 f = __bfloat1622float2(hp[e]);
-      sq += f.x * f.x + f.y * f.y;
+    for (int e = 0; e < 8; ++e) new_kv[d + e] = f[e];
+    if (writer) *reinterpret_cast<uint4*>(kb + static_cast<long long>(new_row) * p.kw + d) = v.u;
+  };
+  const int heads = rank == 0 ? nh + 1 : nh;
+  if (turn8) {
+    const int units = (p.dk >> 3) - h8;
+    for (int i = tid; i < heads * units; i += THREADS) {
+      const int r = i / units, u = i - r * units;
+      const __nv_bfloat16* src = r < nh ? x + p.off_q + (h0 + r) * p.dk : x + p.off_k + g * p.dk;
+      const __nv_bfloat16* gain = r < nh ? static_cast<const __nv_bfloat16*>(p.q_norm) + (h0 + r) * p.dk
+                                         : static_cast<const __nv_bfloat16*>(p.k_norm) + g * p.dk;
+      Piece hi = load_piece(src + (u + h8) * 8), lo = hi;
+      if (u < h8) lo = load_piece(src + u * 8);
+      norm_turn(lo, hi, gain, r < nh ? rq : rk, u, h8, sn, cs);
+      put(r, (u + h8) * 8, hi);
+      if (u < h8) put(r, u * 8, lo);
+    }
+  } else {  // pairs that do not fall into pieces
+    for (int i = tid; i < heads * (p.dk >> 3); i += THREADS) {
+      const int r = i / (p.dk >> 3), d0 = (i - r * (p.dk >> 3)) * 8;
+      const __nv_bfloat16* src = r < nh ? x + p.off_q + (h0 + r) * p.dk : x + p.off_k + g * p.dk;
+      const __nv_bfloat16* gain = r < nh ? static_cast<const __nv_bfloat16*>(p.q_norm) + (h0 + r) * p.dk
+                                         : static_cast<const __nv_bfloat16*>(p.k_norm) + g * p.dk;
+      const float rs = r < nh ? rq : rk;
+      auto normed = [&](int d) { return __bfloat162float(src[d]) * rs * __bfloat162float(gain[d]); };
+      float f[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int d = d0 + e;
+        f[e] = normed(d);
+        if (d < half) f[e] = f[e] * cs[d] - normed(d + half) * sn[d];
+        else if (d < 2 * half) f[e] = f[e] * cs[d - half] + normed(d - half) * sn[d - half];
+      }
+      put(r, d0, pack(f));
     }
   }
   if (rank == 0)
-    for (int i = tid * 8; i < nk; i += THREADS * 8) {
-      const uint4 u = *reinterpret_cast<const uint4*>(x + p.off_k + i);
-      const __nv_bfloat162* hp = reinterpret_cast<const __nv_bfloat162*>(&u);
+    for (int d = tid * 8; d < p.dv; d += THREADS * 8) {
+      const Piece v = load_piece(x + p.off_v + g * p.dv + d);
+      float f[8];
+      unpack(v, f);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(hp[e]);
-        sk += f.x * f.x + f.y * f.y;
-      }
+      for (int e = 0; e < 8; ++e) new_kv[D + d + e] = f[e];
+      if (writer) *reinterpret_cast<uint4*>(vb + static_cast<long long>(new_row) * p.vw + d) = v.u;
     }
-  for (int i = tid; i < half; i += THREADS) sincosf(static_cast<float>(pos) * p.inv_freq[i], &sn[i], &cs[i]);
-  const float rq = 1.f / sqrtf(sum_block(sq, red) / nq + p.eps);
-  const float rk = 1.f / sqrtf(sum_block(sk, red) / nk + p.eps);
-  // dimension d of a normed and rotated head
-  auto turned = [&](const __nv_bfloat16* src, const __nv_bfloat16* gain, float rs, int d) -> float {
-    const float v = __bfloat162float(src[d]) * rs * __bfloat162float(gain[d]);
-    if (d >= 2 * half) return v;
-    const int o = d < half ? d + half : d - half, i = d < half ? d : o;
-    const float w = __bfloat162float(src[o]) * rs * __bfloat162float(gain[o]);
-    return d < half ? v * cs[i] - w * sn[i] : v * cs[i] + w * sn[i];
-  };
-  uint8_t* sq_rows = smem + SM::Q_OFF;
-  for (int i = tid; i < 16 * D; i += THREADS) {
-    const int r = i / D, d = i % D;
-    float v = 0.f;
-    if (r < nh && d < p.dk)
-      v = turned(x + p.off_q + (h0 + r) * p.dk, static_cast<const __nv_bfloat16*>(p.q_norm) + (h0 + r) * p.dk, rq, d);
-    *reinterpret_cast<__nv_bfloat16*>(sq_rows + r * RB + (((d >> 3) ^ (r & 7)) << 4) + (d & 7) * 2) = __float2bfloat16(v);
-  }
-  if (rank == 0) {
-    const bool writer = blockIdx.y % blocks == 0;
-    const int r = static_cast<int>(pos % p.R);
-    for (int d = tid; d < D; d += THREADS) {
-      const __nv_bfloat16 kv = __float2bfloat16(
-          d < p.dk ? turned(x + p.off_k + g * p.dk, static_cast<const __nv_bfloat16*>(p.k_norm) + g * p.dk, rk, d) : 0.f);
-      const __nv_bfloat16 vv = d < p.dv ? x[p.off_v + g * p.dv + d] : __float2bfloat16(0.f);
-      new_kv[d] = __bfloat162float(kv);
-      new_kv[D + d] = __bfloat162float(vv);
-      if (writer && d < p.dk) kb[static_cast<long long>(r) * p.kw + d] = kv;
-      if (writer && d < p.dv) vb[static_cast<long long>(r) * p.vw + d] = vv;
-    }
-  }
   __syncthreads();
   if (rank == 0) {  // the new token's own score, one head a warp at a time
     for (int r = warp; r < nh; r += WARPS) {
@@ -302,14 +317,25 @@ __global__ void __launch_bounds__(THREADS) window_decode_kernel(const Params p) 
   for (int i = rank * THREADS + tid; i < nh * p.dv; i += C * THREADS) {
     const int r = i / p.dv, d = i - r * p.dv;
     const float s = p.sink[h0 + r] * kLog2e;
-    float mx = s;
-    for (int c = 0; c < C; ++c) mx = fmaxf(mx, cluster.map_shared_rank(part_m, c)[r]);
-    float lt = exp2f(s - mx), ot = 0.f;
-    for (int c = 0; c < C; ++c) {
-      const float a = exp2f(cluster.map_shared_rank(part_m, c)[r] - mx);
-      lt += cluster.map_shared_rank(part_l, c)[r] * a;
-      ot += cluster.map_shared_rank(part_o, c)[r * D + d] * a;
+    float pm[MAX_CLUSTER], pl[MAX_CLUSTER], po[MAX_CLUSTER], mx = s;
+#pragma unroll
+    for (int c = 0; c < MAX_CLUSTER; ++c) {  // all reads of other CTAs' shared memory on their way at once
+      const int cc = c < C ? c : 0;
+      pm[c] = cluster.map_shared_rank(part_m, cc)[r];
+      pl[c] = cluster.map_shared_rank(part_l, cc)[r];
+      po[c] = cluster.map_shared_rank(part_o, cc)[r * D + d];
     }
+#pragma unroll
+    for (int c = 0; c < MAX_CLUSTER; ++c)
+      if (c < C) mx = fmaxf(mx, pm[c]);
+    float lt = exp2f(s - mx), ot = 0.f;
+#pragma unroll
+    for (int c = 0; c < MAX_CLUSTER; ++c)
+      if (c < C) {
+        const float a = exp2f(pm[c] - mx);
+        lt += pl[c] * a;
+        ot += po[c] * a;
+      }
     if (RA_IN_BOUNDS(h0 * p.dv + i, 1, p.ldo, kTagWindow)) out[i] = __float2bfloat16(ot / lt);
   }
   cluster.sync();  // nobody's shared memory goes away while it is read
@@ -362,7 +388,7 @@ extern "C" int ra_window_decode(const ra::window::Params* pp, void* stream) {
   const int share = p.H / p.G, nq = share > 8 ? 16 : 8;
   const long long work = static_cast<long long>(p.G) * ((share + nq - 1) / nq) * p.B;
   const long long keys = p.n_max < p.window ? p.n_max : p.window;
-  int c = 8;  // CTAs of a cluster: enough for the machine, at least 64 keys each
+  int c = MAX_CLUSTER;  // CTAs of a cluster: enough for the machine, at least 32 keys each
   while (c > 1 && (work * c > 2 * sm_count() || keys < 32ll * c)) c >>= 1;
   p.splits = c;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

@@ -1,7 +1,7 @@
 // Attention over a sliding window with grouped key/value heads, a sink per head, RMS norms over the whole query and key
 // projections and rotary positions on the first dimensions of a head:
-//   window_prep_kernel   : norms, rotation (queries in place) and the new rows of the key/value ring. One CTA per token; in
-//                          16-byte pieces where the sizes allow it.
+//   window_prep_kernel, window_prep_pieces_kernel : norms, rotation (queries in place) and the new rows of the key/value
+//                          ring. One CTA per token; bf16 in 16-byte pieces where the sizes allow it, a row read once.
 //   window_attend_kernel : one warp per (token, head) on the CUDA cores; any sizes, bf16 or fp32 throughout. bf16 prompts of
 //                          the common sizes run on the tensor cores (attn_fwd_sm100.cu), single tokens in
 //                          window_decode_sm100.cu.
@@ -15,42 +15,64 @@ namespace window {
 constexpr int PREP_THREADS = 256;
 constexpr int MAX_HALF = 256;
 
-template <typename T>
-__device__ __forceinline__ void load8(const T* p, float (&f)[8]) {
-  const float4 a = load4(p), b = load4(p + 4);
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
-template <>
-__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&f)[8]) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+// bf16, head sizes and rot_half multiples of eight. NI: units of query and key heads per thread.
+template <int NI>
+__global__ void __launch_bounds__(PREP_THREADS) window_prep_pieces_kernel(const Params p) {
+  __shared__ float red[64], sn[MAX_HALF], cs[MAX_HALF];
+  const long long row = blockIdx.x;
+  const int b = static_cast<int>(row / p.T), t = static_cast<int>(row - static_cast<long long>(b) * p.T), tid = threadIdx.x;
+  __nv_bfloat16* x = static_cast<__nv_bfloat16*>(p.proj) + row * p.ldp;
+  const int h8 = p.rot_half >> 3, units = (p.dk >> 3) - h8, n = (p.H + p.G) * units, v8 = p.dv >> 3;
+  Piece lo[NI], hi[NI], val;
+  float sq = 0.f, sk = 0.f;
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float2 v = __bfloat1622float2(h[i]);
-    f[2 * i] = v.x;
-    f[2 * i + 1] = v.y;
+  for (int j = 0; j < NI; ++j) {
+    const int i = tid + j * PREP_THREADS, head = i / units, u = i - head * units;
+    if (i >= n) continue;
+    const __nv_bfloat16* src = head < p.H ? x + p.off_q + head * p.dk : x + p.off_k + (head - p.H) * p.dk;
+    hi[j] = load_piece(src + (u + h8) * 8);
+    if (u < h8) lo[j] = load_piece(src + u * 8);
   }
-}
-__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
-  store4(p, make_float4(f[0], f[1], f[2], f[3]));
-  store4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
-}
-__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
-  uint4 u;
-  uint32_t* w = reinterpret_cast<uint32_t*>(&u);
+  if (tid < p.G * v8) val = load_piece(x + p.off_v + tid * 8);
+  const long long pos = *p.pos + t;
+  const int r = static_cast<int>(pos % p.R);
+  for (int i = tid; i < p.rot_half; i += PREP_THREADS)
+    sincosf(static_cast<float>(pos) * p.inv_freq[i], &sn[i], &cs[i]);
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
-    w[i] = *reinterpret_cast<const uint32_t*>(&v);
+  for (int j = 0; j < NI; ++j) {
+    const int i = tid + j * PREP_THREADS, head = i / units, u = i - head * units;
+    if (i >= n) continue;
+    const float s = square_sum(hi[j]) + (u < h8 ? square_sum(lo[j]) : 0.f);
+    if (head < p.H) sq += s;
+    else sk += s;
   }
-  *reinterpret_cast<uint4*>(p) = u;
+  const float2 ss = sum_block2(sq, sk, red);  // its barriers also cover the sines
+  const float rq = 1.f / sqrtf(ss.x / (p.H * p.dk) + p.eps), rk = 1.f / sqrtf(ss.y / (p.G * p.dk) + p.eps);
+  if (!RA_IN_BOUNDS(row, 1, static_cast<long long>(p.B) * p.T, kTagWindow)) return;
+  __nv_bfloat16* kc = static_cast<__nv_bfloat16*>(p.k_cache) + (static_cast<long long>(b) * p.G * p.R + r) * p.kw;
+  __nv_bfloat16* vc = static_cast<__nv_bfloat16*>(p.v_cache) + (static_cast<long long>(b) * p.G * p.R + r) * p.vw;
+#pragma unroll
+  for (int j = 0; j < NI; ++j) {
+    const int i = tid + j * PREP_THREADS, head = i / units, u = i - head * units;
+    if (i >= n) continue;
+    const bool is_q = head < p.H;
+    const int hh = is_q ? head : head - p.H;
+    norm_turn(lo[j], hi[j], static_cast<const __nv_bfloat16*>(is_q ? p.q_norm : p.k_norm) + hh * p.dk, is_q ? rq : rk, u, h8,
+              sn, cs);
+    __nv_bfloat16* dst = is_q ? x + p.off_q + hh * p.dk : kc + static_cast<long long>(hh) * p.R * p.kw;
+    *reinterpret_cast<uint4*>(dst + (u + h8) * 8) = hi[j].u;
+    if (u < h8) *reinterpret_cast<uint4*>(dst + u * 8) = lo[j].u;
+  }
+  for (int i = tid; i < p.G * v8; i += PREP_THREADS) {
+    const int g = i / v8, u = i - g * v8;
+    if (i != tid) val = load_piece(x + p.off_v + i * 8);
+    *reinterpret_cast<uint4*>(vc + static_cast<long long>(g) * p.R * p.vw + u * 8) = val.u;
+  }
 }
 
-// VEC: head sizes and rot_half are multiples of eight.
-template <typename T, bool VEC>
+template <typename T>
 __global__ void __launch_bounds__(PREP_THREADS) window_prep_kernel(const Params p) {
-  __shared__ float red[32], sn[MAX_HALF], cs[MAX_HALF];
+  __shared__ float red[64], sn[MAX_HALF], cs[MAX_HALF];
   const long long row = blockIdx.x;
   const int b = static_cast<int>(row / p.T), t = static_cast<int>(row - static_cast<long long>(b) * p.T);
   const long long pos = *p.pos + t;
@@ -64,65 +86,11 @@ __global__ void __launch_bounds__(PREP_THREADS) window_prep_kernel(const Params 
   const int nq = p.H * p.dk, nk = p.G * p.dk, half = p.rot_half;
   for (int i = tid; i < half; i += PREP_THREADS) sincosf(static_cast<float>(pos) * p.inv_freq[i], &sn[i], &cs[i]);
   float sq = 0.f, sk = 0.f;
-  if (VEC) {
-    for (int i = tid * 8; i < nq; i += PREP_THREADS * 8) {
-      float f[8];
-      load8(q + i, f);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) sq += f[e] * f[e];
-    }
-    for (int i = tid * 8; i < nk; i += PREP_THREADS * 8) {
-      float f[8];
-      load8(k + i, f);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) sk += f[e] * f[e];
-    }
-  } else {
-    for (int i = tid; i < nq; i += PREP_THREADS) sq += to_f(q[i]) * to_f(q[i]);
-    for (int i = tid; i < nk; i += PREP_THREADS) sk += to_f(k[i]) * to_f(k[i]);
-  }
-  const float rq = 1.f / sqrtf(sum_block(sq, red) / nq + p.eps);
-  const float rk = 1.f / sqrtf(sum_block(sk, red) / nk + p.eps);  // its barriers also cover the sines
+  for (int i = tid; i < nq; i += PREP_THREADS) sq += to_f(q[i]) * to_f(q[i]);
+  for (int i = tid; i < nk; i += PREP_THREADS) sk += to_f(k[i]) * to_f(k[i]);
+  const float2 ss = sum_block2(sq, sk, red);  // its barriers also cover the sines
+  const float rq = 1.f / sqrtf(ss.x / nq + p.eps), rk = 1.f / sqrtf(ss.y / nk + p.eps);
   if (!RA_IN_BOUNDS(row, 1, static_cast<long long>(p.B) * p.T, kTagWindow)) return;
-  if (VEC) {
-    const int h8 = half >> 3, units = (p.dk >> 3) - h8;  // a unit turns pieces u and u + h8, or copies piece u + h8
-    for (int i = tid; i < (p.H + p.G) * units; i += PREP_THREADS) {
-      const int head = i / units, u = i - head * units;
-      const bool is_q = head < p.H;
-      const int hh = is_q ? head : head - p.H;
-      const T* src = is_q ? q + hh * p.dk : k + hh * p.dk;
-      const T* gain = is_q ? qw + hh * p.dk : kw + hh * p.dk;
-      T* dst = is_q ? q + hh * p.dk : kc + static_cast<long long>(hh) * p.R * p.kw;
-      const float rs = is_q ? rq : rk;
-      float x[8], w[8];
-      const int hi = (u + h8) * 8;
-      load8(src + hi, x);
-      load8(gain + hi, w);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] *= rs * w[e];
-      if (u < h8) {
-        float y[8];
-        load8(src + u * 8, y);
-        load8(gain + u * 8, w);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float a = y[e] * rs * w[e], s = sn[u * 8 + e], c = cs[u * 8 + e];
-          y[e] = a * c - x[e] * s;
-          x[e] = x[e] * c + a * s;
-        }
-        store8(dst + u * 8, y);
-      }
-      store8(dst + hi, x);
-    }
-    const int v8 = p.dv >> 3;
-    for (int i = tid; i < p.G * v8; i += PREP_THREADS) {
-      const int g = i / v8, u = i - g * v8;
-      float x[8];
-      load8(v + g * p.dv + u * 8, x);
-      store8(vc + static_cast<long long>(g) * p.R * p.vw + u * 8, x);
-    }
-    return;
-  }
   const int rest = p.dk - 2 * half, per = half + rest;  // pairs, then dimensions that pass
   for (int i = tid; i < (p.H + p.G) * per; i += PREP_THREADS) {
     const int head = i / per, u = i - head * per;
@@ -234,11 +202,13 @@ extern "C" int ra_window_prep(const ra::window::Params* p, int f32, void* stream
   if (const int rc = window::check(p)) return rc;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int rows = p->B * p->T;
-  const bool vec = !(p->dk % 8 || p->dv % 8 || p->rot_half % 8);
-  if (f32 && vec) window::window_prep_kernel<float, true><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else if (f32) window::window_prep_kernel<float, false><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else if (vec) window::window_prep_kernel<__nv_bfloat16, true><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else window::window_prep_kernel<__nv_bfloat16, false><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  const int units = (p->H + p->G) * ((p->dk - p->rot_half) / 8);
+  if (f32) window::window_prep_kernel<float><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else if (p->dk % 8 || p->dv % 8 || p->rot_half % 8 || units > 4 * window::PREP_THREADS)
+    window::window_prep_kernel<__nv_bfloat16><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else if (units <= window::PREP_THREADS) window::window_prep_pieces_kernel<1><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else if (units <= 2 * window::PREP_THREADS) window::window_prep_pieces_kernel<2><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else window::window_prep_pieces_kernel<4><<<rows, window::PREP_THREADS, 0, s>>>(*p);
   return check_launch("window_prep_kernel");
 }
 

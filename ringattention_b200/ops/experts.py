@@ -50,7 +50,8 @@ def moe_(x, h, d: int, m, w) -> None:
         return _lib.call("ra_moe_few", ctypes.byref(a), int(f32), _lib.stream_ptr(), n_kernels=2)
     count = torch.zeros(m.experts, device=dev, dtype=torch.int32)
     lists = torch.empty(m.experts, rows, device=dev, dtype=torch.int32)
-    act = torch.empty(rows * m.top, F, device=dev, dtype=h.dtype)
+    n = rows * m.top
+    act = torch.empty(128 * (n // 128 + min(n, m.experts)), F, device=dev, dtype=h.dtype)  # row tiles expert by expert
     y = torch.empty(rows * m.top, dp, device=dev, dtype=h.dtype)
     a.count, a.list, a.act, a.y = p(count), p(lists), p(act), p(y)
     _lib.call("ra_moe_route", ctypes.byref(a), _lib.stream_ptr())
