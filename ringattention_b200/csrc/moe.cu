@@ -27,23 +27,43 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
     f[2 * i + 1] = v.y;
   }
 }
-// dot product of n (multiple of 8) elements of w with x in shared memory, over the lanes of the warp
-template <typename T>
-__device__ __forceinline__ float dot_lane(const T* w, const float* x, int n) {
-  const int lane = threadIdx.x & 31;
-  float acc = 0.f;
-#pragma unroll 4
-  for (int i = lane * 8; i < n; i += 256) {
-    float a[8], b[8];
-    load8(w + i, a);
-    load8(x + i, b);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) acc = fmaf(a[e], b[e], acc);
+// eight elements as they lie in memory: weights are loaded a batch ahead of the arithmetic
+template <typename T> struct Raw8;
+template <> struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = load4(p); b = load4(p + 4); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
   }
-  return acc;
+};
+template <> struct Raw8<__nv_bfloat16> {
+  uint4 u;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { u = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 v = __bfloat1622float2(h[i]);
+      f[2 * i] = v.x;
+      f[2 * i + 1] = v.y;
+    }
+  }
+};
+template <typename T>
+__device__ __forceinline__ void dot2(const Raw8<T>& w0, const Raw8<T>& w1, const float* x, float& a0, float& a1) {
+  float f0[8], f1[8], v[8];
+  w0.get(f0);
+  w1.get(f1);
+  load8(x, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    a0 = fmaf(f0[e], v[e], a0);
+    a1 = fmaf(f1[e], v[e], a1);
+  }
 }
 
-constexpr int FEW_THREADS = 256, FEW_WARPS = 8;
+constexpr int FEW_THREADS = 256, FEW_WARPS = 8, BATCH = 4;
 
 // grid (chunks of the outputs, rows)
 template <typename T>
@@ -85,17 +105,17 @@ __global__ void __launch_bounds__(FEW_THREADS) moe_gateup_kernel(const Params p)
                         : static_cast<const T*>(p.sh_gu) + static_cast<long long>(f) * p.dp;
     const T* u = g + static_cast<long long>(F) * p.dp;
     float a = 0.f, c = 0.f;
-#pragma unroll 4
-    for (int i = lane * 8; i < p.dp; i += 256) {
-      float wg[8], wu[8], xv[8];
-      load8(g + i, wg);
-      load8(u + i, wu);
-      load8(sx + i, xv);
+    for (int i0 = lane * 8; i0 < p.dp; i0 += 256 * BATCH) {
+      Raw8<T> wg[BATCH], wu[BATCH];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        a = fmaf(wg[e], xv[e], a);
-        c = fmaf(wu[e], xv[e], c);
-      }
+      for (int j = 0; j < BATCH; ++j)
+        if (i0 + 256 * j < p.dp) {
+          wg[j].load(g + i0 + 256 * j);
+          wu[j].load(u + i0 + 256 * j);
+        }
+#pragma unroll
+      for (int j = 0; j < BATCH; ++j)
+        if (i0 + 256 * j < p.dp) dot2(wg[j], wu[j], sx + i0 + 256 * j, a, c);
     }
     const float w = routed ? s_w[s] : 1.f;
     a = sum_warp(a) * w;
@@ -104,15 +124,18 @@ __global__ void __launch_bounds__(FEW_THREADS) moe_gateup_kernel(const Params p)
   }
 }
 
-constexpr int DOWN_COLS = 2;  // columns per warp
+constexpr int DOWN_COLS = 2;  // columns per warp, side by side
 
-// grid (chunks of the columns, rows): x[row] += sum over the experts of W_down act
+// grid (chunks of the columns, rows): x[row] += sum over the experts of W_down act. A lane's pieces run through the experts'
+// rows one after the other, so that several experts' weights are on their way at once.
 template <typename T>
 __global__ void __launch_bounds__(FEW_THREADS) moe_down_kernel(const Params p) {
   extern __shared__ __align__(16) float sm_few[];  // [top * F + Fs]
+  __shared__ const T* s_base[MAX_TOP];
   const int row = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int n_in = p.top * p.F + p.Fs;
   const T* act = static_cast<const T*>(p.act) + static_cast<long long>(row) * n_in;
+  if (tid < p.top) s_base[tid] = static_cast<const T*>(p.down) + static_cast<long long>(p.ids[row * p.top + tid]) * p.dp * p.F;
   for (int i = tid * 8; i < n_in; i += FEW_THREADS * 8) {
     float f[8];
     load8(act + i, f);
@@ -120,19 +143,32 @@ __global__ void __launch_bounds__(FEW_THREADS) moe_down_kernel(const Params p) {
     store4(sm_few + i + 4, make_float4(f[4], f[5], f[6], f[7]));
   }
   __syncthreads();
-  const int* ids = p.ids + row * p.top;
-#pragma unroll 1
-  for (int j = 0; j < DOWN_COLS; ++j) {
-    const int c = (blockIdx.x * DOWN_COLS + j) * FEW_WARPS + warp;
-    if (c >= p.d) break;
-    float acc = 0.f;
-    for (int s = 0; s < p.top; ++s)
-      acc += dot_lane(static_cast<const T*>(p.down) + (static_cast<long long>(ids[s]) * p.dp + c) * p.F, sm_few + s * p.F, p.F);
-    if (p.Fs)
-      acc += dot_lane(static_cast<const T*>(p.sh_down) + static_cast<long long>(c) * p.Fs, sm_few + p.top * p.F, p.Fs);
-    acc = sum_warp(acc);
-    if (lane == 0 && RA_IN_BOUNDS(c, 1, p.ldx, kTagMoe)) p.x[row * p.ldx + c] += acc;
+  const int c0 = (blockIdx.x * FEW_WARPS + warp) * DOWN_COLS;
+  if (c0 >= p.d) return;
+  const int c1 = min(c0 + 1, p.d - 1), F8 = p.F >> 3, routed = p.top * F8, pieces = n_in >> 3;
+  float a0 = 0.f, a1 = 0.f;
+  for (int q0 = lane; q0 < pieces; q0 += 32 * BATCH) {
+    Raw8<T> w0[BATCH], w1[BATCH];
+#pragma unroll
+    for (int j = 0; j < BATCH; ++j) {
+      const int q = q0 + 32 * j;
+      if (q >= pieces) continue;
+      const int s = q / F8;
+      const bool in = q < routed;
+      const T* base = in ? s_base[s] : static_cast<const T*>(p.sh_down);
+      const long long ld = in ? p.F : p.Fs;
+      const int i = (in ? q - s * F8 : q - routed) * 8;
+      w0[j].load(base + c0 * ld + i);
+      w1[j].load(base + c1 * ld + i);
+    }
+#pragma unroll
+    for (int j = 0; j < BATCH; ++j)
+      if (q0 + 32 * j < pieces) dot2(w0[j], w1[j], sm_few + (q0 + 32 * j) * 8, a0, a1);
   }
+  a0 = sum_warp(a0);
+  a1 = sum_warp(a1);
+  if (lane < DOWN_COLS && c0 + lane < p.d && RA_IN_BOUNDS(c0 + lane, 1, p.ldx, kTagMoe))
+    p.x[row * p.ldx + c0 + lane] += lane ? a1 : a0;
 }
 
 constexpr int ROUTE_TOKENS = 32, ROUTE_WARPS = 8;  // tokens per CTA
@@ -219,9 +255,10 @@ int launch_few(const Params& p, cudaStream_t s) {
   const size_t smem1 = 4 * (static_cast<size_t>(p.dp) + p.E), smem2 = 4 * static_cast<size_t>(n);
   if (int rc = shared_memory(moe_gateup_kernel<T>, smem1)) return rc;
   if (int rc = shared_memory(moe_down_kernel<T>, smem2)) return rc;
-  // a CTA loads the row and chooses before it streams weights: not more CTAs than fit at once, a few outputs per warp
-  const int want = (n + FEW_WARPS - 1) / FEW_WARPS, fit = (4 * sm_count() + p.rows - 1) / p.rows;
-  moe_gateup_kernel<T><<<dim3(want < fit ? want : fit, p.rows), FEW_THREADS, smem1, s>>>(p);
+  // a CTA loads the row and chooses before it streams weights: not more CTAs than fit at once, equally many outputs each
+  const int want = (n + FEW_WARPS - 1) / FEW_WARPS, fit = (5 * sm_count() + p.rows - 1) / p.rows;
+  const int rounds = (want + fit - 1) / fit;
+  moe_gateup_kernel<T><<<dim3((want + rounds - 1) / rounds, p.rows), FEW_THREADS, smem1, s>>>(p);
   if (int rc = check_launch("moe_gateup_kernel")) return rc;
   const int per = DOWN_COLS * FEW_WARPS;
   moe_down_kernel<T><<<dim3((p.d + per - 1) / per, p.rows), FEW_THREADS, smem2, s>>>(p);

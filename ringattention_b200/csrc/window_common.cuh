@@ -60,22 +60,25 @@ __device__ __forceinline__ float square_sum(const Piece& s) {
   return a;
 }
 // A head's pieces in units: unit u < half / 8 is the pair of pieces u and u + half / 8, which turn; the units after it are
-// pieces u + half / 8 that pass. `lo` (turning units) and `hi` are normed by rs and the gains and turned.
-__device__ __forceinline__ void norm_turn(Piece& lo, Piece& hi, const __nv_bfloat16* gain, float rs, int u, int h8,
-                                          const float* sn, const float* cs) {
-  float x[8], y[8], w[8];
+// pieces u + half / 8 that pass. `lo` (turning units) and `hi` are normed by rs and the gains gl and gh, and turned.
+__device__ __forceinline__ void norm_turn(Piece& lo, Piece& hi, const float (&gl)[8], const float (&gh)[8], float rs, int u,
+                                          int h8, const float* sn, const float* cs) {
+  float x[8], y[8];
   unpack(hi, x);
-  unpack(load_piece(gain + (u + h8) * 8), w);
 #pragma unroll
-  for (int e = 0; e < 8; ++e) x[e] *= rs * w[e];
+  for (int e = 0; e < 8; ++e) x[e] *= rs * gh[e];
   if (u < h8) {
     unpack(lo, y);
-    unpack(load_piece(gain + u * 8), w);
+    float s[8], c[8];
+    *reinterpret_cast<float4*>(s) = load4(sn + u * 8);
+    *reinterpret_cast<float4*>(s + 4) = load4(sn + u * 8 + 4);
+    *reinterpret_cast<float4*>(c) = load4(cs + u * 8);
+    *reinterpret_cast<float4*>(c + 4) = load4(cs + u * 8 + 4);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      const float a = y[e] * rs * w[e], s = sn[u * 8 + e], c = cs[u * 8 + e];
-      y[e] = a * c - x[e] * s;
-      x[e] = x[e] * c + a * s;
+      const float a = y[e] * rs * gl[e];
+      y[e] = a * c[e] - x[e] * s[e];
+      x[e] = x[e] * c[e] + a * s[e];
     }
     lo = pack(y);
   }

@@ -41,7 +41,8 @@ __global__ void __launch_bounds__(THREADS) window_decode_kernel(const Params p) 
   constexpr int NQ = SM::NQ, TILE = SM::TILE, RB = D * 2, PPR = D / 8, NT = D / 8;
   constexpr float kLog2e = 1.4426950408889634f;
   extern __shared__ __align__(16) uint8_t smem[];
-  __shared__ float red[64], sn[D / 2], cs[D / 2], part_m[NQ + 1], part_l[NQ], warp_m[WARPS][NQ], warp_l[WARPS][NQ];
+  __shared__ __align__(16) float sn[D / 2], cs[D / 2];
+  __shared__ float red[64], part_m[NQ + 1], part_l[NQ], warp_m[WARPS][NQ], warp_l[WARPS][NQ];
   __shared__ float new_s[NQ];
   float* part_o = reinterpret_cast<float*>(smem + SM::OUT_OFF);
   float* new_kv = reinterpret_cast<float*>(smem + SM::NEW_OFF);
@@ -122,7 +123,10 @@ __global__ void __launch_bounds__(THREADS) window_decode_kernel(const Params p) 
                                          : static_cast<const __nv_bfloat16*>(p.k_norm) + g * p.dk;
       Piece hi = load_piece(src + (u + h8) * 8), lo = hi;
       if (u < h8) lo = load_piece(src + u * 8);
-      norm_turn(lo, hi, gain, r < nh ? rq : rk, u, h8, sn, cs);
+      float gl[8], gh[8];
+      unpack(load_piece(gain + (u + h8) * 8), gh);
+      if (u < h8) unpack(load_piece(gain + u * 8), gl);
+      norm_turn(lo, hi, gl, gh, r < nh ? rq : rk, u, h8, sn, cs);
       put(r, (u + h8) * 8, hi);
       if (u < h8) put(r, u * 8, lo);
     }
@@ -386,13 +390,14 @@ extern "C" int ra_window_decode(const ra::window::Params* pp, void* stream) {
     return kHostBadArg;
   }
   const int share = p.H / p.G, nq = share > 8 ? 16 : 8;
+  const bool small = p.dk <= 64 && p.dv <= 64;
   const long long work = static_cast<long long>(p.G) * ((share + nq - 1) / nq) * p.B;
   const long long keys = p.n_max < p.window ? p.n_max : p.window;
-  int c = MAX_CLUSTER;  // CTAs of a cluster: enough for the machine, at least 32 keys each
-  while (c > 1 && (work * c > 2 * sm_count() || keys < 32ll * c)) c >>= 1;
+  const long long fit = static_cast<long long>(sm_count()) * (small ? 2 : 1);  // CTAs that run at once
+  int c = MAX_CLUSTER;  // CTAs of a cluster: as many as run at once, at least 32 keys each
+  while (c > 1 && (work * c > fit || keys < 32ll * c)) c >>= 1;
   p.splits = c;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool small = p.dk <= 64 && p.dv <= 64;
   if (nq == 8) return small ? launch_decode<64, false>(p, s) : launch_decode<128, false>(p, s);
   return small ? launch_decode<64, true>(p, s) : launch_decode<128, true>(p, s);
 }

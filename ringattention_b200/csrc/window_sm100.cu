@@ -13,61 +13,103 @@ namespace ra {
 namespace window {
 
 constexpr int PREP_THREADS = 256;
-constexpr int MAX_HALF = 256;
+constexpr int MAX_HALF = 256;  // (dk <= 512)
 
-// bf16, head sizes and rot_half multiples of eight. NI: units of query and key heads per thread.
-template <int NI>
-__global__ void __launch_bounds__(PREP_THREADS) window_prep_pieces_kernel(const Params p) {
-  __shared__ float red[64], sn[MAX_HALF], cs[MAX_HALF];
-  const long long row = blockIdx.x;
-  const int b = static_cast<int>(row / p.T), t = static_cast<int>(row - static_cast<long long>(b) * p.T), tid = threadIdx.x;
-  __nv_bfloat16* x = static_cast<__nv_bfloat16*>(p.proj) + row * p.ldp;
+// bf16, head sizes and rot_half multiples of eight. A CTA takes NROW consecutive tokens of a sequence, a thread the same NI
+// units of query and key heads of each: the kernel is bound by its instructions, and index arithmetic and gains serve all
+// rows. grid (tokens / NROW, sequences).
+template <int NI, int NROW>
+__global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pieces_kernel(const Params p) {
+  __shared__ __align__(16) float red[2 * NROW][8], sn[NROW][MAX_HALF], cs[NROW][MAX_HALF];
+  const int b = blockIdx.y, t0 = blockIdx.x * NROW, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rows = min(NROW, p.T - t0);
+  __nv_bfloat16* x = static_cast<__nv_bfloat16*>(p.proj) + (static_cast<long long>(b) * p.T + t0) * p.ldp;
   const int h8 = p.rot_half >> 3, units = (p.dk >> 3) - h8, n = (p.H + p.G) * units, v8 = p.dv >> 3;
-  Piece lo[NI], hi[NI], val;
-  float sq = 0.f, sk = 0.f;
+  Piece lo[NI][NROW], hi[NI][NROW];
+  int at[NI], unit[NI];  // first dimension of the thread's heads, query heads first; unit, or -1
+  float s[2 * NROW];
+#pragma unroll
+  for (int e = 0; e < 2 * NROW; ++e) s[e] = 0.f;
 #pragma unroll
   for (int j = 0; j < NI; ++j) {
-    const int i = tid + j * PREP_THREADS, head = i / units, u = i - head * units;
-    if (i >= n) continue;
-    const __nv_bfloat16* src = head < p.H ? x + p.off_q + head * p.dk : x + p.off_k + (head - p.H) * p.dk;
-    hi[j] = load_piece(src + (u + h8) * 8);
-    if (u < h8) lo[j] = load_piece(src + u * 8);
+    const int i = tid + j * PREP_THREADS, head = i / units;
+    unit[j] = i < n ? i - head * units : -1;
+    at[j] = head * p.dk;
+    const __nv_bfloat16* src = x + (head < p.H ? p.off_q : p.off_k - p.H * p.dk) + at[j];
+#pragma unroll
+    for (int r = 0; r < NROW; ++r)
+      if (unit[j] >= 0 && r < rows) {
+        hi[j][r] = load_piece(src + r * p.ldp + (unit[j] + h8) * 8);
+        if (unit[j] < h8) lo[j][r] = load_piece(src + r * p.ldp + unit[j] * 8);
+      }
   }
-  if (tid < p.G * v8) val = load_piece(x + p.off_v + tid * 8);
-  const long long pos = *p.pos + t;
-  const int r = static_cast<int>(pos % p.R);
-  for (int i = tid; i < p.rot_half; i += PREP_THREADS)
-    sincosf(static_cast<float>(pos) * p.inv_freq[i], &sn[i], &cs[i]);
-#pragma unroll
-  for (int j = 0; j < NI; ++j) {
-    const int i = tid + j * PREP_THREADS, head = i / units, u = i - head * units;
-    if (i >= n) continue;
-    const float s = square_sum(hi[j]) + (u < h8 ? square_sum(lo[j]) : 0.f);
-    if (head < p.H) sq += s;
-    else sk += s;
+  const long long pos = *p.pos + t0;
+  for (int i = tid; i < rows * p.rot_half; i += PREP_THREADS) {
+    const int r = i / p.rot_half, e = i - r * p.rot_half;
+    sincosf(static_cast<float>(pos + r) * p.inv_freq[e], &sn[r][e], &cs[r][e]);
   }
-  const float2 ss = sum_block2(sq, sk, red);  // its barriers also cover the sines
-  const float rq = 1.f / sqrtf(ss.x / (p.H * p.dk) + p.eps), rk = 1.f / sqrtf(ss.y / (p.G * p.dk) + p.eps);
-  if (!RA_IN_BOUNDS(row, 1, static_cast<long long>(p.B) * p.T, kTagWindow)) return;
-  __nv_bfloat16* kc = static_cast<__nv_bfloat16*>(p.k_cache) + (static_cast<long long>(b) * p.G * p.R + r) * p.kw;
-  __nv_bfloat16* vc = static_cast<__nv_bfloat16*>(p.v_cache) + (static_cast<long long>(b) * p.G * p.R + r) * p.vw;
+#pragma unroll
+  for (int j = 0; j < NI; ++j)
+#pragma unroll
+    for (int r = 0; r < NROW; ++r)
+      if (unit[j] >= 0 && r < rows) {
+        const float v = square_sum(hi[j][r]) + (unit[j] < h8 ? square_sum(lo[j][r]) : 0.f);
+        s[2 * r] += at[j] < p.H * p.dk ? v : 0.f;
+        s[2 * r + 1] += at[j] < p.H * p.dk ? 0.f : v;
+      }
+#pragma unroll
+  for (int e = 0; e < 2 * NROW; ++e) {
+    s[e] = sum_warp(s[e]);
+    if (lane == 0) red[e][warp] = s[e];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int e = 0; e < 2 * NROW; ++e) {
+    const float4 u = load4(red[e]), w = load4(red[e] + 4);
+    const float sum = ((u.x + u.y) + (u.z + u.w)) + ((w.x + w.y) + (w.z + w.w));
+    s[e] = 1.f / sqrtf(sum / (e & 1 ? p.G * p.dk : p.H * p.dk) + p.eps);
+  }
+  if (!RA_IN_BOUNDS(t0, rows, p.T, kTagWindow)) return;
+  const int ring0 = static_cast<int>(static_cast<unsigned>(pos) % static_cast<unsigned>(p.R));
+  auto ring_row = [&](int r) { return ring0 + r >= p.R ? ring0 + r - p.R : ring0 + r; };
+  __nv_bfloat16* kc = static_cast<__nv_bfloat16*>(p.k_cache) + static_cast<long long>(b) * p.G * p.R * p.kw;
+  __nv_bfloat16* vc = static_cast<__nv_bfloat16*>(p.v_cache) + static_cast<long long>(b) * p.G * p.R * p.vw;
 #pragma unroll
   for (int j = 0; j < NI; ++j) {
-    const int i = tid + j * PREP_THREADS, head = i / units, u = i - head * units;
-    if (i >= n) continue;
+    if (unit[j] < 0) continue;
+    const int u = unit[j], head = at[j] / p.dk;
     const bool is_q = head < p.H;
-    const int hh = is_q ? head : head - p.H;
-    norm_turn(lo[j], hi[j], static_cast<const __nv_bfloat16*>(is_q ? p.q_norm : p.k_norm) + hh * p.dk, is_q ? rq : rk, u, h8,
-              sn, cs);
-    __nv_bfloat16* dst = is_q ? x + p.off_q + hh * p.dk : kc + static_cast<long long>(hh) * p.R * p.kw;
-    *reinterpret_cast<uint4*>(dst + (u + h8) * 8) = hi[j].u;
-    if (u < h8) *reinterpret_cast<uint4*>(dst + u * 8) = lo[j].u;
+    const __nv_bfloat16* gain = is_q ? static_cast<const __nv_bfloat16*>(p.q_norm) + at[j]
+                                     : static_cast<const __nv_bfloat16*>(p.k_norm) + at[j] - p.H * p.dk;
+    float gh[8], gl[8];
+    unpack(load_piece(gain + (u + h8) * 8), gh);
+    if (u < h8) unpack(load_piece(gain + u * 8), gl);
+#pragma unroll
+    for (int r = 0; r < NROW; ++r) {
+      if (r >= rows) break;
+      norm_turn(lo[j][r], hi[j][r], gl, gh, is_q ? s[2 * r] : s[2 * r + 1], u, h8, sn[r], cs[r]);
+      __nv_bfloat16* dst = is_q ? x + r * p.ldp + p.off_q + at[j]
+                                : kc + (static_cast<long long>(head - p.H) * p.R + ring_row(r)) * p.kw;
+      *reinterpret_cast<uint4*>(dst + (u + h8) * 8) = hi[j][r].u;
+      if (u < h8) *reinterpret_cast<uint4*>(dst + u * 8) = lo[j][r].u;
+    }
   }
   for (int i = tid; i < p.G * v8; i += PREP_THREADS) {
     const int g = i / v8, u = i - g * v8;
-    if (i != tid) val = load_piece(x + p.off_v + i * 8);
-    *reinterpret_cast<uint4*>(vc + static_cast<long long>(g) * p.R * p.vw + u * 8) = val.u;
+#pragma unroll
+    for (int r = 0; r < NROW; ++r)
+      if (r < rows)
+        *reinterpret_cast<uint4*>(vc + (static_cast<long long>(g) * p.R + ring_row(r)) * p.vw + u * 8) =
+            load_piece(x + r * p.ldp + p.off_v + i * 8).u;
   }
+}
+
+template <int NI>
+void launch_pieces(const Params& p, cudaStream_t s) {
+  constexpr int NROW = 2;
+  if (p.T >= 64)
+    window_prep_pieces_kernel<NI, NROW><<<dim3((p.T + NROW - 1) / NROW, p.B), PREP_THREADS, 0, s>>>(p);
+  else window_prep_pieces_kernel<NI, 1><<<dim3(p.T, p.B), PREP_THREADS, 0, s>>>(p);
 }
 
 template <typename T>
@@ -204,11 +246,11 @@ extern "C" int ra_window_prep(const ra::window::Params* p, int f32, void* stream
   const int rows = p->B * p->T;
   const int units = (p->H + p->G) * ((p->dk - p->rot_half) / 8);
   if (f32) window::window_prep_kernel<float><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else if (p->dk % 8 || p->dv % 8 || p->rot_half % 8 || units > 4 * window::PREP_THREADS)
+  else if (p->dk % 8 || p->dv % 8 || p->rot_half % 8 || units > 4 * window::PREP_THREADS || p->B > 65535)
     window::window_prep_kernel<__nv_bfloat16><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else if (units <= window::PREP_THREADS) window::window_prep_pieces_kernel<1><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else if (units <= 2 * window::PREP_THREADS) window::window_prep_pieces_kernel<2><<<rows, window::PREP_THREADS, 0, s>>>(*p);
-  else window::window_prep_pieces_kernel<4><<<rows, window::PREP_THREADS, 0, s>>>(*p);
+  else if (units <= window::PREP_THREADS) window::launch_pieces<1>(*p, s);
+  else if (units <= 2 * window::PREP_THREADS) window::launch_pieces<2>(*p, s);
+  else window::launch_pieces<4>(*p, s);
   return check_launch("window_prep_kernel");
 }
 

@@ -127,7 +127,8 @@ def test_stream_beside_embedding(dtype, d):
 # ---------------------------------------------------------------------------------------------- attention alone
 # heads, kv_heads, dim, vdim, window, rotary dims
 SHAPES = [(6, 2, 20, 28, 5, 6), (4, 2, 128, 64, 130, 64), (3, 3, 64, 128, 128, 0), (16, 1, 64, 64, 200, 32),
-          (40, 2, 48, 40, 33, 16), (8, 8, 128, 128, 1, 128), (2, 1, 160, 136, 90, 80), (5, 1, 8, 24, 129, 8)]
+          (40, 2, 48, 40, 33, 16), (8, 8, 128, 128, 1, 128), (2, 1, 160, 136, 90, 80), (5, 1, 8, 24, 129, 8),
+          (32, 8, 128, 128, 70, 64), (48, 2, 128, 64, 90, 0), (72, 8, 112, 16, 50, 48)]
 
 
 def attention_setup(shape, dtype, T, seed=0):
@@ -186,7 +187,7 @@ def attention_error(m, t, dtype, sizes, max_step=8192, context=1024):
     return (got.double().cpu() - attention_reference(m, t)).abs().max().item()
 
 
-ATT_TOL = {torch.float32: 1e-5, torch.bfloat16: 3e-2}
+ATT_TOL = {torch.float32: 5e-5, torch.bfloat16: 3e-2}  # (32-bit angles are off by some 1e-5 at these positions)
 
 
 @pytest.mark.parametrize("dtype", BOTH)
