@@ -19,14 +19,14 @@ constexpr int MAX_HALF = 256;  // (dk <= 512)
 // units of query and key heads of each: the kernel is bound by its instructions, and index arithmetic and gains serve all
 // rows. grid (tokens / NROW, sequences).
 template <int NI, int NROW>
-__global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pieces_kernel(const Params p) {
+__global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 4 : 1) window_prep_pieces_kernel(const Params p) {
   __shared__ __align__(16) float red[2 * NROW][8], sn[NROW][MAX_HALF], cs[NROW][MAX_HALF];
   const int b = blockIdx.y, t0 = blockIdx.x * NROW, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rows = min(NROW, p.T - t0);
   __nv_bfloat16* x = static_cast<__nv_bfloat16*>(p.proj) + (static_cast<long long>(b) * p.T + t0) * p.ldp;
   const int h8 = p.rot_half >> 3, units = (p.dk >> 3) - h8, n = (p.H + p.G) * units, v8 = p.dv >> 3;
   Piece lo[NI][NROW], hi[NI][NROW];
-  int at[NI], unit[NI];  // first dimension of the thread's heads, query heads first; unit, or -1
+  int heads[NI], unit[NI];  // the thread's heads, query heads first, and units (-1: none)
   float s[2 * NROW];
 #pragma unroll
   for (int e = 0; e < 2 * NROW; ++e) s[e] = 0.f;
@@ -34,8 +34,8 @@ __global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pie
   for (int j = 0; j < NI; ++j) {
     const int i = tid + j * PREP_THREADS, head = i / units;
     unit[j] = i < n ? i - head * units : -1;
-    at[j] = head * p.dk;
-    const __nv_bfloat16* src = x + (head < p.H ? p.off_q : p.off_k - p.H * p.dk) + at[j];
+    heads[j] = head;
+    const __nv_bfloat16* src = x + (head < p.H ? p.off_q : p.off_k - p.H * p.dk) + head * p.dk;
 #pragma unroll
     for (int r = 0; r < NROW; ++r)
       if (unit[j] >= 0 && r < rows) {
@@ -54,8 +54,8 @@ __global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pie
     for (int r = 0; r < NROW; ++r)
       if (unit[j] >= 0 && r < rows) {
         const float v = square_sum(hi[j][r]) + (unit[j] < h8 ? square_sum(lo[j][r]) : 0.f);
-        s[2 * r] += at[j] < p.H * p.dk ? v : 0.f;
-        s[2 * r + 1] += at[j] < p.H * p.dk ? 0.f : v;
+        s[2 * r] += heads[j] < p.H ? v : 0.f;
+        s[2 * r + 1] += heads[j] < p.H ? 0.f : v;
       }
 #pragma unroll
   for (int e = 0; e < 2 * NROW; ++e) {
@@ -63,11 +63,13 @@ __global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pie
     if (lane == 0) red[e][warp] = s[e];
   }
   __syncthreads();
-#pragma unroll
-  for (int e = 0; e < 2 * NROW; ++e) {
+  {  // lane e of every warp makes the e-th factor
+    const int e = lane < 2 * NROW ? lane : 0;
     const float4 u = load4(red[e]), w = load4(red[e] + 4);
     const float sum = ((u.x + u.y) + (u.z + u.w)) + ((w.x + w.y) + (w.z + w.w));
-    s[e] = 1.f / sqrtf(sum / (e & 1 ? p.G * p.dk : p.H * p.dk) + p.eps);
+    const float rs = 1.f / sqrtf(sum / (e & 1 ? p.G * p.dk : p.H * p.dk) + p.eps);
+#pragma unroll
+    for (int i = 0; i < 2 * NROW; ++i) s[i] = __shfl_sync(0xffffffffu, rs, i);
   }
   if (!RA_IN_BOUNDS(t0, rows, p.T, kTagWindow)) return;
   const int ring0 = static_cast<int>(static_cast<unsigned>(pos) % static_cast<unsigned>(p.R));
@@ -77,10 +79,10 @@ __global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pie
 #pragma unroll
   for (int j = 0; j < NI; ++j) {
     if (unit[j] < 0) continue;
-    const int u = unit[j], head = at[j] / p.dk;
+    const int u = unit[j], head = heads[j], at = head * p.dk;
     const bool is_q = head < p.H;
-    const __nv_bfloat16* gain = is_q ? static_cast<const __nv_bfloat16*>(p.q_norm) + at[j]
-                                     : static_cast<const __nv_bfloat16*>(p.k_norm) + at[j] - p.H * p.dk;
+    const __nv_bfloat16* gain = is_q ? static_cast<const __nv_bfloat16*>(p.q_norm) + at
+                                     : static_cast<const __nv_bfloat16*>(p.k_norm) + at - p.H * p.dk;
     float gh[8], gl[8];
     unpack(load_piece(gain + (u + h8) * 8), gh);
     if (u < h8) unpack(load_piece(gain + u * 8), gl);
@@ -88,7 +90,7 @@ __global__ void __launch_bounds__(PREP_THREADS, NI <= 2 ? 3 : 1) window_prep_pie
     for (int r = 0; r < NROW; ++r) {
       if (r >= rows) break;
       norm_turn(lo[j][r], hi[j][r], gl, gh, is_q ? s[2 * r] : s[2 * r + 1], u, h8, sn[r], cs[r]);
-      __nv_bfloat16* dst = is_q ? x + r * p.ldp + p.off_q + at[j]
+      __nv_bfloat16* dst = is_q ? x + r * p.ldp + p.off_q + at
                                 : kc + (static_cast<long long>(head - p.H) * p.R + ring_row(r)) * p.kw;
       *reinterpret_cast<uint4*>(dst + (u + h8) * 8) = hi[j][r].u;
       if (u < h8) *reinterpret_cast<uint4*>(dst + u * 8) = lo[j][r].u;
