@@ -529,15 +529,15 @@ class HybridConfig:
             return dict(layers=tuple(LayerConfig(lat if i % 4 == 3 else dl, DenseConfig(ff)) for i in range(n)))
 
         def kalonex(n, heads, kv_heads, dim, window, ff, experts, top, expert_ff, shared_ff):
-            """``n`` layer runs: a dense layer, (n - 2) / 2 passes over a routed and a dense layer, a routed layer. The
-            routed layers' active feed-forward (top experts and the shared one) is as wide as the dense one."""
+            """``n`` layer runs: a dense and a routed layer, then (n - 2) / 2 passes over two more of them. The routed
+            layers' active feed-forward (top experts and the shared one) is as wide as the dense one."""
             if n < 4 or n % 2:
                 raise ValueError("this preset has an even number of layer runs, at least four")
             at = WindowAttentionConfig(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5,
                                        rot=RotaryConfig(10000.0, dim // 2), window=window)
             dense, moe = DenseConfig(ff, gated=True), MoEConfig(experts, top, expert_ff, shared_ff)
             return dict(layers=tuple(LayerConfig(at, f) for f in (dense, moe, dense, moe)),
-                        loop=LoopConfig(1, 3, (n - 2) // 2))
+                        loop=LoopConfig(2, 4, (n - 2) // 2))
 
         presets = {
             "dafelorn-7b": dict(vocab_size=32000, d_model=4096, rms_eps=1e-6,
